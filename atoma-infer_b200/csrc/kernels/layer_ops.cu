@@ -282,6 +282,7 @@ extern "C" int scaled_add_rmsnorm(float* resid, const void* delta, int delta_dty
 //  * the first `rot` dims of every q and k head rotate by position * inv_freq[i], dimension i with i + rot/2;
 //  * with head_norm: after the rotation every q head and every k head is divided by its own root mean square over d
 //    (eps inside the root; no weight);
+//  * with q_head_scale: query head h is multiplied by q_head_scale[h] (what multiplies a query multiplies its scores);
 //  * with v_first: v <- (1 - lambda) v + lambda v_first (the same token's values of an earlier layer, rows of
 //    nkv * dv); with v_out: the layer's values (biases added) are left there for later layers;
 //  * q goes to q_out [T, nq, dp], k and v to the token's slot of its page, heads of dp elements (dp >= d, dv;
@@ -295,7 +296,7 @@ qkv_prepare_kernel(const T* __restrict__ qkv, long long qkv_stride, const TP* __
                    const float* __restrict__ v_lambda, T* __restrict__ v_out, T* __restrict__ q_out,
                    T* __restrict__ cache, int nq, int nkv, int d, int dv, int dp, int page_size, int num_pages,
                    int store_kv, int vec4, int head_norm, int interleaved, float qt_coef, int qt_every,
-                   int* __restrict__ status) {
+                   const float* __restrict__ q_head_scale, int* __restrict__ status) {
     // the q and k parts of the row, then cos[rot / 2], sin[rot / 2] of the token
     extern __shared__ __align__(16) float vals[];
     __shared__ float red[66];
@@ -430,7 +431,7 @@ qkv_prepare_kernel(const T* __restrict__ qkv, long long qkv_stride, const TP* __
                     T* dst = is_q ? q_out + ((size_t)t * nq + h) * dp : kpage + (size_t)(h - nq) * head_block;
                     // k heads follow the q heads in vals; a weight beside a norm per head has d elements, for every head
                     const int base = h * d, nb = head_inv ? 0 : (is_q ? base : base - NQ);
-                    const float inv = (head_inv ? hinv[h] : (is_q ? inv_q : inv_k)) * (is_q ? q_temp : 1.f);
+                    const float inv = (head_inv ? hinv[h] : (is_q ? inv_q : inv_k)) * (is_q ? (q_head_scale ? q_temp * q_head_scale[h] : q_temp) : 1.f);
                     const TP* nw = is_q ? q_norm : k_norm;
                     auto normed4 = [&](int j, float (&o)[4]) {
                         float wv[4] = {1.f, 1.f, 1.f, 1.f};
@@ -517,7 +518,7 @@ qkv_prepare_kernel(const T* __restrict__ qkv, long long qkv_stride, const TP* __
                 } else {
                     r = normed(i);
                 }
-                if (is_q) r *= q_temp;
+                if (is_q) r *= q_head_scale ? q_temp * q_head_scale[h] : q_temp;
             }
             dst[i] = from_float<T>(r);
         }
@@ -541,7 +542,7 @@ extern "C" int qkv_prepare(const void* qkv, long long qkv_stride, int dtype, con
                            const int* positions, const int* token_entry, const int* meta, int group, const float* inv_freq,
                            int rot, const void* v_first, const float* v_lambda, void* v_out, void* q_out, void* cache, int T,
                            int nq, int nkv, int d, int dv, int dp, int page_size, int num_pages, int store_kv, int head_norm,
-                           int interleaved, float qt_coef, int qt_every, int* status, cudaStream_t stream) {
+                           int interleaved, float qt_coef, int qt_every, const float* q_head_scale, int* status, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (interleaved && rot % 2) return (int)cudaErrorInvalidValue;
     const size_t smem = ((size_t)(nq + nkv) * d + rot + (head_norm ? (size_t)(nq + nkv) * (d / 4 + 1) : 0)) * sizeof(float);
@@ -564,7 +565,7 @@ extern "C" int qkv_prepare(const void* qkv, long long qkv_stride, int dtype, con
         return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, qkv_prepare_kernel<TT, TP>, T, threads, smem, stream, \
                                       (const TT*)qkv, qkv_stride, (const TP*)bias, (const TP*)q_norm, (const TP*)k_norm, eps, positions, token_entry, meta, group, inv_freq, rot, \
                                       (const TT*)v_first, v_lambda, (TT*)v_out, (TT*)q_out, (TT*)cache, nq, nkv, d, dv, dp, \
-                                      page_size, num_pages, store_kv, vec4, head_norm, interleaved, qt_coef, qt_every, status); \
+                                      page_size, num_pages, store_kv, vec4, head_norm, interleaved, qt_coef, qt_every, q_head_scale, status); \
     } while (0)
     if (dtype == DT_F32 && param_dtype != DT_F32) return (int)cudaErrorInvalidValue;
     if (dtype == DT_F32) PREP_CASE(float, float, 0);

@@ -100,6 +100,112 @@ extern "C" int moe_route_biased(const void* h, int dtype, const float* w, const 
                                   (const __nv_bfloat16*)h, w, ids, wts, meta, H, E, top, bias, over_chosen);
 }
 
+// Sigmoid scores, a correction that only the choice sees, choice within the best groups.  Per token: s_e = sigmoid(w_router[e] .
+// h) (float32, the logits as above), choice score c_e = s_e + correction[e].  With groups > 1 the experts form that many equal
+// groups of neighbours; a group's score is the sum of its two largest choice scores (its only one in groups of one), and only
+// experts of the `keep` best groups can be chosen.  The `top` largest choice scores choose (ties to the lower index, for
+// groups too); the weights are the chosen experts' s as they are.  The choice runs on the first warp.
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_route_sigmoid_kernel(const T* __restrict__ h, const float* __restrict__ w, const float* __restrict__ correction,
+                         int* __restrict__ ids, float* __restrict__ wts, const int* __restrict__ meta, int H, int E, int top, int groups,
+                         int keep) {
+    extern __shared__ float z[];  // E scores, E choice scores, `groups` group scores, `groups` marks
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t = blockIdx.x;
+    if (t >= meta[META_NUM_TOKENS]) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const T* x = h + (size_t)t * H;
+    const bool vec = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
+    float *c = z + E, *gs = c + E;
+    for (int e = warp; e < E; e += nwarps) {
+        const float* we = w + (size_t)e * H;
+        float acc = 0.f;
+        if (vec) {
+            float part[4] = {0.f, 0.f, 0.f, 0.f};
+            for (int k = lane * 4; k < H; k += 128) {
+                float xv[4], wv[4];
+                load4(x + k, xv);
+                load4(we + k, wv);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) part[i] = fmaf(xv[i], wv[i], part[i]);
+            }
+            acc = (part[0] + part[1]) + (part[2] + part[3]);
+        } else {
+            for (int k = lane; k < H; k += 32) acc = fmaf(to_float(x[k]), we[k], acc);
+        }
+        acc = warp_sum(acc);
+        if (lane == 0) {
+            const float s = 1.f / (1.f + expf(-acc));
+            z[e] = s;
+            c[e] = s + correction[e];
+        }
+    }
+    __syncthreads();
+    if (warp != 0) return;
+    // the largest of n values in shared memory, ties to the lower index; the winner is struck out
+    auto take_best = [&](float* v, int n) {
+        float bv = -INFINITY;
+        int best = n;
+        for (int i = lane; i < n; i += 32)
+            if (v[i] > bv) { bv = v[i]; best = i; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, best, o);
+            if (ov > bv || (ov == bv && oi < best)) { bv = ov; best = oi; }
+        }
+        __syncwarp();
+        if (best < n && lane == 0) v[best] = -INFINITY;
+        __syncwarp();
+        return best;
+    };
+    if (groups > 1) {
+        const int per = E / groups;
+        int* kept = reinterpret_cast<int*>(gs + groups);
+        for (int g = lane; g < groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;
+            for (int i = g * per; i < (g + 1) * per; ++i) {
+                if (c[i] > a) { b = a; a = c[i]; }
+                else if (c[i] > b) b = c[i];
+            }
+            gs[g] = per > 1 ? a + b : a;
+            kept[g] = 0;
+        }
+        __syncwarp();
+        for (int k = 0; k < keep; ++k) {
+            const int g = take_best(gs, groups);
+            if (g < groups && lane == 0) kept[g] = 1;
+            __syncwarp();
+        }
+        for (int e = lane; e < E; e += 32)
+            if (!kept[e / per]) c[e] = -INFINITY;
+        __syncwarp();
+    }
+    for (int k = 0; k < top; ++k) {
+        int best = take_best(c, E);
+        if (best >= E) best = 0;  // (scores that are no numbers: any expert)
+        if (lane == 0) {
+            ids[(size_t)t * top + k] = best;
+            wts[(size_t)t * top + k] = z[best];
+        }
+    }
+}
+
+extern "C" int moe_route_sigmoid(const void* h, int dtype, const float* w, const float* correction, int* ids, float* wts, const int* meta,
+                                 int T, int H, int E, int top, int groups, int keep, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    const size_t smem = ((size_t)2 * E + (groups > 1 ? 2 * groups : 0)) * sizeof(float);
+    if (smem > 48 * 1024 || top > E || groups < 1 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < top)
+        return (int)cudaErrorInvalidValue;
+    if (dtype == DT_F32)
+        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, moe_route_sigmoid_kernel<float>, T, 256, smem, stream, (const float*)h, w,
+                                      correction, ids, wts, meta, H, E, top, groups, keep);
+    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, moe_route_sigmoid_kernel<__nv_bfloat16>, T, 256, smem, stream,
+                                  (const __nv_bfloat16*)h, w, correction, ids, wts, meta, H, E, top, groups, keep);
+}
+
 // ----------------------------------------------------------------------------- pairs sorted by expert
 // One block.  offsets[e] .. offsets[e + 1] is expert e's stretch of `order`, which lists its pairs (token * top + choice)
 // in ascending order.  A warp takes the experts e = warp, warp + warps, ...: it walks all pairs 32 at a time and

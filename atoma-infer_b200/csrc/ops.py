@@ -30,9 +30,12 @@ GEMM_SOURCES = ["kernels/gemm_tcgen05.cu"]
 ATTENTION_TC_SOURCES = ["kernels/attention_tcgen05.cu"]
 DECODE_STACK_SOURCES = ["kernels/decode_stack.cu"]
 # parallel blocks, state-space mixers, latent attention, routed experts: built when a model first uses one of them
-MIXER_SOURCES = ["kernels/stream_ops.cu", "kernels/ssm.cu", "kernels/latent.cu", "kernels/moe.cu", "kernels/gated_stream.cu"]
+MIXER_SOURCES = ["kernels/stream_ops.cu", "kernels/ssm.cu", "kernels/latent.cu", "kernels/moe.cu", "kernels/gated_stream.cu",
+                 "kernels/normed_stream.cu", "kernels/talking_heads.cu"]
 # recurrences whose decay differs from row to row (gated linear attention, the selective scan): built at first use too
 RECURRENT_SOURCES = ["kernels/recurrent.cu"]
+# recurrences whose query reads more than the decayed state (a bonus for the current token, a memory with a normalizer)
+MATRIX_RECURRENT_SOURCES = ["kernels/matrix_recurrent.cu"]
 ATTENTION_TC_HEAD_DIMS = (64, 128)  # head sizes of the tcgen05 prefill attention
 ATTENTION_HEAD_DIMS = tuple(range(16, 257, 16))  # every head size the kernels take; the build check builds them all, a model only its own
 
@@ -128,7 +131,7 @@ class CudaOps:
         self.lib.kernels_set_pdl(int(on))
         for lib in self._attn_libs.values():
             lib.kernels_set_pdl(1 if on else 0)
-        for name in ("_mixer_lib", "_recurrent_lib"):
+        for name in ("_mixer_lib", "_recurrent_lib", "_matrix_recurrent_lib"):
             if getattr(self, name, None) is not None:
                 getattr(self, name).kernels_set_pdl(int(on))
 
@@ -268,6 +271,13 @@ class CudaOps:
             return out
         return y
 
+    def linears(self, x, w, *, meta=None):
+        """Several linears of one size, each with rows of its own: x [n, M, K], w [n, N, K] -> n results [M, N]."""
+        n, M, K = x.shape
+        if x.dtype == torch.bfloat16 and M > SKINNY_MAX_ROWS:
+            return tuple(torch.bmm(x, w.transpose(1, 2)))
+        return tuple(self.linear(x[i], w[i], meta=meta) for i in range(n))
+
     def linear_streamed(self, x, w, *, out_dtype=None, silu_mul: bool = False, scale_from=None, add_into=None):
         """``linear`` on the TMA-fed persistent kernel whatever the policy says (bfloat16, at most 16 rows, K a multiple
         of 64, contiguous operands).  An RMSNorm can be folded into the linears around it:
@@ -391,7 +401,7 @@ class CudaOps:
     def qkv_prepare(self, qkv, ctx, cache_layer, group: int, q_out, *, nq: int, nkv: int, d: int, dv: int, dp: int,
                     page_size: int, num_pages: int, store_kv: bool, bias=None, q_norm=None, k_norm=None, eps: float = 0.0,
                     inv_freq=None, rot: int = 0, v_first=None, v_lambda=None, v_out=None, head_norm: bool = False,
-                    interleaved: bool = False, q_temp=None):
+                    interleaved: bool = False, q_temp=None, q_head_scale=None):
         """Rows [q | k | v] of the fused projection become attention's inputs: biases, root-mean-square norms over
         the whole q and the whole k part (weights ``q_norm`` / ``k_norm``), rotation of the first ``rot`` dims of
         every head, with ``head_norm`` every q and k head divided by its own root mean square (``eps``) after the rotation,
@@ -400,11 +410,14 @@ class CudaOps:
         ``bias``, ``q_norm`` and ``k_norm`` share one type, float32 or (beside bfloat16 rows) bfloat16.
         With ``head_norm`` AND weights, the weights have ``d`` elements, shared by all heads, and the norm comes before the
         rotation.  ``interleaved``: the rotation pairs dimension 2i with 2i + 1 (else i with i + rot / 2).  ``q_temp`` =
-        (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)."""
+        (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).  ``q_head_scale``
+        (float32 [nq]): query head h is multiplied by its h-th number."""
         if head_norm and (q_norm is not None or k_norm is not None) and (q_norm is None or k_norm is None
                                                                            or q_norm.numel() != d or k_norm.numel() != d):
             raise KernelError("weights beside a norm per head have the head's size, for queries and for keys")
         qt_coef, qt_every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
+        if q_head_scale is not None and (q_head_scale.dtype != torch.float32 or q_head_scale.numel() != nq):
+            raise KernelError("a scale per query head is one float32 number per head")
         params = [t for t in (bias, q_norm, k_norm) if t is not None]
         if len({t.dtype for t in params}) > 1:
             raise KernelError("biases and norm weights of the attention rows must share one type")
@@ -414,7 +427,7 @@ class CudaOps:
                                          _p(ctx.positions), _p(ctx.token_entry), _p(ctx.meta), max(group, 0), _p(inv_freq),
                                          int(rot) if inv_freq is not None else 0, _p(v_first), _p(v_lambda), _p(v_out),
                                          _p(q_out), _p(cache_layer), ctx.T, nq, nkv, d, dv, dp, page_size, num_pages,
-                                         int(store_kv), int(head_norm), int(interleaved), ctypes.c_float(qt_coef), qt_every,
+                                         int(store_kv), int(head_norm), int(interleaved), ctypes.c_float(qt_coef), qt_every, _p(q_head_scale),
                                          _p(self.status), self._stream()), "qkv_prepare")
 
     def narrow(self, x, dtype):
@@ -913,6 +926,161 @@ class CudaOps:
         self.launches += 1
         self._check(lib.moe_combine(_p(y), DT_F32, None, _p(wts), _p(shared), _p(out), _code(out), _p(meta), T, top, H,
                                     self._stream()), "moe_combine")
+
+    def moe_route_sigmoid(self, h, w_router, correction, ids, wts, meta, groups=None):
+        """Per token: scores s = sigmoid(w_router h) in float32, choice scores s + ``correction`` (float32 [experts]); the
+        ids.shape[1] largest choice scores (ties to the lower index) into ``ids``, the chosen experts' s as they are into
+        ``wts``.  ``groups`` = (count, keep): the experts form that many equal groups of neighbours, and only experts of the
+        ``keep`` groups whose two largest choice scores sum highest can be chosen."""
+        E, H = w_router.shape
+        count, keep = groups or (1, 1)
+        self._check(self._mixers().moe_route_sigmoid(_p(h), _code(h), _p(w_router), _p(correction), _p(ids), _p(wts), _p(meta),
+                                                     h.shape[0], H, E, ids.shape[1], int(count), int(keep), self._stream()),
+                    "moe_route_sigmoid")
+
+    # ------------------------------------------------------------------ blocks whose only norm stands on a sublayer's result
+    def norm_add(self, resid, pending, w, eps: float, ctx, *, layer_norm: bool, out=None):
+        """resid[t] += norm(y[t]) * w with y = mult * (f0 n0(t0[t]) + f1 n1(t1[t]) + ...) + vector, the terms, weights, norms,
+        factor and vector of ``pending`` (a ``PendingSum``; up to four terms of one type; n_j divides a term by its root mean
+        square over the width and multiplies it by a weight where the sum says so).  ``layer_norm``: the norm takes the mean off
+        first.  ``out``: the new rows in the compute type, the next sublayer's input."""
+        terms, norms = list(pending.terms), list(pending.term_norms())
+        if not 0 < len(terms) <= 4 or len({t.dtype for t in terms}) > 1:
+            raise KernelError("a normed sum has one to four terms, of one type")
+        if pending.rows is not None:
+            raise KernelError("a normed sum has terms, weights, norms, a factor and a vector only")
+        n = len(terms)
+        ptrs = (ctypes.c_void_p * 4)(*[t.data_ptr() for t in terms])
+        facs = (ctypes.c_float * 4)(*pending.weights())
+        wptrs = (ctypes.c_void_p * 4)(*[nm[0].data_ptr() if nm is not None else None for nm in norms])
+        weps = (ctypes.c_float * 4)(*[float(nm[1]) if nm is not None else 0.0 for nm in norms])
+        self._check(self._mixers().norm_add(_p(resid), n, ptrs, facs, wptrs, weps, _code(terms[0]), ctypes.c_float(pending.mult),
+                                            _p(pending.vector), _p(w), ctypes.c_float(eps), int(layer_norm), _p(out),
+                                            _code(out) if out is not None else _code(terms[0]), _p(ctx.meta), ctx.T, resid.shape[1],
+                                            self._stream()), "norm_add")
+
+    def layer_norm(self, resid, w, eps: float, out, meta, n: int, rows=None):
+        """out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w of the float32 rows (of ``rows`` alone if given)."""
+        self._check(self._mixers().layer_norm_rows(_p(resid), _p(rows), _p(w), ctypes.c_float(eps), _p(out), _code(out), _p(meta), n,
+                                                   resid.shape[1], self._stream()), "layer_norm_rows")
+
+    @staticmethod
+    def _kept_row(state, H: int, what: str):
+        if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] != H:
+            raise KernelError(f"{what}: the kept row is float32 [slots, H] with contiguous rows")
+        return ctypes.c_longlong(state.stride(0))
+
+    def token_mix(self, x, mu, state, ctx, out) -> bool:
+        """out[k, t] = x[t] + (x[t - 1] - x[t]) * mu[k] for every weight of ``mu`` (float32 [count, H]); x[t - 1] is the row of
+        the token before in the same request: of this step, the row kept in ``state`` (float32 [slots, H] with a slot
+        stride), or zeros at position 0.  Returns whether the kept rows have been replaced too (steps of one token per entry);
+        if not, ``keep_last_rows`` does it afterwards."""
+        count, H = mu.shape
+        stride = self._kept_row(state, H, "token_mix")
+        if not x.is_contiguous() or not out.is_contiguous() or tuple(out.shape) != (count, ctx.T, H):
+            raise KernelError("token_mix: rows [T, H] and results [count, T, H] are contiguous")
+        save = bool(ctx.decode_only and ctx.T == ctx.S)
+        self._check(self._mixers().token_mix(_p(x), _code(x), _p(mu), count, _p(state), stride, _p(out), _code(out), _p(ctx.meta),
+                                             _p(ctx.positions), _p(ctx.token_entry), _p(ctx.cu_tokens), _p(ctx.state_slots), ctx.T, H,
+                                             int(save), self._stream()), "token_mix")
+        return save
+
+    def keep_last_rows(self, x, state, ctx):
+        """Every entry's last row of x goes to its slot of ``state`` (see ``token_mix``)."""
+        stride = self._kept_row(state, x.shape[1], "keep_last_rows")
+        self._check(self._mixers().keep_last_rows(_p(x), _code(x), _p(state), stride, _p(ctx.meta), _p(ctx.cu_tokens),
+                                                  _p(ctx.state_slots), ctx.S, x.shape[1], self._stream()), "keep_last_rows")
+
+    def tanh_rows(self, z, out, meta):
+        """out = tanh(z): float32 rows in, rounded once to the type of ``out``."""
+        self._check(self._mixers().tanh_rows(_p(z), _p(out), _code(out), _p(meta), z.shape[0], z.shape[1], self._stream()), "tanh_rows")
+
+    # ------------------------------------------------------------------ attention with weights mixed across heads
+    def talking_attention(self, q, q_stride: int, cache_layer, ctx, group: int, out, nq: int, nkv: int, d: int, page_size: int,
+                          num_pages: int, scale: float, talk, *, chunk: int = 0):
+        """Attention over what the requests have cached whose softmax weights are mixed across the query heads, p'_h = sum_g
+        talk[h, g] p_g, before head h weighs the values of its own key/value head; ``talk`` float32 [nq, nq].  ``chunk`` as for
+        ``attention``."""
+        if talk.dtype != torch.float32 or tuple(talk.shape) != (nq, nq) or not talk.is_contiguous():
+            raise KernelError("the heads' mixing weights are contiguous float32 [heads, heads]")
+        self._check(self._mixers().talk_attn_plain(_p(q), q_stride, _p(cache_layer), _code(q), _p(ctx.meta), group, _p(ctx.token_entry),
+                                                   _p(ctx.positions), _p(out), ctx.T, nq, nkv, d, page_size, num_pages, int(chunk),
+                                                   ctypes.c_float(scale), _p(talk), _p(self.status), self._stream()), "talk_attn_plain")
+
+    # ------------------------------------------------------------------ recurrences whose query reads more than the decayed state
+    def _matrix_recurrent(self):
+        lib = getattr(self, "_matrix_recurrent_lib", None)
+        if lib is None:
+            lib = self._matrix_recurrent_lib = build.load_library("matrix_recurrent", MATRIX_RECURRENT_SOURCES, cuda=True)
+            lib.bonus_scan_scratch_floats.restype = ctypes.c_size_t
+            lib.memory_scan_scratch_floats.restype = ctypes.c_size_t
+            lib.kernels_set_pdl(int(self.pdl))
+        return lib
+
+    def bonus_scan(self, r, k, v, z, z_bias, bonus, state, ctx, o, *, heads: int, dim: int, vdim: int):
+        """Per head o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T r_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T with w_t =
+        exp(-exp(z_t + z_bias)).  r, k [T, heads * dim] and v [T, heads * vdim] are slices of wider rows, ``z`` float32
+        [T, heads * dim], ``z_bias`` and ``bonus`` float32 [heads * dim], ``state`` float32 [slots, heads, dim, vdim] (read and
+        updated), ``o`` float32 [T, heads * vdim]."""
+        lib = self._matrix_recurrent()
+        slot_stride = self._slot_state(state, (heads, dim, vdim), "bonus_scan")
+        if z.dtype != torch.float32 or o.dtype != torch.float32 or not o.is_contiguous():
+            raise KernelError("bonus_scan: decay logits and outputs are float32")
+        if bonus.numel() != heads * dim or z_bias.numel() != heads * dim:
+            raise KernelError("bonus_scan: bonus and the logits' bias are one number per head and key channel")
+        (rp, rs), (kp, ks), (vp, vs), (zp, zs) = (self._rows(t, "bonus_scan") for t in (r, k, v, z))
+        chunk, chunks = self._scan_chunks(ctx)
+        scratch = (torch.empty(lib.bonus_scan_scratch_floats(ctx.S, heads, dim, vdim, chunks), dtype=torch.float32, device=o.device)
+                   if chunk else None)
+        self._check(lib.bonus_scan(rp, rs, kp, ks, vp, vs, _code(r), zp, zs, _p(z_bias), _p(bonus), _p(state), slot_stride, _p(o),
+                                   _p(ctx.meta), _p(ctx.cu_tokens), _p(ctx.state_slots), ctx.S, heads, dim, vdim, chunk, chunks,
+                                   _p(scratch), self._stream()), "bonus_scan")
+        if chunk:
+            self.launches += 2
+
+    def memory_scan(self, q, k, v, logits, bias, cap: float, q_scale: float, state, n_state, m_state, ctx, o, nq, floor, *, heads: int,
+                    dim: int, vdim: int):
+        """The matrix memory with exponential gates: i = cap tanh((x_i + b_i) / cap), f = log sigmoid(cap tanh((x_f + b_f) / cap))
+        from ``logits`` (float32 [T, 2 * heads], the input gates' first) and ``bias`` (float32 [2 * heads]); m_t = max(f + m_(t-1),
+        i); S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k_t v_t^T, n_t likewise with k alone; ``o`` = S_t^T (q_scale q_t)
+        (float32 [T, heads * vdim]), ``nq`` = n_t . (q_scale q_t) and ``floor`` = exp(-m_t) (float32 [T, heads]), which
+        ``head_weight_norm_gate`` divides by.  The states (float32, read and updated, views with one slot stride): ``state``
+        [slots, heads, dim, vdim], ``n_state`` [slots, heads, dim], ``m_state`` [slots, heads]."""
+        lib = self._matrix_recurrent()
+        slot_stride = self._slot_state(state, (heads, dim, vdim), "memory_scan")
+        n_stride = self._slot_state(n_state, (heads, dim), "memory_scan")
+        if n_stride.value != slot_stride.value or m_state.stride(0) != slot_stride.value or m_state.stride(1) != 1:
+            raise KernelError("memory_scan: the three parts of a request's state share one slot")
+        for t in (logits, o, nq, floor):
+            if t.dtype != torch.float32 or not t.is_contiguous():
+                raise KernelError("memory_scan: gate logits and outputs are contiguous float32")
+        if logits.shape[1] != 2 * heads or bias.numel() != 2 * heads:
+            raise KernelError("memory_scan: two gates per head")
+        (qp, qs), (kp, ks), (vp, vs) = (self._rows(t, "memory_scan") for t in (q, k, v))
+        gates = torch.empty((ctx.T, heads, 2), dtype=torch.float32, device=o.device)
+        self._check(lib.memory_gates(_p(logits), _p(bias), ctypes.c_float(cap), _p(m_state), slot_stride, _p(gates), _p(floor),
+                                     _p(ctx.meta), _p(ctx.cu_tokens), _p(ctx.state_slots), ctx.S, heads, ctx.max_tokens_per_entry,
+                                     self._stream()), "memory_gates")
+        chunk, chunks = self._scan_chunks(ctx)
+        scratch = (torch.empty(lib.memory_scan_scratch_floats(ctx.S, heads, dim, vdim, chunks), dtype=torch.float32, device=o.device)
+                   if chunk else None)
+        self._check(lib.memory_scan(qp, qs, kp, ks, vp, vs, _code(q), _p(gates), ctypes.c_float(q_scale), _p(state), _p(n_state),
+                                    slot_stride, _p(o), _p(nq), _p(ctx.meta), _p(ctx.cu_tokens), _p(ctx.state_slots), ctx.S, heads, dim,
+                                    vdim, chunk, chunks, _p(scratch), self._stream()), "memory_scan")
+        if chunk:
+            self.launches += 2
+
+    def head_weight_norm_gate(self, o, gate, w, eps: float, out, meta, heads: int, *, kind: str, nq=None, floor=None):
+        """out[t, h] = v / sqrt(mean(v^2) + eps) * w[h] * gate_fn(gate[t, h]) with v = o[t, h], or with ``nq`` and ``floor`` (float32
+        [T, heads]) v = o[t, h] / (max(|nq|, floor) + 1e-6).  ``o`` float32 [T, heads * P], ``gate`` a slice of wider rows, ``w``
+        float32 [heads * P]; ``kind``: "sigmoid" or "silu"."""
+        gp, gs = self._rows(gate, "head_weight_norm_gate")
+        if w.numel() != o.shape[1] or w.dtype != torch.float32:
+            raise KernelError("head_weight_norm_gate: one float32 weight per channel of every head")
+        self._check(self._matrix_recurrent().head_weight_norm_gate(_p(o), _p(nq), _p(floor), gp, _code(gate), gs, _p(w),
+                                                                   ctypes.c_float(eps), {"sigmoid": 0, "silu": 1}[kind], _p(out), _p(meta),
+                                                                   o.shape[0], heads, o.shape[1] // heads, self._stream()),
+                    "head_weight_norm_gate")
 
     # ------------------------------------------------------------------ whole layers of a decode step
     def _decode_stack_library(self, d: int):

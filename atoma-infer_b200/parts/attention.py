@@ -40,6 +40,9 @@ the mixer's result into the stream takes in float32);
 ``sink: "learned"``: the sink's score is a learned number per head (``.sink``), not 0;
 ``head_gate``: head h's output is multiplied by sigmoid(W_g x)_h, one number per head (W_g [heads, hidden] joins the fused
 matrix).
+``head_scale``: head h's scores are multiplied by a learned number per head (``.temp``; it multiplies the query);
+``talk``: the softmax weights are mixed across the heads, p_h <- sum_g T[h, g] p_g with a learned T [heads, heads] (``.talk``),
+before head h weighs the values of its own key/value head (goes with ``chunk``; not with a window, a sink or score options).
 The position encoding's ``interleaved`` pairs dimension 2i with 2i + 1.
 With any of ``v_head_dim``, ``bias``, ``qk_norm``, ``v_mix``, ``head_norm`` (and the options above that touch the rows) the rows are prepared by one kernel (``qkv_prepare``) that writes queries, keys and values
 as heads of one padded size, the next multiple of 16 above both sizes, which the tensor-core kernels read like any
@@ -88,6 +91,9 @@ class Attention(Mixer):
         self.taps = int(p.get("conv") or 0)
         self.head_gate = bool(p.get("head_gate", False))
         self.learned_sink = p.get("sink") == "learned"
+        self.head_scale, self.talk = bool(p.get("head_scale", False)), bool(p.get("talk", False))
+        if self.talk and (self.window or self.sink or self.softcap or self.distance_bias):
+            raise ValueError("talk goes with plain scores over all keys or a chunk of them")
         if self.gate and self.head_gate:
             raise ValueError("gate and head_gate exclude each other")
         if self.keep_first and not self.window:
@@ -95,12 +101,12 @@ class Attention(Mixer):
         interleaved = bool((p.get("position") or {}).get("interleaved", False))
         self.prepared = bool(self.bias or self.qk_norm is not None or self.v_mix is not None or self.head_norm is not None
                              or self.gate or self.v_head_dim != self.head_dim or interleaved or self.q_temp or self.taps
-                             or self.head_gate)
+                             or self.head_gate or self.head_scale or self.talk)
         self.padded_dim = -(-max(self.head_dim, self.v_head_dim) // 16) * 16 if self.prepared else self.head_dim
         self.names = {"q": ".q_proj.weight", "k": ".k_proj.weight", "v": ".v_proj.weight", "o": ".o_proj.weight",
                       "q_bias": ".q_proj.bias", "k_bias": ".k_proj.bias", "v_bias": ".v_proj.bias",
                       "q_norm": ".q_norm.weight", "k_norm": ".k_norm.weight", "v_mix": ".v_mix", "gate": ".g_proj.weight",
-                      "o_bias": ".o_proj.bias", "sink": ".sink", "conv": ".conv", **(p.get("names") or {})}
+                      "o_bias": ".o_proj.bias", "sink": ".sink", "conv": ".conv", "temp": ".temp", "talk": ".talk", **(p.get("names") or {})}
         pos = dict(p.get("position") or {"kind": "none"})
         pos.setdefault("head_dim", self.head_dim)
         self.position = part_class("position", pos["kind"])(pos, prefix)
@@ -160,6 +166,10 @@ class Attention(Mixer):
             decls.append(TensorDecl(pre + n["o_bias"], (self.hidden,)))
         if self.learned_sink:
             decls.append(TensorDecl(pre + n["sink"], (self.num_heads,)))
+        if self.head_scale:
+            decls.append(TensorDecl(pre + n["temp"], (self.num_heads,), init="ones"))
+        if self.talk:
+            decls.append(TensorDecl(pre + n["talk"], (self.num_heads, self.num_heads)))
         if self.head_gate:
             decls.append(TensorDecl(pre + n["gate"], (self.num_heads, self.hidden)))
         if self.taps:
@@ -182,6 +192,8 @@ class Attention(Mixer):
         f32 = lambda name: tensors[pre + n[name]].to(torch.float32).contiguous()  # noqa: E731  (exact widening)
         self.b_o = f32("o_bias") if self.out_bias else None
         self.sinks = f32("sink") if self.learned_sink else None
+        self.w_temp = f32("temp") if self.head_scale else None
+        self.w_talk = f32("talk") if self.talk else None
         # slope_h = 2^(-8 (h + 1) / heads), taken in float64 and rounded once
         self.slopes = (torch.tensor([2.0 ** (-8.0 * (h + 1) / self.num_heads) for h in range(self.num_heads)], dtype=torch.float64)
                        .to(torch.float32).to(rt.device).contiguous() if self.distance_bias else None)
@@ -250,12 +262,17 @@ class Attention(Mixer):
                         v_lambda=self.v_lambda if v_first is not None else None, v_out=v_out,
                         **({"head_norm": True} if self.head_norm is not None else {}),
                         **({"interleaved": True} if getattr(self.position, "interleaved", False) else {}),
-                        **({"q_temp": (float(self.q_temp["coef"]), int(self.q_temp["every"]))} if self.q_temp else {}))
+                        **({"q_temp": (float(self.q_temp["coef"]), int(self.q_temp["every"]))} if self.q_temp else {}),
+                        **({"q_head_scale": self.w_temp} if self.head_scale else {}))
         out = torch.empty((ctx.T, H * dp), dtype=x.dtype, device=x.device)
-        scores = self._score_options()
-        ops.attention(q, H * dp, cache.pages, ctx, cache.group, out, H, G, dp, cache.page_size, cache.num_pages,
-                      int(self.window or 0), self.scale, chunk=self.chunk, sink=self.sinks if self.learned_sink else self.sink,
-                      **scores)
+        if self.talk:
+            ops.talking_attention(q, H * dp, cache.pages, ctx, cache.group, out, H, G, dp, cache.page_size, cache.num_pages,
+                                  self.scale, self.w_talk, chunk=self.chunk)
+        else:
+            scores = self._score_options()
+            ops.attention(q, H * dp, cache.pages, ctx, cache.group, out, H, G, dp, cache.page_size, cache.num_pages,
+                          int(self.window or 0), self.scale, chunk=self.chunk, sink=self.sinks if self.learned_sink else self.sink,
+                          **scores)
         if self.gate:
             ops.sigmoid_gate(out.view(ctx.T, H, dp)[:, :, :self.v_head_dim], gate, ctx.meta)
         elif self.head_gate:

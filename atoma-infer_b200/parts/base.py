@@ -70,7 +70,8 @@ class StepContext:
     table_offsets: Sequence[int] = ()   # per cache group: where its block tables start in ``meta`` ...
     table_strides: Sequence[int] = ()   # ... and how long a request's row is
     # What one layer leaves for later layers of the same step (an earlier layer's values that later ones mix in,
-    # for instance), by a name the parts agree on.  Lives as long as the step.
+    # for instance), by a name the parts agree on.  Lives as long as the step.  ``"mixer_rows"``: a block whose mixer reads the
+    # stream itself leaves the float32 rows there of which the mixer's input is the rounding.
     shared: Dict[str, Any] = field(default_factory=dict)
 
     def block_table(self, group: int) -> torch.Tensor:
@@ -89,16 +90,36 @@ class PendingSum:
     result is a weighted sum of several outputs; the sum is then ((f0 t0 + f1 t1) + ...) in this order.  A mixer may
     return a ``PendingSum`` of terms and factors instead of a tensor.  The norm that follows (``Norm.forward``) takes the
     sum in float32, term by term in this order, in the pass in which it also norms the updated row; a block that has no
-    norm for it calls ``apply_pending``."""
+    norm for it calls ``apply_pending``.  ``norms``: per term None, or (weight float32 [H], eps): the term is divided by its
+    root mean square over the width and multiplied by the weight before it is weighed (None: no term is).  A block that
+    norms a sublayer's result takes such a sum in one pass; everywhere else ``without_norms`` makes the terms first."""
 
     terms: Sequence[torch.Tensor] = ()
     mult: float = 1.0
     rows: Optional[torch.Tensor] = None
     vector: Optional[torch.Tensor] = None
     factors: Optional[Sequence[float]] = None
+    norms: Optional[Sequence[Any]] = None
+
+    def term_norms(self) -> Sequence[Any]:
+        return tuple(self.norms) if self.norms is not None else (None,) * len(self.terms)
 
     def weights(self) -> Sequence[float]:
         return tuple(self.factors) if self.factors is not None else (1.0,) * len(self.terms)
+
+
+def without_norms(ops, pending, ctx: "StepContext"):
+    """The same sum with every normed term replaced by its normed rows, in the terms' type."""
+    if not isinstance(pending, PendingSum) or pending.norms is None:
+        return pending
+    terms = []
+    for t, nm in zip(pending.terms, pending.term_norms()):
+        if nm is not None:
+            out = torch.empty_like(t)
+            ops.rms_rows(t, nm[0], nm[1], out, ctx.meta)
+            t = out
+        terms.append(t)
+    return PendingSum(tuple(terms), pending.mult, pending.rows, pending.vector, pending.factors)
 
 
 def join_terms(parts, mult: float = 1.0) -> "PendingSum":
@@ -107,7 +128,7 @@ def join_terms(parts, mult: float = 1.0) -> "PendingSum":
     terms, factors = [], []
     for p in parts:
         if isinstance(p, PendingSum):
-            if p.rows is not None or p.vector is not None:
+            if p.rows is not None or p.vector is not None or p.norms is not None:
                 raise ValueError("a sublayer's result has terms and factors only")
             terms += list(p.terms)
             factors += [p.mult * f for f in p.weights()]
@@ -122,6 +143,7 @@ def apply_pending(ops, resid: torch.Tensor, delta, ctx: "StepContext") -> None:
     if delta is None:
         return
     if isinstance(delta, PendingSum):
+        delta = without_norms(ops, delta, ctx)
         ops.sum_rmsnorm(resid, delta, None, 0.0, None, ctx.meta, ctx.T)
     else:
         resid.add_(delta)

@@ -10,7 +10,8 @@ sequence filter (f1, f2: a short convolution over time, whose state the block ke
 ``norm``, ``mixer``, ``feed_forward`` (None: the layer has no second sublayer), ``alpha``, ``filter`` (spec or
 None), ``names``.
 
-Parallel and sandwich arrangements: see ``ParallelBlock`` and ``SandwichBlock``.
+Parallel and sandwich arrangements: see ``ParallelBlock`` and ``SandwichBlock``.  Norms on the results alone: see
+``ResultNormBlock``.
 """
 from __future__ import annotations
 
@@ -21,7 +22,7 @@ import torch
 
 from ..config.registry import part_class, register_part
 from ..weights.loader import TensorDecl
-from .base import Block, PendingSum, apply_pending, join_terms
+from .base import Block, PendingSum, apply_pending, join_terms, without_norms
 
 _DEFAULT_NAMES = {"norm1": "input_layernorm", "mixer": "self_attn", "norm2": "post_attention_layernorm",
                   "feed_forward": "mlp"}
@@ -305,7 +306,7 @@ class SandwichBlock(Block):
             last = torch.empty((ctx.S, W), dtype=torch.float32, device=dev)
         ops.norm_shift(resid, self.norm1.weight, self.norm1.eps, ctx, shift=self.mu, state=kept, h=h,
                        hs=hs if self.shift else None, last=last)
-        a = self.mixer.forward(hs, ctx, mixer_cache)
+        a = without_norms(ops, self.mixer.forward(hs, ctx, mixer_cache), ctx)
         if not isinstance(a, PendingSum):
             a = PendingSum((a,))
         g = ops.linear(h, self.w_gate1, out_dtype=torch.float32, meta=ctx.meta)
@@ -325,3 +326,69 @@ class SandwichBlock(Block):
 
 
 register_part("block", "sandwich", SandwichBlock)
+
+
+class ResultNormBlock(Block):
+    """Norms on the sublayers' results only: x <- x + norm1(mixer(x)); x <- x + norm2(ff(x)).
+
+    The sublayers read the stream itself, rounded to the compute type; a mixer that needs its rows as they are finds them
+    under ``ctx.shared["mixer_rows"]``.  The kernel that norms a result adds it into the float32 stream and leaves the next
+    sublayer's input, also the next block's (``ctx.shared["prepared_input"]``), so the block leaves nothing pending.
+    Parameters: ``norm``, ``mixer``, ``feed_forward`` (None: the mixer alone), ``names``."""
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        names = {"norm1": "norm1", "norm2": "norm2", "mixer": "mix", "feed_forward": "mlp", **(params.get("names") or {})}
+        mk = lambda fam, spec, name: part_class(fam, spec["kind"])(spec, f"{prefix}.{name}")  # noqa: E731
+        self.norm1 = mk("norm", params["norm"], names["norm1"])
+        self.mixer = mk("mixer", params["mixer"], names["mixer"])
+        ff = params.get("feed_forward")
+        self.feed_forward = mk("feed_forward", ff, names["feed_forward"]) if ff else None
+        self.norm2 = mk("norm", params["norm"], names["norm2"]) if ff else None
+
+    def parts(self):
+        return [p for p in (self.mixer, self.norm1, self.feed_forward, self.norm2) if p is not None]
+
+    def streamed_weights(self):
+        return self.mixer.streamed_weights() + (self.feed_forward.streamed_weights() if self.feed_forward else [])
+
+    def activation_width(self):
+        return max(p.activation_width() for p in self.parts())
+
+    def declare(self):
+        return [d for p in self.parts() for d in p.declare()]
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        for p in self.parts():
+            p.bind(tensors, rt)
+
+    def _result(self, norm, resid, result, ctx, wanted):
+        """The normed result enters the stream; returns the new rows in the compute type if ``wanted``."""
+        if not wanted or self.rt.dtype == torch.float32:
+            norm.add_result(resid, result, ctx)
+            return resid if wanted else None
+        out = torch.empty(resid.shape, dtype=self.rt.dtype, device=resid.device)
+        norm.add_result(resid, result, ctx, out=out)
+        return out
+
+    def forward(self, resid, delta, ctx, cache):
+        apply_pending(self.rt.ops, resid, delta, ctx)  # a block of another kind before this one may have left its addition pending
+        ready = ctx.shared.pop("prepared_input", None)  # the block before may have left this block's input
+        h = ready[1] if ready is not None and ready[0] is self and delta is None else self.rt.ops.narrow(resid, self.rt.dtype)
+        ctx.shared["mixer_rows"] = resid
+        a = self.mixer.forward(h, ctx, cache)
+        ctx.shared.pop("mixer_rows", None)
+        nxt = ctx.shared.get("next_run")
+        follows = nxt is not None and isinstance(nxt[0], ResultNormBlock)
+        if self.feed_forward is None:
+            h = self._result(self.norm1, resid, a, ctx, follows)
+        else:
+            h = self._result(self.norm1, resid, a, ctx, True)
+            h = self._result(self.norm2, resid, self.feed_forward.forward(h, ctx), ctx, follows)
+        if follows:
+            ctx.shared["prepared_input"] = (nxt[0], h)
+        return None
+
+
+register_part("block", "result_norm", ResultNormBlock)

@@ -18,12 +18,12 @@ import torch
 from ..cache.spec import CacheGroup, CacheNeed
 from ..config.registry import part_class
 from ..weights.loader import TensorDecl
-from .base import LayerCache, PendingSum, Runtime, StepContext, apply_pending
+from .base import LayerCache, PendingSum, Runtime, StepContext, apply_pending, without_norms
 from .decode_stack import MAX_ROWS as STACK_MAX_ROWS, plan_stacks
 
 # the registrations of the built-in parts
-from . import (attention, block, embedding, feed_forward, filter, head, latent_attention, linear_attention, moe, norm,  # noqa: F401
-               position, selective_scan, side_by_side, ssm)
+from . import (attention, block, embedding, feed_forward, filter, head, latent_attention, linear_attention, matrix_memory, moe,  # noqa: F401
+               norm, position, selective_scan, side_by_side, ssm, token_mixing)
 
 
 @dataclass
@@ -198,6 +198,7 @@ class DecoderModel:
                 if delta.rows is not None or delta.vector is not None:
                     apply_pending(self.rt.ops, resid, delta, ctx)
                     delta = PendingSum()
+                delta = without_norms(self.rt.ops, delta, ctx)
                 delta = PendingSum(delta.terms, delta.mult, first if add.embedding else None,
                                    self.stream_tables[add.table][add.row] if add.table is not None else None, delta.factors)
             if stack is not None and isinstance(delta, PendingSum):

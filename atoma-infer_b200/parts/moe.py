@@ -13,7 +13,10 @@ that order (gate and up stacked, SiLU * up in the epilogue); a last kernel weigh
 
 Parameters: ``hidden``, ``experts``, ``top``, ``intermediate``, ``shared_intermediate`` (0: none), ``names``,
 ``router_bias`` (the logits get a learned bias, ``<prefix>.router.b``), ``weights`` (``"all"``, the default: as above;
-``"chosen"``: the softmax over the chosen experts' logits alone).
+``"chosen"``: the softmax over the chosen experts' logits alone; ``"sigmoid"``: scores s = sigmoid(z), the choice by s plus a
+learned correction per expert, ``<prefix>.correction``, the weights the chosen s as they are), ``groups`` (with
+``"sigmoid"``: ``{"count": n, "keep": m}``, the experts form n equal groups of neighbours and only those of the m groups
+whose two largest choice scores sum highest can be chosen).
 Checkpoint tensors: ``<prefix>.router`` [experts, hidden], ``<prefix>.e<j>.{gate,up,down}``,
 ``<prefix>.shared.{gate,up,down}``.
 """
@@ -33,11 +36,19 @@ class RoutedExperts(FeedForward):
         self.hidden, self.experts, self.top = int(p["hidden"]), int(p["experts"]), int(p["top"])
         self.intermediate, self.shared = int(p["intermediate"]), int(p.get("shared_intermediate") or 0)
         self.router_bias, self.over_chosen = bool(p.get("router_bias", False)), p.get("weights", "all") == "chosen"
-        if p.get("weights", "all") not in ("all", "chosen"):
-            raise ValueError(f"weights {p.get('weights')!r} is not known (known: 'all', 'chosen')")
+        self.sigmoid = p.get("weights", "all") == "sigmoid"
+        groups = p.get("groups")
+        self.groups = (int(groups["count"]), int(groups["keep"])) if groups else (1, 1)
+        if p.get("weights", "all") not in ("all", "chosen", "sigmoid"):
+            raise ValueError(f"weights {p.get('weights')!r} is not known (known: 'all', 'chosen', 'sigmoid')")
+        if groups and not self.sigmoid or self.sigmoid and self.router_bias:
+            raise ValueError("groups go with sigmoid scores, and a router bias does not")
+        if self.experts % self.groups[0] or not 0 < self.groups[1] <= self.groups[0] \
+                or self.groups[1] * (self.experts // self.groups[0]) < self.top:
+            raise ValueError(f"{self.experts} experts in {self.groups[0]} groups of which {self.groups[1]} are kept cannot give {self.top}")
         if not 0 < self.top <= self.experts:
             raise ValueError(f"top ({self.top}) must lie in 1 .. experts ({self.experts})")
-        self.names = {"router": ".router", "router_bias": ".router.b", "expert": ".e{}", "shared": ".shared", "gate": ".gate", "up": ".up", "down": ".down",
+        self.names = {"router": ".router", "router_bias": ".router.b", "correction": ".correction", "expert": ".e{}", "shared": ".shared", "gate": ".gate", "up": ".up", "down": ".down",
                       **(p.get("names") or {})}
 
     def activation_width(self):
@@ -52,6 +63,8 @@ class RoutedExperts(FeedForward):
         decls = [TensorDecl(self.prefix + self.names["router"], (self.experts, self.hidden))]
         if self.router_bias:
             decls.append(TensorDecl(self.prefix + self.names["router_bias"], (self.experts,)))
+        if self.sigmoid:
+            decls.append(TensorDecl(self.prefix + self.names["correction"], (self.experts,)))
         for j in list(range(self.experts)) + ([None] if self.shared else []):
             f = self.shared if j is None else self.intermediate
             g, u, d = self._expert(j)
@@ -63,6 +76,7 @@ class RoutedExperts(FeedForward):
         self.w_router = tensors[self.prefix + self.names["router"]].to(torch.float32).contiguous()  # widened exactly
         self.b_router = (tensors[self.prefix + self.names["router_bias"]].to(torch.float32).contiguous()
                          if self.router_bias else None)
+        self.correction = (tensors[self.prefix + self.names["correction"]].to(torch.float32).contiguous() if self.sigmoid else None)
         gu, dn = [], []
         for j in range(self.experts):
             g, u, d = self._expert(j)
@@ -82,7 +96,9 @@ class RoutedExperts(FeedForward):
         ops, T = self.rt.ops, ctx.T
         ids = torch.empty((T, self.top), dtype=torch.int32, device=x.device)
         wts = torch.empty((T, self.top), dtype=torch.float32, device=x.device)
-        if self.router_bias or self.over_chosen:
+        if self.sigmoid:
+            ops.moe_route_sigmoid(x, self.w_router, self.correction, ids, wts, ctx.meta, groups=self.groups)
+        elif self.router_bias or self.over_chosen:
             ops.moe_route(x, self.w_router, ids, wts, ctx.meta, bias=self.b_router, over_chosen=self.over_chosen)
         else:
             ops.moe_route(x, self.w_router, ids, wts, ctx.meta)

@@ -10,6 +10,7 @@ import torch
 
 import plain_bumolix as PB
 import plain_dosovik as PD
+import plain_kavotar as PV
 import plain_kulivik as PK
 import plain_tutezen as PT
 import plain_llama as P
@@ -131,7 +132,7 @@ class HostOps:
 
     def qkv_prepare(self, qkv, ctx, cache, group, q_out, *, nq, nkv, d, dv, dp, page_size, num_pages, store_kv, bias=None,
                     q_norm=None, k_norm=None, eps=0.0, inv_freq=None, rot=0, v_first=None, v_lambda=None, v_out=None,
-                    head_norm=False, interleaved=False, q_temp=None):
+                    head_norm=False, interleaved=False, q_temp=None, q_head_scale=None):
         self._count()
         meta = ctx.meta
         n = int(meta[META_NUM_TOKENS])
@@ -164,6 +165,8 @@ class HostOps:
         if q_temp:
             p = ctx.positions[:n].double()
             q = q * (1.0 + q_temp[0] * torch.log(torch.floor((p + 1) / q_temp[1]) + 1.0)).float()[:, None, None]
+        if q_head_scale is not None:
+            q = q * q_head_scale[:, None]
         if v_out is not None:
             v_out[:n] = v.to(v_out.dtype)
         if v_first is not None:
@@ -467,6 +470,111 @@ class HostOps:
         n = int(meta[META_NUM_ROWS])
         z = logits[:n] * scale
         logits[:n] = cap * torch.tanh(z / cap) if cap else z
+
+    # -- blocks whose only norm stands on a sublayer's result, and what such layers bring along
+    def linears(self, x, w, *, meta=None):
+        return tuple(self.linear(x[i], w[i], meta=meta) for i in range(x.shape[0]))
+
+    def norm_add(self, resid, pending, w, eps, ctx, *, layer_norm, out=None):
+        self._count()
+        n = int(ctx.meta[META_NUM_TOKENS])
+        y = torch.zeros_like(resid[:n])
+        for t, f, nm in zip(pending.terms, pending.weights(), pending.term_norms()):
+            a = t[:n].float()
+            y = y + f * (a if nm is None else PV.rms(a, nm[1]) * nm[0])
+        y = pending.mult * y
+        if pending.vector is not None:
+            y = y + pending.vector
+        if layer_norm:
+            y = y - y.mean(-1, keepdim=True)
+        resid[:n] += PV.rms(y, eps) * w
+        if out is not None:
+            out[:n] = resid[:n].to(out.dtype)
+
+    def layer_norm(self, resid, w, eps, out, meta, n, rows=None):
+        self._count()
+        x = resid[:int(meta[META_NUM_TOKENS])] if rows is None else resid[rows[:int(meta[META_NUM_ROWS])].long()]
+        x = x - x.mean(-1, keepdim=True)
+        out[:x.shape[0]] = (PV.rms(x, eps) * w).to(out.dtype)
+
+    def token_mix(self, x, mu, state, ctx, out):
+        self._count()
+        for _, a, b, slot in self._entries(ctx):
+            first = state[slot].clone() if int(ctx.positions[a]) > 0 else torch.zeros_like(state[slot])
+            rows = x[a:b].float()
+            before = torch.cat([first[None], rows[:-1]], 0)
+            out[:, a:b] = (rows + (before - rows) * mu[:, None]).to(out.dtype)
+        return False
+
+    def keep_last_rows(self, x, state, ctx):
+        self._count()
+        for _, a, b, slot in self._entries(ctx):
+            state[slot] = x[b - 1].float()
+
+    def tanh_rows(self, z, out, meta):
+        self._count()
+        n = int(meta[META_NUM_TOKENS])
+        out[:n] = torch.tanh(z[:n]).to(out.dtype)
+
+    def talking_attention(self, q, q_stride, cache, ctx, group, out, nq, nkv, d, page_size, num_pages, scale, talk, *, chunk=0):
+        self._count()
+        meta = ctx.meta
+        off, stride = int(meta[META_BT_OFFSET + group]), int(meta[META_BT_STRIDE + group])
+        g = nq // nkv
+        for t in range(int(meta[META_NUM_TOKENS])):
+            pos, e = int(ctx.positions[t]), int(ctx.token_entry[t])
+            idx = range(pos - pos % chunk if chunk else 0, pos + 1)
+            pages = [int(meta[off + e * stride + j // page_size]) for j in idx]
+            k = torch.stack([cache[p, 0, :, j % page_size] for p, j in zip(pages, idx)]).float()
+            v = torch.stack([cache[p, 1, :, j % page_size] for p, j in zip(pages, idx)]).float()
+            qq = q[t].view(-1, d)[:nq].float()
+            w = talk @ torch.stack([torch.softmax((k[:, h // g] @ qq[h]) * scale, 0) for h in range(nq)])
+            for h in range(nq):
+                out[t, h * d:(h + 1) * d] = (w[h] @ v[:, h // g]).to(out.dtype)
+
+    def bonus_scan(self, r, k, v, z, z_bias, bonus, state, ctx, o, *, heads, dim, vdim):
+        self._count()
+        for _, a, b, slot in self._entries(ctx):
+            for t in range(a, b):
+                rt, kt, vt = r[t].float().view(heads, dim), k[t].float().view(heads, dim), v[t].float().view(heads, vdim)
+                decay = torch.exp(-torch.exp(z[t] + z_bias)).view(heads, dim)
+                for h in range(heads):
+                    kv = torch.outer(kt[h], vt[h])
+                    o[t, h * vdim:(h + 1) * vdim] = (state[slot, h] + bonus.view(heads, dim)[h][:, None] * kv).T @ rt[h]
+                    state[slot, h] = decay[h][:, None] * state[slot, h] + kv
+
+    def memory_scan(self, q, k, v, logits, bias, cap, q_scale, state, n_state, m_state, ctx, o, nq, floor, *, heads, dim, vdim):
+        self._count()
+        x = PV.soft_limit(logits + bias, cap)
+        log_i, log_f = x[:, :heads], PV.log_sigmoid(x[:, heads:])
+        for _, a, b, slot in self._entries(ctx):
+            for t in range(a, b):
+                qt, kt, vt = q[t].float().view(heads, dim) * q_scale, k[t].float().view(heads, dim), v[t].float().view(heads, vdim)
+                for h in range(heads):
+                    m = torch.maximum(log_f[t, h] + m_state[slot, h], log_i[t, h])
+                    keep, take = torch.exp(log_f[t, h] + m_state[slot, h] - m), torch.exp(log_i[t, h] - m)
+                    state[slot, h] = keep * state[slot, h] + take * torch.outer(kt[h], vt[h])
+                    n_state[slot, h] = keep * n_state[slot, h] + take * kt[h]
+                    m_state[slot, h] = m
+                    o[t, h * vdim:(h + 1) * vdim] = state[slot, h].T @ qt[h]
+                    nq[t, h], floor[t, h] = n_state[slot, h] @ qt[h], torch.exp(-m)
+
+    def head_weight_norm_gate(self, o, gate, w, eps, out, meta, heads, *, kind, nq=None, floor=None):
+        self._count()
+        n = int(meta[META_NUM_TOKENS])
+        v = o[:n].view(n, heads, -1)
+        if nq is not None:
+            v = v / (torch.maximum(nq[:n].abs(), floor[:n]) + 1e-6)[:, :, None]
+        g = gate[:n].float()
+        g = PV.silu(g) if kind == "silu" else torch.sigmoid(g)
+        out[:n] = (PV.rms(v, eps).reshape(n, -1) * w * g).to(out.dtype)
+
+    def moe_route_sigmoid(self, h, w_router, correction, ids, wts, meta, groups=None):
+        self._count()
+        n = int(meta[META_NUM_TOKENS])
+        count, keep = groups or (1, 1)
+        idx, wt = PV.choose(torch.sigmoid(h[:n].float() @ w_router.T).double(), correction, ids.shape[1], {"count": count, "keep": keep})
+        ids[:n], wts[:n] = idx.to(torch.int32), wt.float()
 
     def sample(self, logits, temperature, top_k, top_p, seed, step, out, num_rows=None, slots=None):
         self._count()
