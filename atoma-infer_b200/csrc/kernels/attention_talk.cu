@@ -1,0 +1,628 @@
+// bfloat16 attention whose softmax weights are mixed across the query heads (talking_heads.cu says how), on the paged cache,
+// specialised by head size (-DHEAD_DIM=...).  The mix needs every head's finished softmax, so neither kernel can run heads
+// apart from one another:
+//
+//  * talk_decode: one thread-block cluster per request (steps in which every request brings one token), its blocks share
+//    the visible keys.  Every block scores its keys for all heads (mma.sync, key fragments straight from the pages), the
+//    cluster exchanges the heads' maxima and sums through distributed shared memory, every block mixes its finished
+//    weights in float32 and weighs its values, and the cluster adds the blocks' results up in order.  Each key and value
+//    byte is read once; nothing goes through scratch memory.
+//  * talk_prefill: one block per 16 tokens and request, all heads.  A first walk over the keys takes every head's maximum
+//    and sum; a second one takes the finished weights of a key tile for all heads into shared memory, mixes them on the
+//    tensor cores (a [heads x heads] times [heads x positions] product) and weighs the tile's values.
+#include <cooperative_groups.h>
+
+#include "attention_tiles.cuh"
+
+namespace cg = cooperative_groups;
+
+int g_use_pdl = 1;
+extern "C" void kernels_set_pdl(int mode) { g_use_pdl = mode; }
+extern "C" int attn_talk_head_dim() { return D; }
+
+// ----------------------------------------------------------------------------- decode
+namespace {
+constexpr int TD_THREADS = 256, TD_WARPS = TD_THREADS / 32;
+constexpr int TD_MAX_SPLITS = 8;
+constexpr int TD_HB = 4;                  // heads whose outputs a thread accumulates at a time
+constexpr int TD_LPK = D / 8;             // lanes that hold one value row (8 elements each)
+constexpr int TD_KPW = 32 / TD_LPK;       // value rows a warp reads at once
+
+// Warps that share an item (a key/value head and up to TD_HB of its query heads) of the value phase.
+__host__ __device__ inline int td_key_parts(int H, int G) {
+    const int items = G * ((H / G + TD_HB - 1) / TD_HB);
+    return items >= TD_WARPS ? 1 : TD_WARPS / items;
+}
+// Shared memory of a block for n keys: q, the mixing weights transposed, weights, mixed weights, partial outputs, (m, l) pairs.
+__host__ __device__ inline int td_row(int n) { return (n + 31) / 32 * 32 + 4; }
+inline size_t td_smem(int H, int G, int n) {
+    return (size_t)H * D * sizeof(bf16) + ((size_t)H * ((H + 7) / 8 * 8) + 2 * (size_t)H * td_row(n) + (size_t)td_key_parts(H, G) * H * D + 4 * (size_t)H) * sizeof(float);
+}
+}  // namespace
+
+__global__ void __launch_bounds__(TD_THREADS)
+talk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ cache, CacheLayout L, const int* __restrict__ meta,
+                   int group, const int* __restrict__ positions, bf16* __restrict__ out, int H, int chunk, float scale_log2,
+                   const float* __restrict__ talk, int num_pages, int splits, int max_keys, int* __restrict__ status) {
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    const int G = L.num_kv_heads, HG = H / G, HP = (H + 7) / 8 * 8, NS = td_row(max_keys), parts = td_key_parts(H, G);
+    bf16* qs = reinterpret_cast<bf16*>(smem_raw);                              // [H][D]
+    float* tt = reinterpret_cast<float*>(smem_raw + (size_t)H * D * sizeof(bf16));  // [H][HP]: talk transposed, tt[g][h]
+    float* sc = tt + (size_t)H * HP;                                           // [H][NS]: scores, then weights
+    float* pm = sc + (size_t)H * NS;                                           // [H][NS]: mixed weights
+    float* po = pm + (size_t)H * NS;                                           // [parts][H][D]
+    float* ml = po + (size_t)parts * H * D;                                    // [H][2] of this block, then [H][2] of all blocks
+    pdl_launch_dependents();
+    const int split = blockIdx.x, e = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    // (a block of a dead request leaves with its whole cluster)
+    if (e >= meta[META_NUM_ENTRIES]) return;
+    const int pos = positions[e], kstart = chunk > 0 ? pos - pos % chunk : 0, len = pos + 1 - kstart;
+    int per = ((len + splits - 1) / splits + 7) / 8 * 8;
+    if (per > max_keys) {  // (the host's bound on the keys of a block does not hold: nothing is read beyond it)
+        if (tid == 0) atomicExch(&status[STATUS_BAD_PAGE], 1 + pos);
+        per = max_keys;
+    }
+    const int lo = kstart + split * per, n = max(0, min(per, pos + 1 - lo));
+    const int* bt = meta + meta[META_BT_OFFSET + group] + (size_t)e * meta[META_BT_STRIDE + group];
+    const int ps = L.page_size, ps_shift = (ps & (ps - 1)) == 0 ? 31 - __clz(ps) : -1;
+    const size_t v_off = (size_t)G * ps * D, page_stride = 2 * v_off;
+    for (int i = tid; i < H * HP; i += TD_THREADS) {
+        const int g = i / HP, h = i % HP;
+        tt[i] = h < H ? talk[(size_t)h * H + g] : 0.f;
+    }
+    pdl_wait();
+    for (int i = tid; i < H * D / 8; i += TD_THREADS)
+        reinterpret_cast<uint4*>(qs)[i] = *reinterpret_cast<const uint4*>(q + (size_t)e * q_stride + (size_t)i * 8);
+    // the row of a key (head 0's element 0 of its page's K block), null where there is none
+    auto key_row = [&](int j) -> const bf16* {
+        if (j >= n) return nullptr;
+        const int at = lo + j, pi = ps_shift >= 0 ? at >> ps_shift : at / ps, page = __ldg(bt + pi);
+        if (page <= 0 || page >= num_pages) {
+            atomicExch(&status[STATUS_BAD_PAGE], 1 + at);
+            return nullptr;
+        }
+        return cache + (size_t)page * page_stride + (size_t)(at - pi * ps) * D;
+    };
+    __syncthreads();
+    // Scores: an item is a key/value head and 32 keys.  Both operands take the 16 dimensions of a k-step in the order
+    // (4t, 4t + 1 | 4t + 2, 4t + 3) for lane t of a quad, so a key fragment is one 8-byte load from the page.
+    const int r = lane >> 2, t4 = (lane & 3) * 4, blocks32 = (n + 31) / 32;
+    for (int item = warp; item < G * blocks32; item += TD_WARPS) {
+        const int c = item % G, k0 = (item / G) * 32;
+        uint2 kf[4][KSTEPS];
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) {
+            const bf16* row = key_row(k0 + nt * 8 + r);
+#pragma unroll
+            for (int ks = 0; ks < KSTEPS; ++ks)
+                kf[nt][ks] = row ? *reinterpret_cast<const uint2*>(row + (size_t)c * ps * D + ks * 16 + t4) : make_uint2(0u, 0u);
+        }
+        for (int m0 = 0; m0 < HG; m0 += 16) {
+            float s[4][4];
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+            const bool in0 = m0 + r < HG, in1 = m0 + r + 8 < HG;
+            const bf16* q0 = qs + (size_t)(c * HG + m0 + r) * D + t4;
+#pragma unroll
+            for (int ks = 0; ks < KSTEPS; ++ks) {
+                const uint2 x = in0 ? *reinterpret_cast<const uint2*>(q0 + ks * 16) : make_uint2(0u, 0u);
+                const uint2 y = in1 ? *reinterpret_cast<const uint2*>(q0 + 8 * D + ks * 16) : make_uint2(0u, 0u);
+                const uint32_t a[4] = {x.x, y.x, x.y, y.y};
+#pragma unroll
+                for (int nt = 0; nt < 4; ++nt) mma_bf16(s[nt], a, kf[nt][ks].x, kf[nt][ks].y);
+            }
+#pragma unroll
+            for (int nt = 0; nt < 4; ++nt) {
+                const int key = k0 + nt * 8 + (lane & 3) * 2;
+                float2 u, v;
+                u.x = key < n ? s[nt][0] * scale_log2 : -INFINITY;
+                u.y = key + 1 < n ? s[nt][1] * scale_log2 : -INFINITY;
+                v.x = key < n ? s[nt][2] * scale_log2 : -INFINITY;
+                v.y = key + 1 < n ? s[nt][3] * scale_log2 : -INFINITY;
+                if (in0) *reinterpret_cast<float2*>(sc + (size_t)(c * HG + m0 + r) * NS + key) = u;
+                if (in1) *reinterpret_cast<float2*>(sc + (size_t)(c * HG + m0 + r + 8) * NS + key) = v;
+            }
+        }
+    }
+    __syncthreads();
+    // every head's maximum and sum over this block's keys, then over the cluster's
+    for (int h = warp; h < H; h += TD_WARPS) {
+        const float* row = sc + (size_t)h * NS;
+        float mx = -INFINITY, sum = 0.f;
+        for (int j = lane; j < n; j += 32) mx = fmaxf(mx, row[j]);
+        mx = warp_max(mx);
+        for (int j = lane; j < n; j += 32) sum += fast_exp2(row[j] - mx);
+        sum = warp_sum(sum);
+        if (lane == 0) ml[2 * h] = mx, ml[2 * h + 1] = sum;
+    }
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();
+    for (int h = tid; h < H; h += TD_THREADS) {
+        float mx = -INFINITY, sum = 0.f;
+        for (int s = 0; s < splits; ++s) mx = fmaxf(mx, cluster.map_shared_rank(ml, s)[2 * h]);
+        for (int s = 0; s < splits; ++s) {
+            const float* o = cluster.map_shared_rank(ml, s);
+            if (o[2 * h] > -INFINITY) sum += o[2 * h + 1] * fast_exp2(o[2 * h] - mx);
+        }
+        ml[2 * H + 2 * h] = mx;
+        ml[2 * H + 2 * h + 1] = 1.f / sum;
+    }
+    __syncthreads();
+    for (int h = warp; h < H; h += TD_WARPS) {
+        float* row = sc + (size_t)h * NS;
+        const float mx = ml[2 * H + 2 * h], inv = ml[2 * H + 2 * h + 1];
+        for (int j = lane; j < n; j += 32) row[j] = fast_exp2(row[j] - mx) * inv;
+    }
+    __syncthreads();
+    // The mix: a warp takes 32 keys and 8 heads at a time.
+    const int hb8 = HP / 8;
+    for (int item = warp; item < hb8 * blocks32; item += TD_WARPS) {
+        const int h0 = (item % hb8) * 8, j = (item / hb8) * 32 + lane;
+        float acc[8] = {};
+        for (int g = 0; g < H; ++g) {
+            const float p = sc[(size_t)g * NS + j];
+            const float4 a = *reinterpret_cast<const float4*>(tt + (size_t)g * HP + h0), b = *reinterpret_cast<const float4*>(tt + (size_t)g * HP + h0 + 4);
+            acc[0] = fmaf(a.x, p, acc[0]); acc[1] = fmaf(a.y, p, acc[1]); acc[2] = fmaf(a.z, p, acc[2]); acc[3] = fmaf(a.w, p, acc[3]);
+            acc[4] = fmaf(b.x, p, acc[4]); acc[5] = fmaf(b.y, p, acc[5]); acc[6] = fmaf(b.z, p, acc[6]); acc[7] = fmaf(b.w, p, acc[7]);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (h0 + i < H) pm[(size_t)(h0 + i) * NS + j] = j < n ? acc[i] : 0.f;
+    }
+    __syncthreads();
+    // Values: an item is a key/value head and up to TD_HB of its query heads; `parts` warps share an item's keys.  Lane
+    // (kl, x) of a warp holds elements 8 x .. of the row of every TD_KPW-th key.
+    const int hbs = (HG + TD_HB - 1) / TD_HB, kl = lane / TD_LPK, x8 = (lane % TD_LPK) * 8, part = warp % parts;
+    for (int item = warp / parts; item < G * hbs; item += TD_WARPS / parts) {
+        const int c = item / hbs, h0 = c * HG + (item % hbs) * TD_HB, nh = min(TD_HB, (c + 1) * HG - h0);
+        float acc[TD_HB][8];
+#pragma unroll
+        for (int i = 0; i < TD_HB; ++i)
+#pragma unroll
+            for (int k = 0; k < 8; ++k) acc[i][k] = 0.f;
+        constexpr int UN = 4;  // rows in flight a lane
+        for (int j0 = part * TD_KPW; j0 < n; j0 += parts * TD_KPW * UN) {
+            uint4 v[UN];
+#pragma unroll
+            for (int u = 0; u < UN; ++u) {
+                const int j = j0 + u * parts * TD_KPW + kl;
+                v[u] = make_uint4(0u, 0u, 0u, 0u);
+                if (kl < TD_KPW) {
+                    const bf16* row = key_row(j);
+                    if (row) v[u] = *reinterpret_cast<const uint4*>(row + v_off + (size_t)c * ps * D + x8);
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < UN; ++u) {
+                const int j = j0 + u * parts * TD_KPW + kl;
+                if (kl < TD_KPW && j < n) {
+                    float f[8];
+                    const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&v[u]);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const float2 z = __bfloat1622float2(b[k]);
+                        f[2 * k] = z.x;
+                        f[2 * k + 1] = z.y;
+                    }
+#pragma unroll
+                    for (int i = 0; i < TD_HB; ++i) {
+                        if (i >= nh) continue;
+                        const float p = pm[(size_t)(h0 + i) * NS + j];
+#pragma unroll
+                        for (int k = 0; k < 8; ++k) acc[i][k] = fmaf(p, f[k], acc[i][k]);
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < TD_HB; ++i) {
+            if (i >= nh) continue;
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+                float a = acc[i][k];
+#pragma unroll
+                for (int o = 1; o < TD_KPW; ++o) a += __shfl_sync(0xffffffffu, acc[i][k], (lane + o * TD_LPK) & 31);
+                if (kl == 0) po[((size_t)part * H + h0 + i) * D + x8 + k] = a;
+            }
+        }
+    }
+    cluster.sync();
+    // the cluster's blocks share the outputs; every sum runs over the blocks in order, and over an item's warps in order
+    for (int i = split * TD_THREADS + tid; i < H * D; i += splits * TD_THREADS) {
+        float a = 0.f;
+        for (int s = 0; s < splits; ++s) {
+            const float* o = cluster.map_shared_rank(po, s);
+            for (int p = 0; p < parts; ++p) a += o[(size_t)p * H * D + i];
+        }
+        out[(size_t)e * H * D + i] = __float2bfloat16_rn(a);
+    }
+    cluster.sync();  // nobody leaves while its shared memory may still be read
+}
+
+// The fewest blocks a request's keys (at most max_keys of them) can be shared by, at most TD_MAX_SPLITS; 0: they do not fit.
+extern "C" int attn_talk_decode_min_splits(int nq, int nkv, int max_keys) {
+    if (nkv <= 0 || nq % nkv) return 0;
+    for (int s = 1; s <= TD_MAX_SPLITS; ++s)
+        if (td_smem(nq, nkv, ((max_keys + s - 1) / s + 7) / 8 * 8) <= 200 * 1024) return s;
+    return 0;
+}
+
+extern "C" int attn_talk_decode(const void* q, int q_stride, const void* cache, const int* meta, int group, const int* positions, void* out,
+                                int S, int nq, int nkv, int page_size, int num_pages, int chunk, float scale, const float* talk, int splits,
+                                int max_context, int* status, cudaStream_t stream) {
+    if (S <= 0) return 0;
+    if (nkv <= 0 || nq % nkv || splits < 1 || splits > TD_MAX_SPLITS || q_stride % 8 || ((uintptr_t)q & 15)) return (int)cudaErrorInvalidValue;
+    const int seen = chunk > 0 && chunk < max_context ? chunk : max_context;
+    const int max_keys = ((seen + splits - 1) / splits + 7) / 8 * 8;
+    const size_t smem = td_smem(nq, nkv, max_keys);
+    if (smem > 220 * 1024) return (int)cudaErrorInvalidValue;
+    static size_t configured = 0;  // grows only, and is not set again inside a stream capture once large enough
+    if (smem > 48 * 1024 && smem > configured) {
+        cudaError_t err = cudaFuncSetAttribute(talk_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (err != cudaSuccess) return (int)err;
+        configured = smem;
+    }
+    const CacheLayout L{nkv, page_size, D};
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(splits, S);
+    cfg.blockDim = dim3(TD_THREADS);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = splits;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = (g_use_pdl & 1) ? 2 : 1;
+    return (int)cudaLaunchKernelEx(&cfg, talk_decode_kernel, (const bf16*)q, q_stride, (const bf16*)cache, L, meta, group, positions,
+                                   (bf16*)out, nq, chunk, scale * LOG2E, talk, num_pages, splits, max_keys, status);
+}
+
+// ----------------------------------------------------------------------------- prefill (and mixed steps)
+namespace {
+constexpr int TP_WARPS = 8, TP_THREADS = TP_WARPS * 32;
+constexpr int TP_TOK = 16;  // tokens of a block
+
+// Heads whose outputs a warp keeps in registers, for H heads (more heads than 8 times this: blocks share them).
+inline int tp_heads_per_warp(int H) {
+    const int most = D <= 64 ? 4 : (D <= 128 ? 2 : 1);
+    int n = 1;
+    while (n < most && n * TP_WARPS < H) n *= 2;
+    return n;
+}
+inline int pad16(int n) { return (n + 15) / 16 * 16; }
+inline size_t tp_smem(int H, int G, int KT, int stages, int bt_cap) {
+    return ((size_t)H * TP_TOK * LDS + (size_t)(stages + 1) * G * KT * LDS + (size_t)pad16(H) * TP_TOK * KT + (size_t)pad16(H) * (pad16(H) + 8)) * sizeof(bf16) +
+           (size_t)2 * H * TP_TOK * sizeof(float) + (size_t)bt_cap * sizeof(int);
+}
+}  // namespace
+
+// Shared memory of the weights: head g's 16 x KT tile as 16-byte pieces of 8 keys, piece n * 16 + row at place (n * 16 + row) ^
+// (g & 7), so that the pieces of 8 neighbouring rows, and those of one row of 8 neighbouring heads, lie in different banks.
+template <int KT>
+__device__ __forceinline__ bf16* tp_piece(bf16* p, int g, int piece) { return p + (size_t)g * TP_TOK * KT + (size_t)((piece ^ (g & 7)) * 8); }
+
+template <int KT, int HPW>
+__global__ void __launch_bounds__(TP_THREADS)
+talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ cache, CacheLayout L, const int* __restrict__ meta,
+                    int group, const int* __restrict__ cu_tokens, const int* __restrict__ ctx_lens, bf16* __restrict__ out, int H,
+                    int chunk, float scale_log2, const float* __restrict__ talk, int num_pages, int bt_cap, int stages,
+                    int* __restrict__ status) {
+    constexpr int NK = KT / 8, MT = TP_WARPS * HPW > 16 ? TP_WARPS * HPW / 16 : 1;
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    const int G = L.num_kv_heads, HG = H / G, HP = (H + 15) / 16 * 16, TS = HP + 8, ps = L.page_size;
+    bf16* qt = reinterpret_cast<bf16*>(smem_raw);             // [H][16][LDS]
+    bf16* kt = qt + (size_t)H * TP_TOK * LDS;                 // [stages][G][KT][LDS]
+    bf16* vt = kt + (size_t)stages * G * KT * LDS;            // [G][KT][LDS]
+    bf16* pt = vt + (size_t)G * KT * LDS;                     // [HP][16 * KT], see tp_piece
+    bf16* tk = pt + (size_t)HP * TP_TOK * KT;                 // [HP][TS]: talk
+    float* ms = reinterpret_cast<float*>(tk + (size_t)HP * TS);  // [H][16]: a row's maximum
+    float* ls = ms + (size_t)H * TP_TOK;                      // [H][16]: its sum, then one over it
+    int* bt_s = reinterpret_cast<int*>(ls + (size_t)H * TP_TOK);
+    pdl_launch_dependents();
+    pdl_wait();
+    // late query tiles see the most keys: they go first
+    const int tile = gridDim.x - 1 - blockIdx.x, hpart = blockIdx.y, e = blockIdx.z;
+    if (e >= meta[META_NUM_ENTRIES]) return;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int row0 = cu_tokens[e], q_len = cu_tokens[e + 1] - row0, t0 = tile * TP_TOK;
+    if (t0 >= q_len) return;
+    const int nt = min(TP_TOK, q_len - t0), p_first = ctx_lens[e] + t0, p_last = p_first + nt - 1;
+    const int* bt = meta + meta[META_BT_OFFSET + group] + (size_t)e * meta[META_BT_STRIDE + group];
+    const int kbeg = chunk > 0 ? p_first - p_first % chunk : 0, kend = p_last + 1;
+    const int page_lo = kbeg / ps;
+    int page_cnt = (kend - 1) / ps - page_lo + 1;
+    if (page_cnt > bt_cap) {
+        if (tid == 0) atomicExch(&status[STATUS_BAD_PAGE], 1 + kend);
+        page_cnt = bt_cap;
+    }
+    stage_block_table(bt_s, bt, page_lo, page_cnt, num_pages, tid, TP_THREADS, status);
+    const int kend_s = min(kend, (page_lo + page_cnt) * ps), ntiles = (kend - kbeg + KT - 1) / KT;
+    const int ps_shift = (ps & (ps - 1)) == 0 ? 31 - __clz(ps) : -1;
+    const size_t v_off = (size_t)G * ps * D, page_stride = 2 * v_off;
+    for (int idx = tid; idx < H * TP_TOK * (D / 8); idx += TP_THREADS) {
+        const int c = idx % (D / 8), h = (idx / (D / 8)) % H, tok = idx / (D / 8) / H;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (tok < nt) v = *reinterpret_cast<const uint4*>(q + (size_t)(row0 + t0 + tok) * q_stride + (size_t)h * D + c * 8);
+        *reinterpret_cast<uint4*>(qt + (size_t)h * TP_TOK * LDS + toff(tok, c * 8)) = v;
+    }
+    for (int idx = tid; idx < HP * HP; idx += TP_THREADS) {
+        const int h = idx / HP, g = idx % HP;
+        tk[h * TS + g] = __float2bfloat16_rn(h < H && g < H ? talk[(size_t)h * H + g] : 0.f);
+    }
+    for (int idx = tid; idx < (HP - H) * TP_TOK * KT; idx += TP_THREADS) pt[(size_t)H * TP_TOK * KT + idx] = __float2bfloat16_rn(0.f);
+    for (int i = tid; i < H * TP_TOK; i += TP_THREADS) ms[i] = -INFINITY, ls[i] = 0.f;
+    // keys (kv = 0) or values (kv = 1) of a tile for every head; positions outside [kbeg, kend_s) as zeros
+    auto load_tile = [&](bf16* dst, int t, int kv) {
+        constexpr int PAIRS = D / 16;
+        for (int idx = tid; idx < G * KT * PAIRS; idx += TP_THREADS) {
+            const int c16 = (idx % PAIRS) * 16, rr = (idx / PAIRS) % KT, c = idx / PAIRS / KT, at = kbeg + t * KT + rr;
+            bf16* base = dst + (size_t)c * KT * LDS;
+            bf16 *d0 = base + toff(rr, c16), *d1 = base + toff(rr, c16 + 8);
+            int page = -1, slot = 0;
+            if (at < kend_s) {
+                const int pi = ps_shift >= 0 ? at >> ps_shift : at / ps;
+                slot = at - pi * ps;
+                page = bt_s[pi - page_lo];
+            }
+            if (page > 0) {
+                const bf16* src = cache + (size_t)page * page_stride + (kv ? v_off : 0) + (size_t)(c * ps + slot) * D + c16;
+                cp_async_16(d0, src);
+                cp_async_16(d1, src + 8);
+            } else {
+                const uint4 z = make_uint4(0u, 0u, 0u, 0u);
+                *reinterpret_cast<uint4*>(d0) = z;
+                *reinterpret_cast<uint4*>(d1) = z;
+            }
+        }
+    };
+    auto k_stage = [&](int t) { return kt + (size_t)(stages == 2 ? t & 1 : 0) * G * KT * LDS; };
+    const int g4 = lane >> 2, pa = g4 < nt ? p_first + g4 : -1, pb = g4 + 8 < nt ? p_first + g4 + 8 : -1;
+    const int ca = chunk > 0 && pa >= 0 ? pa - pa % chunk : 0, cb = chunk > 0 && pb >= 0 ? pb - pb % chunk : 0;
+    const int c_last = chunk > 0 ? p_last - p_last % chunk : 0;
+    // the scores of a head's 16 tokens against a tile, in base 2, masked
+    auto score = [&](int h, int t, float (&s)[NK][4]) {
+        uint32_t qf[Q_IN_REGS ? KSTEPS : 1][4];
+        const bf16* qh = qt + (size_t)h * TP_TOK * LDS;
+        if (Q_IN_REGS) {
+#pragma unroll
+            for (int ks = 0; ks < KSTEPS; ++ks) load_a_frag(qf[ks], qh, ks, lane);
+        }
+        qk_tile<NK>(s, qf, qh, k_stage(t) + (size_t)(h / HG) * KT * LDS, lane);
+        const int k0 = kbeg + t * KT;
+        if (nt == TP_TOK && k0 + KT - 1 <= p_first && k0 >= c_last) {  // a tile that every token sees whole
+#pragma unroll
+            for (int n = 0; n < NK; ++n)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) s[n][c] *= scale_log2;
+            return;
+        }
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int key = k0 + n * 8 + (lane & 3) * 2 + (c & 1);
+                s[n][c] = (c < 2 ? key <= pa && key >= ca : key <= pb && key >= cb) ? s[n][c] * scale_log2 : -INFINITY;
+            }
+    };
+    __syncthreads();  // the table slice is written
+    // ---- first walk: every row's maximum and sum, for every head
+    load_tile(k_stage(0), 0, 0);
+    cp_async_commit();
+    for (int t = 0; t < ntiles; ++t) {
+        if (stages == 2 && t + 1 < ntiles) {
+            load_tile(k_stage(t + 1), t + 1, 0);
+            cp_async_commit();
+            cp_async_wait<1>();
+        } else {
+            cp_async_wait<0>();
+        }
+        __syncthreads();
+        for (int h = warp; h < H; h += TP_WARPS) {
+            float s[NK][4];
+            score(h, t, s);
+#pragma unroll
+            for (int b = 0; b < 2; ++b) {
+                float mx = -INFINITY, sum = 0.f;
+#pragma unroll
+                for (int n = 0; n < NK; ++n) mx = fmaxf(mx, fmaxf(s[n][2 * b], s[n][2 * b + 1]));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+                const int at = h * TP_TOK + g4 + 8 * b;
+                const float old = ms[at], m_new = fmaxf(old, mx), base = m_new == -INFINITY ? 0.f : m_new;
+#pragma unroll
+                for (int n = 0; n < NK; ++n) sum += fast_exp2(s[n][2 * b] - base) + fast_exp2(s[n][2 * b + 1] - base);
+                sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+                sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+                __syncwarp();  // every lane of the quad has read the old maximum
+                if ((lane & 3) == 0) {
+                    ls[at] = ls[at] * fast_exp2(old - base) + sum;
+                    ms[at] = m_new;
+                }
+                __syncwarp();
+            }
+        }
+        __syncthreads();  // the stage may be overwritten
+        if (stages == 1 && t + 1 < ntiles) {
+            load_tile(k_stage(t + 1), t + 1, 0);
+            cp_async_commit();
+        }
+    }
+    for (int i = tid; i < H * TP_TOK; i += TP_THREADS) {
+        ls[i] = ls[i] > 0.f ? 1.f / ls[i] : 0.f;
+        if (ms[i] == -INFINITY) ms[i] = 0.f;  // (a padding row: every weight becomes zero)
+    }
+    // ---- second walk: weights, mix, values
+    const int h_lo = hpart * TP_WARPS * HPW, h_hi = min(H, h_lo + TP_WARPS * HPW);  // the heads whose outputs this block makes
+    float o[HPW][DTILES][4];
+#pragma unroll
+    for (int i = 0; i < HPW; ++i)
+#pragma unroll
+        for (int dt = 0; dt < DTILES; ++dt) o[i][dt][0] = o[i][dt][1] = o[i][dt][2] = o[i][dt][3] = 0.f;
+    load_tile(k_stage(0), 0, 0);
+    cp_async_commit();
+    for (int t = 0; t < ntiles; ++t) {
+        cp_async_wait<0>();
+        __syncthreads();  // keys of the tile are there; values and weights of the tile before are no longer read
+        load_tile(vt, t, 1);
+        cp_async_commit();
+        const bool ahead = stages == 2 && t + 1 < ntiles;
+        if (ahead) {
+            load_tile(k_stage(t + 1), t + 1, 0);
+            cp_async_commit();
+        }
+        for (int h = warp; h < H; h += TP_WARPS) {
+            float s[NK][4];
+            score(h, t, s);
+            const float m0 = ms[h * TP_TOK + g4], m1 = ms[h * TP_TOK + g4 + 8], l0 = ls[h * TP_TOK + g4], l1 = ls[h * TP_TOK + g4 + 8];
+#pragma unroll
+            for (int n = 0; n < NK; ++n) {
+                *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, h, n * 16 + g4) + (lane & 3) * 2) =
+                    pack_bf16(fast_exp2(s[n][0] - m0) * l0, fast_exp2(s[n][1] - m0) * l0);
+                *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, h, n * 16 + g4 + 8) + (lane & 3) * 2) =
+                    pack_bf16(fast_exp2(s[n][2] - m1) * l1, fast_exp2(s[n][3] - m1) * l1);
+            }
+        }
+        __syncthreads();
+        // The mix, in place: a warp owns two pieces (16 positions) at a time of all heads, reads them and writes the heads of
+        // its block's one or two tiles of 16 (a padding head's row and column of the mixing weights are zero).
+        for (int pc = warp * 2; pc < TP_TOK * NK; pc += TP_WARPS * 2) {
+            const int m0 = h_lo / 16 * 16;
+            float acc[MT][2][4];
+#pragma unroll
+            for (int i = 0; i < MT; ++i)
+#pragma unroll
+                for (int b = 0; b < 2; ++b) acc[i][b][0] = acc[i][b][1] = acc[i][b][2] = acc[i][b][3] = 0.f;
+            for (int g0 = 0; g0 < HP; g0 += 16) {
+                uint32_t b[4];
+                const int j = lane >> 3, g = g0 + (lane & 7) + (j & 1) * 8;
+                ldmatrix_x4_trans(b, tp_piece<KT>(pt, g, pc + (j >> 1)));
+#pragma unroll
+                for (int i = 0; i < MT; ++i) {
+                    if (m0 + i * 16 >= h_hi) continue;
+                    uint32_t a[4];
+                    ldmatrix_x4(a, tk + (size_t)(m0 + i * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * TS + g0 + (lane >> 4) * 8);
+                    mma_bf16(acc[i][0], a, b[0], b[1]);
+                    mma_bf16(acc[i][1], a, b[2], b[3]);
+                }
+            }
+            __syncwarp();  // the warp has read its pieces
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+                if (m0 + i * 16 >= h_hi) continue;
+#pragma unroll
+                for (int b = 0; b < 2; ++b) {
+                    *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, m0 + i * 16 + g4, pc + b) + (lane & 3) * 2) = pack_bf16(acc[i][b][0], acc[i][b][1]);
+                    *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, m0 + i * 16 + g4 + 8, pc + b) + (lane & 3) * 2) = pack_bf16(acc[i][b][2], acc[i][b][3]);
+                }
+            }
+        }
+        if (ahead) cp_async_wait<1>();
+        else cp_async_wait<0>();
+        __syncthreads();  // mixed weights and values are there
+        if (stages == 1 && t + 1 < ntiles) {  // (one stage of keys: the next ones come while the values are weighed)
+            load_tile(k_stage(t + 1), t + 1, 0);
+            cp_async_commit();
+        }
+#pragma unroll
+        for (int i = 0; i < HPW; ++i) {
+            const int h = h_lo + warp + i * TP_WARPS;
+            if (h < h_hi) {
+                const bf16* v = vt + (size_t)(h / HG) * KT * LDS;
+#pragma unroll
+                for (int ks = 0; ks < NK / 2; ++ks) {
+                    uint32_t a[4];
+                    const int j = lane >> 3;
+                    ldmatrix_x4(a, tp_piece<KT>(pt, h, (2 * ks + (j >> 1)) * 16 + (lane & 7) + (j & 1) * 8));
+#pragma unroll
+                    for (int dp = 0; dp < DTILES / 2; ++dp) {
+                        uint32_t b[4];
+                        ldmatrix_x4_trans(b, v + toff(ks * 16 + (lane & 7) + (j & 1) * 8, dp * 16 + (j >> 1) * 8));
+                        mma_bf16(o[i][2 * dp], a, b[0], b[1]);
+                        mma_bf16(o[i][2 * dp + 1], a, b[2], b[3]);
+                    }
+                }
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < HPW; ++i) {
+        const int h = h_lo + warp + i * TP_WARPS;
+        if (h >= h_hi) continue;
+#pragma unroll
+        for (int b = 0; b < 2; ++b) {
+            const int tok = g4 + 8 * b;
+            if (tok >= nt) continue;
+            bf16* orow = out + ((size_t)(row0 + t0 + tok) * H + h) * D;
+#pragma unroll
+            for (int dt = 0; dt < DTILES; ++dt)
+                *reinterpret_cast<__nv_bfloat162*>(orow + dt * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(o[i][dt][2 * b], o[i][dt][2 * b + 1]);
+        }
+    }
+}
+
+namespace {
+// Keys of a tile and stages of keys that fit in shared memory: the largest tile first.
+bool tp_geometry(int H, int G, int bt_cap, int* KT, int* stages, size_t* smem) {
+    static const int choices[][2] = {{32, 2}, {32, 1}, {16, 2}, {16, 1}};
+    for (auto& c : choices) {
+        *smem = tp_smem(H, G, c[0], c[1], bt_cap);
+        if (*smem <= 227 * 1024) {
+            *KT = c[0];
+            *stages = c[1];
+            return true;
+        }
+    }
+    return false;
+}
+int tp_table_slice(int chunk, int max_context, int page_size) {
+    const int span = chunk > 0 ? (max_context < chunk + TP_TOK ? max_context : chunk + TP_TOK) : max_context;
+    return span / page_size + 2;
+}
+}  // namespace
+
+extern "C" int attn_talk_prefill_supports(int nq, int nkv, int chunk, int max_context, int page_size) {
+    int KT, stages;
+    size_t smem;
+    return nkv > 0 && nq % nkv == 0 && tp_geometry(nq, nkv, tp_table_slice(chunk, max_context, page_size), &KT, &stages, &smem);
+}
+
+extern "C" int attn_talk_prefill(const void* q, int q_stride, const void* cache, const int* meta, int group, const int* cu_tokens,
+                                 const int* ctx_lens, void* out, int S, int max_q_len, int nq, int nkv, int page_size, int num_pages,
+                                 int chunk, float scale, const float* talk, int max_context, int* status, cudaStream_t stream) {
+    if (S <= 0 || max_q_len <= 0) return 0;
+    if (nkv <= 0 || nq % nkv || q_stride % 8 || ((uintptr_t)q & 15)) return (int)cudaErrorInvalidValue;
+    const int bt_cap = tp_table_slice(chunk, max_context, page_size);
+    int KT = 0, stages = 0;
+    size_t smem = 0;
+    if (!tp_geometry(nq, nkv, bt_cap, &KT, &stages, &smem)) return (int)cudaErrorInvalidValue;
+    const int hpw = tp_heads_per_warp(nq), parts = (nq + TP_WARPS * hpw - 1) / (TP_WARPS * hpw);
+    const dim3 grid((max_q_len + TP_TOK - 1) / TP_TOK, parts, S);
+    const CacheLayout L{nkv, page_size, D};
+#define TALK_PREFILL_CASE(KT_, HPW_)                                                                                       \
+    do {                                                                                                                  \
+        static size_t configured = 0;                                                                                     \
+        if (smem > 48 * 1024 && smem > configured) {                                                                      \
+            cudaError_t err = cudaFuncSetAttribute(talk_prefill_kernel<KT_, HPW_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (err != cudaSuccess) return (int)err;                                                                      \
+            configured = smem;                                                                                            \
+        }                                                                                                                 \
+        return (int)launch_kernel(talk_prefill_kernel<KT_, HPW_>, grid, TP_THREADS, smem, stream, (const bf16*)q, q_stride, (const bf16*)cache, \
+                                  L, meta, group, cu_tokens, ctx_lens, (bf16*)out, nq, chunk, scale * LOG2E, talk, num_pages, bt_cap, stages, \
+                                  status);                                                                                \
+    } while (0)
+#define TALK_PREFILL_TILE(HPW_)                    \
+    do {                                           \
+        if (KT == 32) TALK_PREFILL_CASE(32, HPW_); \
+        TALK_PREFILL_CASE(16, HPW_);               \
+    } while (0)
+    if (hpw == 1) TALK_PREFILL_TILE(1);
+    if constexpr (D <= 128) if (hpw == 2) TALK_PREFILL_TILE(2);
+    if constexpr (D <= 64) if (hpw == 4) TALK_PREFILL_TILE(4);
+    return (int)cudaErrorInvalidValue;
+#undef TALK_PREFILL_TILE
+#undef TALK_PREFILL_CASE
+}

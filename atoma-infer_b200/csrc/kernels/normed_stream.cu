@@ -35,32 +35,52 @@ struct NormedTerms {
     int n;
 };
 
-#define NS_CHUNKS 4  // fours of values a thread keeps in registers
-template <typename TD, typename TO>
+#define NS_CHUNKS 4  // most fours of values a thread keeps in registers
+// Four stored values as they were loaded (a bfloat16 row costs half the registers of a float32 one until it is used).
+template <typename T> struct RawFour;
+template <> struct RawFour<float> { float4 v; };
+template <> struct RawFour<__nv_bfloat16> { uint2 v; };
+template <typename T> __device__ __forceinline__ RawFour<T> raw_four(const T* p) { return *reinterpret_cast<const RawFour<T>*>(p); }
+template <typename T> __device__ __forceinline__ void widen_four(const RawFour<T>& r, float (&v)[4]) { load4(reinterpret_cast<const T*>(&r), v); }
+
+// The row form: CH fours a thread, every load of the row on its way before the first is used; NT terms (0: `terms.n`, at most
+// four).  The mean of y follows from the first pass's sums (of every normed term the sum of squares and the weighted sum, of
+// every other term the sum), so there are two block-wide reductions.
+template <typename TD, typename TO, int NT, int CH>
 __global__ void __launch_bounds__(1024)
 norm_add_kernel(float* __restrict__ resid, const NormedTerms terms, float mult, const float* __restrict__ vec,
-                const float* __restrict__ w, float eps, int layer_norm, TO* __restrict__ out, const int* __restrict__ meta, int H,
-                int vec4) {
-    __shared__ float red[2][NS_MAX_SUMS * 33];
-    extern __shared__ __align__(16) float row[];  // the scalar form's row
-    const int t = blockIdx.x;
+                const float* __restrict__ w, float eps, int layer_norm, TO* __restrict__ out, const int* __restrict__ meta, int H) {
+    constexpr int MAXT = NT ? NT : NS_MAX_TERMS;
+    __shared__ float red[3][NS_MAX_SUMS * 33];
+    const int t = blockIdx.x, n = NT ? NT : terms.n;
     const bool live = t < meta[META_NUM_TOKENS];
     pdl_wait();
     pdl_launch_dependents();
     if (!live) return;
     const float inv_h = 1.f / (float)H;
     float* x = resid + (size_t)t * H;
-    TO* o = out ? out + (size_t)t * H : nullptr;
-    // First pass: of every normed term the sum of squares and the weighted sum, of every other term the sum.  The mean of y
-    // follows from them without another pass.
-    float sums[2 * NS_MAX_TERMS] = {};
-    if (vec4) {
-        for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+    RawFour<TD> raw[MAXT][CH];
+    float4 old[CH];
 #pragma unroll
-            for (int j = 0; j < NS_MAX_TERMS; ++j) {
-                if (j >= terms.n) continue;
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * 4;
+        if (i < H) {
+#pragma unroll
+            for (int j = 0; j < MAXT; ++j)
+                if (j < n) raw[j][c] = raw_four((const TD*)terms.p[j] + (size_t)t * H + i);
+            old[c] = *reinterpret_cast<const float4*>(x + i);
+        }
+    }
+    float sums[2 * MAXT] = {};
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * 4;
+        if (i < H) {
+#pragma unroll
+            for (int j = 0; j < MAXT; ++j) {
+                if (j >= n) continue;
                 float a[4], wv[4] = {1.f, 1.f, 1.f, 1.f};
-                load4((const TD*)terms.p[j] + (size_t)t * H + i, a);
+                widen_four(raw[j][c], a);
                 if (terms.w[j]) load4(terms.w[j] + i, wv);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
@@ -69,16 +89,88 @@ norm_add_kernel(float* __restrict__ resid, const NormedTerms terms, float mult, 
                 }
             }
         }
-    } else {
-        for (int i = threadIdx.x; i < H; i += blockDim.x)
-#pragma unroll
-            for (int j = 0; j < NS_MAX_TERMS; ++j) {
-                if (j >= terms.n) continue;
-                const float a = to_float(((const TD*)terms.p[j])[(size_t)t * H + i]), wv = terms.w[j] ? terms.w[j][i] : 1.f;
-                sums[2 * j] = fmaf(a, a, sums[2 * j]);
-                sums[2 * j + 1] = fmaf(a, wv, sums[2 * j + 1]);
-            }
     }
+    block_totals(sums, 2 * n, red[0]);
+    float fac[MAXT], mean = 0.f;
+#pragma unroll
+    for (int j = 0; j < MAXT; ++j) {
+        fac[j] = j < n ? mult * terms.f[j] * (terms.w[j] ? rsqrtf(sums[2 * j] * inv_h + terms.eps[j]) : 1.f) : 0.f;
+        mean = fmaf(fac[j], sums[2 * j + 1] * inv_h, mean);
+    }
+    if (vec) {  // (a bias of the result: its mean joins the terms')
+        float s[1] = {0.f};
+        for (int i = threadIdx.x; i < H; i += blockDim.x) s[0] += vec[i];
+        block_totals(s, 1, red[2]);
+        mean += s[0] * inv_h;
+    }
+    if (!layer_norm) mean = 0.f;
+    float ss[1] = {0.f}, y[CH][4];
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * 4;
+        if (i < H) {
+            float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int j = 0; j < MAXT; ++j) {
+                if (j >= n) continue;
+                float a[4], wv[4] = {1.f, 1.f, 1.f, 1.f};
+                widen_four(raw[j][c], a);
+                if (terms.w[j]) load4(terms.w[j] + i, wv);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) s[k] = fmaf(fac[j] * wv[k], a[k], s[k]);
+            }
+            if (vec) {
+                float b[4];
+                load4(vec + i, b);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) s[k] += b[k];
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                y[c][k] = s[k] - mean;
+                ss[0] = fmaf(y[c][k], y[c][k], ss[0]);
+            }
+        }
+    }
+    block_totals(ss, 1, red[1]);
+    const float inv = rsqrtf(ss[0] * inv_h + eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+        const int i = (c * blockDim.x + threadIdx.x) * 4;
+        if (i < H) {
+            float wv[4], v[4] = {old[c].x, old[c].y, old[c].z, old[c].w};
+            load4(w + i, wv);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = fmaf(y[c][k] * inv, wv[k], v[k]);
+            store4(x + i, v);
+            if (out) store4(out + (size_t)t * H + i, v);
+        }
+    }
+}
+
+// The same for rows of any width and alignment, value by value; y waits in shared memory.
+template <typename TD, typename TO>
+__global__ void __launch_bounds__(256)
+norm_add_scalar_kernel(float* __restrict__ resid, const NormedTerms terms, float mult, const float* __restrict__ vec,
+                       const float* __restrict__ w, float eps, int layer_norm, TO* __restrict__ out, const int* __restrict__ meta, int H) {
+    __shared__ float red[3][NS_MAX_SUMS * 33];
+    extern __shared__ __align__(16) float row[];
+    const int t = blockIdx.x;
+    const bool live = t < meta[META_NUM_TOKENS];
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!live) return;
+    const float inv_h = 1.f / (float)H;
+    float* x = resid + (size_t)t * H;
+    float sums[2 * NS_MAX_TERMS] = {};
+    for (int i = threadIdx.x; i < H; i += blockDim.x)
+#pragma unroll
+        for (int j = 0; j < NS_MAX_TERMS; ++j) {
+            if (j >= terms.n) continue;
+            const float a = to_float(((const TD*)terms.p[j])[(size_t)t * H + i]), wv = terms.w[j] ? terms.w[j][i] : 1.f;
+            sums[2 * j] = fmaf(a, a, sums[2 * j]);
+            sums[2 * j + 1] = fmaf(a, wv, sums[2 * j + 1]);
+        }
     block_totals(sums, 2 * terms.n, red[0]);
     float fac[NS_MAX_TERMS], mean = 0.f;
 #pragma unroll
@@ -86,89 +178,33 @@ norm_add_kernel(float* __restrict__ resid, const NormedTerms terms, float mult, 
         fac[j] = j < terms.n ? mult * terms.f[j] * (terms.w[j] ? rsqrtf(sums[2 * j] * inv_h + terms.eps[j]) : 1.f) : 0.f;
         mean = fmaf(fac[j], sums[2 * j + 1] * inv_h, mean);
     }
-    if (vec) {  // (a bias of the result: its mean joins the terms')
+    if (vec) {
         float s[1] = {0.f};
         for (int i = threadIdx.x; i < H; i += blockDim.x) s[0] += vec[i];
-        block_totals(s, 1, red[1]);
+        block_totals(s, 1, red[2]);
         mean += s[0] * inv_h;
-        __syncthreads();
     }
     if (!layer_norm) mean = 0.f;
-    // Second pass: y less its mean, and its mean square.
     float ss[1] = {0.f};
-    float y[NS_CHUNKS][4];
-    if (vec4) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        float s = 0.f;
 #pragma unroll
-        for (int c = 0; c < NS_CHUNKS; ++c) {
-            const int i = (c * blockDim.x + threadIdx.x) * 4;
-            if (i < H) {
-                float s[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-                for (int j = 0; j < NS_MAX_TERMS; ++j) {
-                    if (j >= terms.n) continue;
-                    float a[4], wv[4] = {1.f, 1.f, 1.f, 1.f};
-                    load4((const TD*)terms.p[j] + (size_t)t * H + i, a);
-                    if (terms.w[j]) load4(terms.w[j] + i, wv);
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) s[k] = fmaf(fac[j] * wv[k], a[k], s[k]);
-                }
-                if (vec) {
-                    float b[4];
-                    load4(vec + i, b);
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) s[k] += b[k];
-                }
-#pragma unroll
-                for (int k = 0; k < 4; ++k) {
-                    y[c][k] = s[k] - mean;
-                    ss[0] = fmaf(y[c][k], y[c][k], ss[0]);
-                }
-            }
+        for (int j = 0; j < NS_MAX_TERMS; ++j) {
+            if (j >= terms.n) continue;
+            s = fmaf(fac[j] * (terms.w[j] ? terms.w[j][i] : 1.f), to_float(((const TD*)terms.p[j])[(size_t)t * H + i]), s);
         }
-    } else {
-        for (int i = threadIdx.x; i < H; i += blockDim.x) {
-            float s = 0.f;
-#pragma unroll
-            for (int j = 0; j < NS_MAX_TERMS; ++j) {
-                if (j >= terms.n) continue;
-                s = fmaf(fac[j] * (terms.w[j] ? terms.w[j][i] : 1.f), to_float(((const TD*)terms.p[j])[(size_t)t * H + i]), s);
-            }
-            if (vec) s += vec[i];
-            s -= mean;
-            row[i] = s;
-            ss[0] = fmaf(s, s, ss[0]);
-        }
+        if (vec) s += vec[i];
+        s -= mean;
+        row[i] = s;
+        ss[0] = fmaf(s, s, ss[0]);
     }
     block_totals(ss, 1, red[1]);
     const float inv = rsqrtf(ss[0] * inv_h + eps);
-    if (vec4) {
-#pragma unroll
-        for (int c = 0; c < NS_CHUNKS; ++c) {
-            const int i = (c * blockDim.x + threadIdx.x) * 4;
-            if (i < H) {
-                float v[4], wv[4];
-                load4(x + i, v);
-                load4(w + i, wv);
-#pragma unroll
-                for (int k = 0; k < 4; ++k) v[k] = fmaf(y[c][k] * inv, wv[k], v[k]);
-                store4(x + i, v);
-                if (o) store4(o + i, v);
-            }
-        }
-        return;
-    }
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         const float v = fmaf(row[i] * inv, w[i], x[i]);
         x[i] = v;
-        if (o) o[i] = from_float<TO>(v);
+        if (out) out[(size_t)t * H + i] = from_float<TO>(v);
     }
-}
-
-// Threads of a block for rows of H values: fours in registers, at most NS_CHUNKS of them a thread (0: too wide for that).
-static int row_threads(int H) {
-    int threads = H <= 512 ? 128 : 256;
-    while (threads < 1024 && H > threads * 4 * NS_CHUNKS) threads *= 2;
-    return H <= threads * 4 * NS_CHUNKS ? threads : 0;
 }
 
 extern "C" int norm_add(float* resid, int num_terms, const void* const* term_ptrs, const float* factors, const float* const* term_weights,
@@ -186,27 +222,43 @@ extern "C" int norm_add(float* resid, int num_terms, const void* const* term_ptr
         terms.eps[j] = term_eps[j];
         all |= (uintptr_t)term_ptrs[j] | (uintptr_t)term_weights[j];
     }
-    int threads = row_threads(H);
-    const int vec4 = threads && H % 4 == 0 && (all & 15) == 0;
-    if (!vec4) threads = 256;
+    // rows of fours in registers: one, two or four of them a thread
+    const int fours = (H + 3) / 4, ch = fours <= 128 ? 1 : (fours <= 1024 ? 2 : 4);
+    const int threads = ((fours + ch - 1) / ch + 31) / 32 * 32;
+    const bool vec4 = H % 4 == 0 && (all & 15) == 0 && threads <= 1024;
     const size_t smem = vec4 ? 0 : (size_t)H * sizeof(float);
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+#define NORM_ADD_ROW(TD, TO, NT, CH)                                                                                       \
+    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, norm_add_kernel<TD, TO, NT, CH>, T, threads, 0, stream, resid, terms, mult, vec, w, \
+                                  eps, layer_norm, (TO*)out, meta, H)
+#define NORM_ADD_TERMS(TD, TO, CH)                        \
+    do {                                                  \
+        if (num_terms == 1) NORM_ADD_ROW(TD, TO, 1, CH);  \
+        if (num_terms == 2) NORM_ADD_ROW(TD, TO, 2, CH);  \
+        NORM_ADD_ROW(TD, TO, 0, CH);                      \
+    } while (0)
 #define NORM_ADD_CASE(TD, TO)                                                                                              \
     do {                                                                                                                  \
+        if (vec4) {                                                                                                       \
+            if (ch == 1) NORM_ADD_TERMS(TD, TO, 1);                                                                       \
+            if (ch == 2) NORM_ADD_TERMS(TD, TO, 2);                                                                       \
+            NORM_ADD_TERMS(TD, TO, NS_CHUNKS);                                                                            \
+        }                                                                                                                 \
         static size_t configured = 0;                                                                                     \
         if (smem > 40 * 1024 && smem > configured) {                                                                      \
-            cudaError_t ce = cudaFuncSetAttribute(norm_add_kernel<TD, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t ce = cudaFuncSetAttribute(norm_add_scalar_kernel<TD, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (ce != cudaSuccess) return (int)ce;                                                                        \
             configured = smem;                                                                                            \
         }                                                                                                                 \
-        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, norm_add_kernel<TD, TO>, T, threads, smem, stream, resid, terms, mult, vec, w, \
-                                      eps, layer_norm, (TO*)out, meta, H, vec4);                                          \
+        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, norm_add_scalar_kernel<TD, TO>, T, 256, smem, stream, resid, terms, mult, vec, w, \
+                                      eps, layer_norm, (TO*)out, meta, H);                                                \
     } while (0)
     if (term_dtype == DT_F32 && out_dtype == DT_F32) NORM_ADD_CASE(float, float);
     if (term_dtype == DT_BF16 && out_dtype == DT_BF16) NORM_ADD_CASE(__nv_bfloat16, __nv_bfloat16);
-    if (term_dtype == DT_F32) NORM_ADD_CASE(float, __nv_bfloat16);
     return (int)cudaErrorInvalidValue;
 #undef NORM_ADD_CASE
+#undef NORM_ADD_TERMS
+#undef NORM_ADD_ROW
 }
 
 // ----------------------------------------------------------------------------- layer norm of rows

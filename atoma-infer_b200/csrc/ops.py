@@ -29,6 +29,7 @@ ATTENTION_SOURCES = ["kernels/attention_bf16.cu"]
 GEMM_SOURCES = ["kernels/gemm_tcgen05.cu"]
 ATTENTION_TC_SOURCES = ["kernels/attention_tcgen05.cu"]
 DECODE_STACK_SOURCES = ["kernels/decode_stack.cu"]
+ATTENTION_TALK_SOURCES = ["kernels/attention_talk.cu"]  # weights mixed across heads; one library per head size
 # parallel blocks, state-space mixers, latent attention, routed experts: built when a model first uses one of them
 MIXER_SOURCES = ["kernels/stream_ops.cu", "kernels/ssm.cu", "kernels/latent.cu", "kernels/moe.cu", "kernels/gated_stream.cu",
                  "kernels/normed_stream.cu", "kernels/talking_heads.cu"]
@@ -68,6 +69,8 @@ class CudaOps:
         self.launches = 0  # own kernel launches, counted for the benchmark record
         self._attn_libs = {}
         self._attn_tc_libs = {}
+        self._talk_libs = {}
+        self.fast_talking_attention = True  # tensor-core kernels for weights mixed across heads (False: the plain one; a test lever)
         # levers for the kernel tests (each kernel is compared with the one it stands in for)
         self.tc_attention = True    # tcgen05 prefill attention where the geometry allows
         self.decode_cluster = True  # split merge of the decode attention inside a cluster
@@ -129,7 +132,7 @@ class CudaOps:
     def set_pdl(self, on: bool) -> None:
         self.pdl = int(on)
         self.lib.kernels_set_pdl(int(on))
-        for lib in self._attn_libs.values():
+        for lib in list(self._attn_libs.values()) + list(self._talk_libs.values()):
             lib.kernels_set_pdl(1 if on else 0)
         for name in ("_mixer_lib", "_recurrent_lib", "_matrix_recurrent_lib"):
             if getattr(self, name, None) is not None:
@@ -1000,12 +1003,43 @@ class CudaOps:
                           num_pages: int, scale: float, talk, *, chunk: int = 0):
         """Attention over what the requests have cached whose softmax weights are mixed across the query heads, p'_h = sum_g
         talk[h, g] p_g, before head h weighs the values of its own key/value head; ``talk`` float32 [nq, nq].  ``chunk`` as for
-        ``attention``."""
+        ``attention``.  bfloat16 with a head size in steps of 16 up to 256 runs the tensor-core kernels where their shared
+        memory takes the heads (and, in decode steps, a request's visible keys); anything else runs the plain kernel."""
         if talk.dtype != torch.float32 or tuple(talk.shape) != (nq, nq) or not talk.is_contiguous():
             raise KernelError("the heads' mixing weights are contiguous float32 [heads, heads]")
+        if q.dtype == torch.bfloat16 and self.fast_talking_attention and d % 16 == 0 and d <= 256 and q_stride % 8 == 0:
+            lib = self._talk_library(d)
+            if ctx.decode_only:
+                seen = min(ctx.max_context, chunk) if chunk else ctx.max_context
+                least = lib.attn_talk_decode_min_splits(nq, nkv, seen)
+                if least:
+                    # about two blocks a multiprocessor, but no block of fewer than 64 keys; a request's blocks are one cluster
+                    splits = max(least, min(8, 2 * self.num_sms // max(ctx.S, 1), -(-seen // 64)), 1)
+                    if ctx.S <= SKINNY_MAX_ROWS:
+                        self._prefetch_next_weight(ctx.S)
+                    self._check(lib.attn_talk_decode(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.positions), _p(out),
+                                                     ctx.S, nq, nkv, page_size, num_pages, int(chunk), ctypes.c_float(scale), _p(talk),
+                                                     splits, ctx.max_context, _p(self.status), self._stream()), "attn_talk_decode")
+                    return
+            elif lib.attn_talk_prefill_supports(nq, nkv, int(chunk), ctx.max_context, page_size):
+                self._check(lib.attn_talk_prefill(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.cu_tokens),
+                                                  _p(ctx.context_lens), _p(out), ctx.S, ctx.max_tokens_per_entry, nq, nkv, page_size,
+                                                  num_pages, int(chunk), ctypes.c_float(scale), _p(talk), ctx.max_context,
+                                                  _p(self.status), self._stream()), "attn_talk_prefill")
+                return
         self._check(self._mixers().talk_attn_plain(_p(q), q_stride, _p(cache_layer), _code(q), _p(ctx.meta), group, _p(ctx.token_entry),
                                                    _p(ctx.positions), _p(out), ctx.T, nq, nkv, d, page_size, num_pages, int(chunk),
                                                    ctypes.c_float(scale), _p(talk), _p(self.status), self._stream()), "talk_attn_plain")
+
+    def _talk_library(self, d: int):
+        lib = self._talk_libs.get(d)
+        if lib is None:
+            lib = build.load_library(f"attention_talk_d{d}", ATTENTION_TALK_SOURCES, cuda=True, defines={"HEAD_DIM": d})
+            lib.kernels_set_pdl(1 if self.pdl else 0)
+            if lib.attn_talk_head_dim() != d:
+                raise KernelError(f"attention library was built for head size {lib.attn_talk_head_dim()}, wanted {d}")
+            self._talk_libs[d] = lib
+        return lib
 
     # ------------------------------------------------------------------ recurrences whose query reads more than the decayed state
     def _matrix_recurrent(self):
@@ -1049,7 +1083,8 @@ class CudaOps:
         lib = self._matrix_recurrent()
         slot_stride = self._slot_state(state, (heads, dim, vdim), "memory_scan")
         n_stride = self._slot_state(n_state, (heads, dim), "memory_scan")
-        if n_stride.value != slot_stride.value or m_state.stride(0) != slot_stride.value or m_state.stride(1) != 1:
+        # (with one slot the stride is nobody's business, and views may name any)
+        if state.shape[0] > 1 and (n_stride.value != slot_stride.value or m_state.stride(0) != slot_stride.value) or m_state.stride(1) != 1:
             raise KernelError("memory_scan: the three parts of a request's state share one slot")
         for t in (logits, o, nq, floor):
             if t.dtype != torch.float32 or not t.is_contiguous():

@@ -11,7 +11,8 @@ fraction of the measured HBM bandwidth.  Prints ONE JSON line.
 
 ``--designs`` instead of the benchmark: prefill and decode throughput of the Dosovik design beside Llama at equal
 layer sizes, and the design's own kernels beside Llama's like kernels with their fractions of the copy bandwidth.
-``--kulivik``: the same for the Kulivik design (windowed, biased and convolved attention, linear attention with constant
+``--kavotar``: the same for the Kavotar design (attention with weights mixed across heads beside a decaying state with a
+bonus, matrix memories with exponential gates, routed experts), beside Llama and Kulivik.  ``--kulivik``: the same for the Kulivik design (windowed, biased and convolved attention, linear attention with constant
 decays, routed experts), beside Llama and Bumolix.  ``--bumolix``: the same for the Bumolix design (attention beside gated linear attention, selective-scan layers), beside
 Llama and Tutezen.  ``--tutezen``: the same for the Tutezen design (state-space and latent-attention layers, routed experts) at Llama's width
 and as many layer runs.
@@ -307,6 +308,21 @@ def kulivik_config(size: str, layers: int, vocab: int = 32768, window: int = 102
             "layers": [kinds[i % 3] for i in range(layers)]}
 
 
+def kavotar_config(size: str, layers: int, vocab: int = 32768, chunk: int = 1024):
+    """A Kavotar configuration of the width and heads of ``size``: layers whose mixer is attention with weights mixed across
+    the heads (chunks of ``chunk``, half of a head rotated) beside token mixing with a bonus (heads of 64, as wide as the
+    model) alternate with matrix memories (width / 256 heads of 128 key and 256 value channels); every layer has routed
+    experts (a quarter of the feed-forward size of ``size`` each, two of sixteen chosen, from three of four groups)."""
+    H, I, nq, nkv, d = DESIGN_SIZES[size]
+    left = {"heads": nq, "kv_heads": nkv, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": chunk},
+            "rot": {"dims": d // 2, "base": 500000.0}}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 3}}, "expert": {"ff": I // 4}}
+    pair = [{"type": "parallel", "mixer": {"left": left, "right": {"heads": H // 64, "dim": 64}}, "mlp": moe},
+            {"type": "mlstm", "mixer": {"heads": H // 256, "dim": 128, "vdim": 256, "gate_cap": 15.0}, "mlp": moe}]
+    return {"architecture": "Kavotar", "vocab": vocab, "width": H, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [pair[i % 2] for i in range(layers)]}
+
+
 def design_comparison(args, other: str = "dosovik") -> int:
     """Prefill (one prompt of 2,048 tokens) and decode (8 requests, 2,048 tokens cached each, captured graphs)
     through the step function for both designs at each size; then single kernels.  Timing: CUDA events, the median
@@ -335,7 +351,7 @@ def design_comparison(args, other: str = "dosovik") -> int:
         return statistics.median(out)
 
     rows = []
-    for size in DESIGN_SIZES:
+    for size in () if args.kernels_alone else DESIGN_SIZES:
         pairs = design_configs(size, layers)
         names = ("llama", other)
         if other == "tutezen":  # two layers fewer: the middle two run twice, so a step runs as many layers as Llama's
@@ -346,6 +362,9 @@ def design_comparison(args, other: str = "dosovik") -> int:
         if other == "kulivik":  # beside Llama (equal sizes) and Bumolix (the closest design: two mixers side by side)
             names = ("llama", "bumolix", other)
             pairs = (pairs[0], bumolix_config(size, layers), kulivik_config(size, layers))
+        if other == "kavotar":  # beside Llama (equal sizes) and Kulivik (the closest design: two mixers side by side, routed experts)
+            names = ("llama", "kulivik", other)
+            pairs = (pairs[0], kulivik_config(size, layers), kavotar_config(size, layers))
         for name, cfg in zip(names, pairs):
             with tempfile.TemporaryDirectory() as d:
                 with open(os.path.join(d, "config.json"), "w") as f:
@@ -389,7 +408,8 @@ def design_comparison(args, other: str = "dosovik") -> int:
             print(json.dumps(row), flush=True)
             del lm
             torch.cuda.empty_cache()
-    kernels = {"tutezen": tutezen_kernels, "bumolix": bumolix_kernels, "kulivik": kulivik_kernels}.get(other, design_kernels)
+    kernels = {"tutezen": tutezen_kernels, "bumolix": bumolix_kernels, "kulivik": kulivik_kernels,
+               "kavotar": kavotar_kernels}.get(other, design_kernels)
     kernels(make_runtime("bfloat16", "cuda:0"), hbm, median_ms)
     return 0
 
@@ -835,6 +855,136 @@ def kulivik_kernels(rt, hbm, median_ms) -> None:
     ops.check_status()
 
 
+def kavotar_kernels(rt, hbm, median_ms) -> None:
+    """The Kavotar layers' own kernels beside the framework's like kernels, alone, at width 2048 (the sizes of
+    ``kavotar_config("w2048-h64", ...)``): microseconds a call and the fraction of the copy bandwidth that the bytes each
+    must move give; for the recurrences and the attention kernels the rate of their arithmetic.  Rows of 16,384 tokens and of
+    8 tokens (a decode step: the time of a launch inside a graph)."""
+    import torch
+
+    sys.path.insert(0, os.path.join(ROOT, "tests"))
+    import kernel_utils as K
+    from atoma_infer_b200.parts.base import PendingSum
+
+    ops, dev, bf = rt.ops, rt.device, torch.bfloat16
+    H, I = 2048, 8192
+    nq, nkv, d = 32, 8, 64
+    rh, rN, rank = 32, 64, 16          # token mixing: heads, channels of a head, the decay map's width
+    gh, gN, gP = 8, 128, 256           # matrix memory, and Bumolix's gated linear attention
+    E, top = 16, 2
+    print(f"kernels alone (copy bandwidth {hbm:.0f} GB/s): name, rows, us, bytes moved / time / copy bandwidth, or the rate")
+    for T in (16384, 8):
+        entries = [(0, T)] if T > 64 else [(100 + i, 1) for i in range(T)]
+        S = len(entries)
+        tables, num_pages = K.scrambled_tables([c + n for c, n in entries], PAGE, 0)
+        ctx, _ = K.make_context(rt, entries, PAGE, tables)
+        rnd = lambda *shape: torch.randn(*shape, device=dev)  # noqa: E731
+        resid, w = rnd(T, H), torch.ones(H, device=dev)
+        a, b, c = (rnd(T, H).to(bf) for _ in range(3))
+        out, out2 = (torch.empty(T, H, device=dev, dtype=bf) for _ in range(2))
+        mu5, mixed = torch.rand(5, H, device=dev), torch.empty(5, T, H, device=dev, dtype=bf)
+        mu, kept, last = torch.rand(H, device=dev), torch.zeros(S, H, device=dev), torch.empty(S, H, device=dev)
+        gate32, gbias = rnd(T, H), torch.zeros(H, device=dev)
+        qkv = rnd(T, (nq + 2 * nkv) * d).to(bf)
+        cache = torch.zeros(num_pages, 2, nkv, PAGE, d, device=dev, dtype=bf)
+        q_out = torch.empty(T, nq * d, device=dev, dtype=bf)
+        bias, inv_freq = torch.ones((nq + 2 * nkv) * d, device=dev, dtype=bf), torch.ones(d // 2, device=dev)
+        hw, temp = torch.ones(d, device=dev, dtype=bf), torch.ones(nq, device=dev)
+        I4 = rh * rN
+        r_in = (rnd(3, T, I4) * 0.5).to(bf)
+        r_z, r_w0, r_u = rnd(T, I4) - 3.0, torch.zeros(I4, device=dev), torch.ones(I4, device=dev)
+        r_state, r_o, r_y = torch.zeros(S, rh, rN, rN, device=dev), torch.empty(T, I4, device=dev), torch.empty(T, I4, device=dev, dtype=bf)
+        r_w = torch.ones(I4, device=dev)
+        w_in = (rnd(4, I4, H) * 0.02).to(bf)
+        low, act16 = rnd(T, rank), torch.empty(T, rank, device=dev, dtype=bf)
+        g_proj = (rnd(T, 2 * gh * gN + 2 * gh * gP) * 0.5).to(bf)
+        g_z, g_bias = rnd(T, gh * gN), torch.zeros(gh * gN, device=dev)
+        flat = torch.zeros(S, gh * gN * gP + gh * gN + gh, device=dev)
+        m_state, m_n, m_m = flat[:, :gh * gN * gP].view(S, gh, gN, gP), flat[:, gh * gN * gP:gh * gN * gP + gh * gN].view(S, gh, gN), flat[:, gh * gN * gP + gh * gN:]
+        g_state, g_o = torch.zeros(S, gh, gN, gP, device=dev), torch.empty(T, gh * gP, device=dev)
+        m_logits, m_bias, m_nq, m_floor = rnd(T, 2 * gh), torch.zeros(2 * gh, device=dev), torch.empty(T, gh, device=dev), torch.ones(T, gh, device=dev)
+        g_y, g_w, m_w = torch.empty(T, gh * gP, device=dev, dtype=bf), torch.ones(gP, device=dev), torch.ones(gh * gP, device=dev)
+        x, wr, rb = rnd(T, H).to(bf), rnd(E, H), rnd(E)
+        ids, wts = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, device=dev)
+        twice = 2 if T >= 128 else 1  # (chunks of time run twice)
+        rows_b = T * (nq + 2 * nkv) * d * 2 * 2
+        qk, kk, vv = g_proj[:, :gh * gN], g_proj[:, gh * gN:2 * gh * gN], g_proj[:, 2 * gh * gN:2 * gh * gN + gh * gP]
+        gg = g_proj[:, 2 * gh * gN + gh * gP:]
+        cases = [
+            ("kavotar: layer norm of two normed terms, sum into the stream + next input",
+             lambda: ops.norm_add(resid, PendingSum((a, b), 1.0, factors=(0.5, 0.5), norms=((w, 1e-5), (w, 1e-5))), w, 1e-5, ctx, layer_norm=True, out=out),
+             T * H * (2 * 2 + 4 + 4 + 2), None),
+            ("kavotar: layer norm of one term, sum into the stream + next input",
+             lambda: ops.norm_add(resid, PendingSum((a,)), w, 1e-5, ctx, layer_norm=True, out=out), T * H * (2 + 4 + 4 + 2), None),
+            ("kulivik: gate, norm of two weighted terms, sum into the stream + next norm",
+             lambda: ops.gated_norm_add(resid, PendingSum((a, b), 1.0, factors=(0.7, 0.4)), gate32, gbias, w, 1e-6, ctx, next_norm=(w, 1e-6, out), keep=(last, kept)),
+             T * H * (2 * 2 + 4 + 4 + 4 + 2), None),
+            ("llama:   add + RMSNorm", lambda: ops.add_rmsnorm(resid, a, w, 1e-5, out, ctx.meta, T), T * H * (4 + 2 + 4 + 2), None),
+            ("kavotar: five rows moved toward the token before (+ kept row)",
+             lambda: (ops.token_mix(resid, mu5, kept, ctx, mixed) or ops.keep_last_rows(resid, kept, ctx)), T * H * (4 + 5 * 2), None),
+            ("kulivik: norm + row shifted toward the token before", lambda: ops.norm_shift(resid, w, 1e-6, ctx, shift=mu, state=kept, h=out, hs=out2, last=last),
+             T * H * (4 + 2 + 2), None),
+            ("kavotar: four linears of 2048 x 2048 with rows of their own", lambda: ops.linears(mixed[:4], w_in, meta=ctx.meta),
+             4 * I4 * H * 2 + 4 * T * (H + I4) * 2, 2.0 * 4 * T * I4 * H),
+            ("llama:   one linear of 8192 x 2048", lambda: ops.linear(mixed[0], w_in.view(4 * I4, H), meta=ctx.meta), 4 * I4 * H * 2 + T * (H + 4 * I4) * 2,
+             2.0 * 4 * T * I4 * H),
+            ("kavotar: tanh of the decay map", lambda: ops.tanh_rows(low, act16, ctx.meta), T * rank * 6, None),
+            ("kavotar: attention rows (weighted norm per head, half rotation, scale per head, pages)",
+             lambda: ops.qkv_prepare(qkv, ctx, cache, 0, q_out, nq=nq, nkv=nkv, d=d, dv=d, dp=d, page_size=PAGE, num_pages=num_pages,
+                                     store_kv=True, q_norm=hw, k_norm=hw, eps=1e-5, inv_freq=inv_freq[:d // 4], rot=d // 2, head_norm=True, q_head_scale=temp),
+             rows_b, None),
+            ("kulivik: attention rows (bias, weighted norm per head, interleaved rotation, pages)",
+             lambda: ops.qkv_prepare(qkv, ctx, cache, 0, q_out, nq=nq, nkv=nkv, d=d, dv=d, dp=d, page_size=PAGE, num_pages=num_pages,
+                                     store_kv=True, bias=bias, q_norm=hw, k_norm=hw, eps=1e-6, inv_freq=inv_freq, rot=d, head_norm=True, interleaved=True),
+             rows_b, None),
+            ("kavotar: scan with a bonus, 32 x 64 x 64 (float32 FMA)",
+             lambda: ops.bonus_scan(r_in[0], r_in[1], r_in[2], r_z, r_w0, r_u, r_state, ctx, r_o, heads=rh, dim=rN, vdim=rN),
+             T * I4 * (3 * 2 + 4 + 4) + 2 * S * rh * rN * rN * 4, 6.0 * T * rh * rN * rN * twice),
+            ("kavotar: memory with exponential gates, 8 x 128 x 256 (float32 FMA)",
+             lambda: ops.memory_scan(qk, kk, vv, m_logits, m_bias, 15.0, gN ** -0.5, m_state, m_n, m_m, ctx, g_o, m_nq, m_floor, heads=gh, dim=gN, vdim=gP),
+             T * (2 * gh * gN * 2 + gh * gP * 2 + gh * gP * 4) + 2 * S * gh * gN * gP * 4, 6.0 * T * gh * gN * gP * twice),
+            ("bumolix: gated linear attention, 8 x 128 x 256 (float32 FMA)",
+             lambda: ops.gla_scan(qk, kk, vv, g_z, g_bias, 8.0, gN ** -0.5, g_state, ctx, g_o, heads=gh, dim=gN, vdim=gP),
+             T * (2 * gh * gN * 2 + gh * gP * 2 + gh * gN * 4 + gh * gP * 4) + 2 * S * gh * gN * gP * 4, 6.0 * T * gh * gN * gP * twice),
+            ("kavotar: norm per head, weight per channel, SiLU gate (32 x 64)",
+             lambda: ops.head_weight_norm_gate(r_o, r_in[0], r_w, 1e-5, r_y, ctx.meta, rh, kind="silu"), T * I4 * (4 + 2 + 2), None),
+            ("kavotar: normalizer, norm per head, weight per channel, sigmoid gate (8 x 256)",
+             lambda: ops.head_weight_norm_gate(g_o, gg, m_w, 1e-5, g_y, ctx.meta, gh, kind="sigmoid", nq=m_nq, floor=m_floor), T * gh * gP * (4 + 2 + 2), None),
+            ("bumolix: norm per head, shared weight, SiLU gate", lambda: ops.head_norm_gate(g_o, gg, g_w, 1e-5, g_y, ctx.meta, gh),
+             T * gh * gP * (4 + 2 + 2), None),
+            ("kavotar: router (sigmoid, correction, groups)", lambda: ops.moe_route_sigmoid(x, wr, rb, ids, wts, ctx.meta, groups=(4, 3)), T * H * 2, None),
+            ("kulivik: router (bias, weights over the chosen)", lambda: ops.moe_route(x, wr, ids, wts, ctx.meta, bias=rb, over_chosen=True), T * H * 2, None),
+        ]
+        for name, fn, nbytes, flops in cases:
+            us = _graph_us(fn, n=16 if T <= 64 else 2)
+            rate = f"  {flops / (us * 1e-6) / 1e12:7.1f} TFLOP/s" if flops else ""
+            print(f"  {name:88s} {T:5d} rows {us:9.1f} us  {nbytes / (us * 1e-6) / (hbm * 1e9):5.2f}{rate}")
+    # attention: a prompt of 16,384 tokens, and decode tokens over 2,048 cached ones (a chunk's last place: 1,024 keys)
+    talk = (torch.randn(nq, nq, device=dev) * 0.2).to(bf).float()
+    for T in (16384, 8, 64):
+        entries = [(0, T)] if T > 64 else [(2047, 1)] * T
+        tables, num_pages = K.scrambled_tables([c + n for c, n in entries], PAGE, 1)
+        ctx, _ = K.make_context(rt, entries, PAGE, tables)
+        cache = torch.randn(num_pages, 2, nkv, PAGE, d, device=dev).to(bf)
+        q, o = torch.randn(T, nq * d, device=dev).to(bf), torch.empty(T, nq * d, device=dev, dtype=bf)
+        for name, chunk, mixes in (("llama:   attention, 32 x 64 over 8 x 64, all keys", 0, False), ("bumolix: attention, chunks of 1024 + sink", 1024, False),
+                                   ("kavotar: attention, chunks of 1024, weights mixed across 32 heads", 1024, True),
+                                   ("kavotar: attention, all keys, weights mixed across 32 heads", 0, True)):
+            if mixes and chunk == 0 and T > 64:
+                continue
+            if mixes:
+                call = lambda: ops.talking_attention(q, nq * d, cache, ctx, 0, o, nq, nkv, d, PAGE, num_pages, 0.125, talk, chunk=chunk)  # noqa: E731
+            else:
+                kw = {"chunk": chunk, "sink": True} if chunk else {}
+                call = lambda: ops.attention(q, nq * d, cache, ctx, 0, o, nq, nkv, d, PAGE, num_pages, 0, 0.125, **kw)  # noqa: E731
+            us = _graph_us(call, n=4)
+            keys = (chunk or T) / 2 if T > 64 else (chunk or 2048)
+            flops = (4.0 * d + (2.0 * nq if mixes else 0.0)) * T * nq * keys
+            of_copy = f"  {T * keys * nkv * d * 4 / (us * 1e-6) / (hbm * 1e9):5.2f}" if T <= 64 else "       "
+            print(f"  {name:88s} {T:5d} rows {us:9.1f} us{of_copy}  {flops / (us * 1e-6) / 1e12:7.1f} TFLOP/s")
+    ops.check_status()
+
+
 def layer_kernel_phases(eng, args, prompt, greedy, cfg) -> int:
     """Decode steps through the persistent layer kernel (csrc/kernels/decode_stack.cu), eagerly, with every block
     writing the global clock after each phase and each barrier of each layer; prints the mean, the slowest and the
@@ -947,6 +1097,9 @@ def main() -> int:
                          "width and as many layer runs (a JSON line each), then the design's kernels alone beside like kernels")
     ap.add_argument("--kulivik", action="store_true",
                     help="the Kulivik design beside Llama and Bumolix at equal layer sizes through the step function, then its kernels alone")
+    ap.add_argument("--kavotar", action="store_true",
+                    help="the Kavotar design beside Llama and Kulivik at equal layer sizes through the step function, then its kernels alone")
+    ap.add_argument("--kernels-alone", action="store_true", help="with an option that compares designs: only the kernels alone")
     ap.add_argument("--bumolix", action="store_true",
                     help="instead of the benchmark: prefill and decode throughput of the Bumolix design beside Llama and Tutezen "
                          "at equal width and as many layer runs (a JSON line each), then the design's kernels alone beside like kernels")
@@ -972,6 +1125,8 @@ def main() -> int:
         return design_comparison(args, other="tutezen")
     if args.bumolix:
         return design_comparison(args, other="bumolix")
+    if args.kavotar:
+        return design_comparison(args, other="kavotar")
     if args.kulivik:
         return design_comparison(args, other="kulivik")
     if args.model != "1b":
