@@ -5,8 +5,8 @@
 //  * talk_decode: one thread-block cluster per request (steps in which every request brings one token), its blocks share
 //    the visible keys.  Every block scores its keys for all heads (mma.sync, key fragments straight from the pages), the
 //    cluster exchanges the heads' maxima and sums through distributed shared memory, every block mixes its finished
-//    weights in float32 and weighs its values, and the cluster adds the blocks' results up in order.  Each key and value
-//    byte is read once; nothing goes through scratch memory.
+//    weights in float32 and weighs its values (mma.sync, value fragments straight from the pages), and the cluster adds
+//    the blocks' results up in order.  Each key and value byte is read once; nothing goes through scratch memory.
 //  * talk_prefill: one block per 16 tokens and request, all heads.  A first walk over the keys takes every head's maximum
 //    and sum; a second one takes the finished weights of a key tile for all heads into shared memory, mixes them on the
 //    tensor cores (a [heads x heads] times [heads x positions] product) and weighs the tile's values.
@@ -22,21 +22,43 @@ extern "C" int attn_talk_head_dim() { return D; }
 
 // ----------------------------------------------------------------------------- decode
 namespace {
-constexpr int TD_THREADS = 256, TD_WARPS = TD_THREADS / 32;
+constexpr int TD_THREADS = D <= 64 ? 512 : 256, TD_WARPS = TD_THREADS / 32;  // (wider heads need the registers)
 constexpr int TD_MAX_SPLITS = 8;
-constexpr int TD_HB = 4;                  // heads whose outputs a thread accumulates at a time
-constexpr int TD_LPK = D / 8;             // lanes that hold one value row (8 elements each)
-constexpr int TD_KPW = 32 / TD_LPK;       // value rows a warp reads at once
+constexpr int TD_DPR = D / 8;  // dimensions of a value row that a lane of the value phase holds
 
-// Warps that share an item (a key/value head and up to TD_HB of its query heads) of the value phase.
+// Warps that share an item (a key/value head and up to 16 of its query heads) of the value phase.
 __host__ __device__ inline int td_key_parts(int H, int G) {
-    const int items = G * ((H / G + TD_HB - 1) / TD_HB);
+    const int items = G * ((H / G + 15) / 16);
     return items >= TD_WARPS ? 1 : TD_WARPS / items;
 }
-// Shared memory of a block for n keys: q, the mixing weights transposed, weights, mixed weights, partial outputs, (m, l) pairs.
-__host__ __device__ inline int td_row(int n) { return (n + 31) / 32 * 32 + 4; }
-inline size_t td_smem(int H, int G, int n) {
-    return (size_t)H * D * sizeof(bf16) + ((size_t)H * ((H + 7) / 8 * 8) + 2 * (size_t)H * td_row(n) + (size_t)td_key_parts(H, G) * H * D + 4 * (size_t)H) * sizeof(float);
+__host__ __device__ inline int td_row(int n) { return (n + 31) / 32 * 32 + 4; }       // floats of a head's scores
+__host__ __device__ inline int td_mixed_row(int n) { return (n + 31) / 32 * 32 + 8; }  // elements of a head's mixed weights
+__host__ __device__ inline int td_owned(int H, int splits) { return ((H * D + splits - 1) / splits + 3) / 4 * 4; }
+// Shared memory of a block for n keys: q, the keys' places, the mixing weights transposed, weights, mixed weights, partial
+// outputs, the other blocks' parts of this block's outputs, (m, l) pairs, factors.
+inline size_t td_smem(int H, int G, int n, int splits) {
+    return (size_t)H * D * sizeof(bf16) + (size_t)td_row(n) * sizeof(long long) + (size_t)H * ((H + 7) / 8 * 8) * sizeof(float) +
+           (size_t)H * td_row(n) * sizeof(float) + (size_t)H * td_mixed_row(n) * sizeof(bf16) +
+           ((size_t)td_key_parts(H, G) * H * D + (size_t)splits * td_owned(H, splits) + 3 * (size_t)H) * sizeof(float);
+}
+// TD_DPR consecutive elements of a row as words of two (TD_DPR is even; a row's piece starts on TD_DPR * 2 bytes).
+__device__ __forceinline__ void load_words(const bf16* p, uint32_t (&w)[TD_DPR / 2]) {
+    if constexpr (TD_DPR % 8 == 0) {
+#pragma unroll
+        for (int i = 0; i < TD_DPR / 8; ++i) {
+            const uint4 v = reinterpret_cast<const uint4*>(p)[i];
+            w[4 * i] = v.x, w[4 * i + 1] = v.y, w[4 * i + 2] = v.z, w[4 * i + 3] = v.w;
+        }
+    } else if constexpr (TD_DPR % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < TD_DPR / 4; ++i) {
+            const uint2 v = reinterpret_cast<const uint2*>(p)[i];
+            w[2 * i] = v.x, w[2 * i + 1] = v.y;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < TD_DPR / 2; ++i) w[i] = reinterpret_cast<const uint32_t*>(p)[i];
+    }
 }
 }  // namespace
 
@@ -45,13 +67,17 @@ talk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
                    int group, const int* __restrict__ positions, bf16* __restrict__ out, int H, int chunk, float scale_log2,
                    const float* __restrict__ talk, int num_pages, int splits, int max_keys, int* __restrict__ status) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int G = L.num_kv_heads, HG = H / G, HP = (H + 7) / 8 * 8, NS = td_row(max_keys), parts = td_key_parts(H, G);
-    bf16* qs = reinterpret_cast<bf16*>(smem_raw);                              // [H][D]
-    float* tt = reinterpret_cast<float*>(smem_raw + (size_t)H * D * sizeof(bf16));  // [H][HP]: talk transposed, tt[g][h]
-    float* sc = tt + (size_t)H * HP;                                           // [H][NS]: scores, then weights
-    float* pm = sc + (size_t)H * NS;                                           // [H][NS]: mixed weights
-    float* po = pm + (size_t)H * NS;                                           // [parts][H][D]
-    float* ml = po + (size_t)parts * H * D;                                    // [H][2] of this block, then [H][2] of all blocks
+    const int G = L.num_kv_heads, HG = H / G, HP = (H + 7) / 8 * 8, NS = td_row(max_keys), NM = td_mixed_row(max_keys), parts = td_key_parts(H, G);
+    const int owned = td_owned(H, splits);
+    long long* off = reinterpret_cast<long long*>(smem_raw);                   // [NS]: a key's place in the cache, -1: none
+    bf16* qs = reinterpret_cast<bf16*>(off + NS);                              // [H][D]
+    bf16* pm = qs + (size_t)H * D;                                             // [H][NM]: mixed weights
+    float* tt = reinterpret_cast<float*>(pm + (size_t)H * NM);                 // [H][HP]: talk transposed, tt[g][h], then times g's factor
+    float* sc = tt + (size_t)H * HP;                                           // [H][NS]: scores, then their exponentials
+    float* po = sc + (size_t)H * NS;                                           // [parts][H][D]
+    float* recv = po + (size_t)parts * H * D;                                  // [splits][owned]
+    float* ml = recv + (size_t)splits * owned;                                 // [H][2]
+    float* fac = ml + 2 * (size_t)H;                                           // [H]
     pdl_launch_dependents();
     const int split = blockIdx.x, e = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     // (a block of a dead request leaves with its whole cluster)
@@ -62,99 +88,123 @@ talk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
         if (tid == 0) atomicExch(&status[STATUS_BAD_PAGE], 1 + pos);
         per = max_keys;
     }
-    const int lo = kstart + split * per, n = max(0, min(per, pos + 1 - lo));
+    const int lo = kstart + split * per, n = max(0, min(per, pos + 1 - lo)), blocks32 = (n + 31) / 32;
     const int* bt = meta + meta[META_BT_OFFSET + group] + (size_t)e * meta[META_BT_STRIDE + group];
-    const int ps = L.page_size, ps_shift = (ps & (ps - 1)) == 0 ? 31 - __clz(ps) : -1;
+    const int ps = L.page_size;
     const size_t v_off = (size_t)G * ps * D, page_stride = 2 * v_off;
+    for (int j = tid; j < blocks32 * 32; j += TD_THREADS) {
+        long long at = -1;
+        if (j < n) {
+            const int k = lo + j, page = bt[k / ps];
+            if (page > 0 && page < num_pages) at = (long long)((size_t)page * page_stride + (size_t)(k % ps) * D);
+            else atomicExch(&status[STATUS_BAD_PAGE], 1 + k);
+        }
+        off[j] = at;
+    }
     for (int i = tid; i < H * HP; i += TD_THREADS) {
-        const int g = i / HP, h = i % HP;
-        tt[i] = h < H ? talk[(size_t)h * H + g] : 0.f;
+        const int h = i / H, g = i % H;  // (neighbouring threads read neighbouring weights)
+        tt[g * HP + h] = h < H ? talk[(size_t)h * H + g] : 0.f;
     }
     pdl_wait();
     for (int i = tid; i < H * D / 8; i += TD_THREADS)
         reinterpret_cast<uint4*>(qs)[i] = *reinterpret_cast<const uint4*>(q + (size_t)e * q_stride + (size_t)i * 8);
-    // the row of a key (head 0's element 0 of its page's K block), null where there is none
-    auto key_row = [&](int j) -> const bf16* {
-        if (j >= n) return nullptr;
-        const int at = lo + j, pi = ps_shift >= 0 ? at >> ps_shift : at / ps, page = __ldg(bt + pi);
-        if (page <= 0 || page >= num_pages) {
-            atomicExch(&status[STATUS_BAD_PAGE], 1 + at);
-            return nullptr;
-        }
-        return cache + (size_t)page * page_stride + (size_t)(at - pi * ps) * D;
-    };
     __syncthreads();
-    // Scores: an item is a key/value head and 32 keys.  Both operands take the 16 dimensions of a k-step in the order
-    // (4t, 4t + 1 | 4t + 2, 4t + 3) for lane t of a quad, so a key fragment is one 8-byte load from the page.
-    const int r = lane >> 2, t4 = (lane & 3) * 4, blocks32 = (n + 31) / 32;
-    for (int item = warp; item < G * blocks32; item += TD_WARPS) {
-        const int c = item % G, k0 = (item / G) * 32;
-        uint2 kf[4][KSTEPS];
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt) {
-            const bf16* row = key_row(k0 + nt * 8 + r);
-#pragma unroll
-            for (int ks = 0; ks < KSTEPS; ++ks)
-                kf[nt][ks] = row ? *reinterpret_cast<const uint2*>(row + (size_t)c * ps * D + ks * 16 + t4) : make_uint2(0u, 0u);
-        }
-        for (int m0 = 0; m0 < HG; m0 += 16) {
-            float s[4][4];
-#pragma unroll
-            for (int nt = 0; nt < 4; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
-            const bool in0 = m0 + r < HG, in1 = m0 + r + 8 < HG;
-            const bf16* q0 = qs + (size_t)(c * HG + m0 + r) * D + t4;
-#pragma unroll
-            for (int ks = 0; ks < KSTEPS; ++ks) {
-                const uint2 x = in0 ? *reinterpret_cast<const uint2*>(q0 + ks * 16) : make_uint2(0u, 0u);
-                const uint2 y = in1 ? *reinterpret_cast<const uint2*>(q0 + 8 * D + ks * 16) : make_uint2(0u, 0u);
-                const uint32_t a[4] = {x.x, y.x, x.y, y.y};
-#pragma unroll
-                for (int nt = 0; nt < 4; ++nt) mma_bf16(s[nt], a, kf[nt][ks].x, kf[nt][ks].y);
-            }
+    // Scores: an item is a key/value head and 32 keys; the next item's keys are on their way while one is computed.  Both
+    // operands take the 16 dimensions of a k-step in the order (4t, 4t + 1 | 4t + 2, 4t + 3) for lane t of a quad, so a key
+    // fragment is one 8-byte load from the page.
+    const int r = lane >> 2, t4 = (lane & 3) * 4;
+    {
+        constexpr bool AHEAD = KSTEPS <= 8;
+        const int items = G * blocks32;
+        uint2 cur[4][KSTEPS], nxt[AHEAD ? 4 : 1][AHEAD ? KSTEPS : 1];
+        auto load_keys = [&](int item, auto& kf) {
+            const bf16* base = cache + (size_t)(item % G) * ps * D + t4;
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) {
-                const int key = k0 + nt * 8 + (lane & 3) * 2;
-                float2 u, v;
-                u.x = key < n ? s[nt][0] * scale_log2 : -INFINITY;
-                u.y = key + 1 < n ? s[nt][1] * scale_log2 : -INFINITY;
-                v.x = key < n ? s[nt][2] * scale_log2 : -INFINITY;
-                v.y = key + 1 < n ? s[nt][3] * scale_log2 : -INFINITY;
-                if (in0) *reinterpret_cast<float2*>(sc + (size_t)(c * HG + m0 + r) * NS + key) = u;
-                if (in1) *reinterpret_cast<float2*>(sc + (size_t)(c * HG + m0 + r + 8) * NS + key) = v;
+                const long long at = off[(item / G) * 32 + nt * 8 + r];
+#pragma unroll
+                for (int ks = 0; ks < KSTEPS; ++ks)
+                    kf[nt][ks] = at >= 0 ? *reinterpret_cast<const uint2*>(base + at + ks * 16) : make_uint2(0u, 0u);
+            }
+        };
+        if (AHEAD && warp < items) load_keys(warp, cur);
+        for (int item = warp; item < items; item += TD_WARPS) {
+            if constexpr (AHEAD) {
+                if (item + TD_WARPS < items) load_keys(item + TD_WARPS, nxt);
+            } else {
+                load_keys(item, cur);
+            }
+            const int c = item % G, k0 = (item / G) * 32;
+            for (int m0 = 0; m0 < HG; m0 += 16) {
+                float s[4][4];
+#pragma unroll
+                for (int nt = 0; nt < 4; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+                const bool in0 = m0 + r < HG, in1 = m0 + r + 8 < HG;
+                const bf16* q0 = qs + (size_t)(c * HG + m0 + r) * D + t4;
+#pragma unroll
+                for (int ks = 0; ks < KSTEPS; ++ks) {
+                    const uint2 x = in0 ? *reinterpret_cast<const uint2*>(q0 + ks * 16) : make_uint2(0u, 0u);
+                    const uint2 y = in1 ? *reinterpret_cast<const uint2*>(q0 + 8 * D + ks * 16) : make_uint2(0u, 0u);
+                    const uint32_t a[4] = {x.x, y.x, x.y, y.y};
+#pragma unroll
+                    for (int nt = 0; nt < 4; ++nt) mma_bf16(s[nt], a, cur[nt][ks].x, cur[nt][ks].y);
+                }
+#pragma unroll
+                for (int nt = 0; nt < 4; ++nt) {
+                    const int key = k0 + nt * 8 + (lane & 3) * 2;
+                    const bool k_in = key < n, k1_in = key + 1 < n;
+                    if (in0) *reinterpret_cast<float2*>(sc + (size_t)(c * HG + m0 + r) * NS + key) =
+                        make_float2(k_in ? s[nt][0] * scale_log2 : -INFINITY, k1_in ? s[nt][1] * scale_log2 : -INFINITY);
+                    if (in1) *reinterpret_cast<float2*>(sc + (size_t)(c * HG + m0 + r + 8) * NS + key) =
+                        make_float2(k_in ? s[nt][2] * scale_log2 : -INFINITY, k1_in ? s[nt][3] * scale_log2 : -INFINITY);
+                }
+            }
+            if constexpr (AHEAD) {
+#pragma unroll
+                for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+                    for (int ks = 0; ks < KSTEPS; ++ks) cur[nt][ks] = nxt[nt][ks];
             }
         }
     }
     __syncthreads();
-    // every head's maximum and sum over this block's keys, then over the cluster's
+    // every head's maximum and sum over this block's keys; the scores become exponentials against that maximum
     for (int h = warp; h < H; h += TD_WARPS) {
-        const float* row = sc + (size_t)h * NS;
+        float* row = sc + (size_t)h * NS;
         float mx = -INFINITY, sum = 0.f;
         for (int j = lane; j < n; j += 32) mx = fmaxf(mx, row[j]);
         mx = warp_max(mx);
-        for (int j = lane; j < n; j += 32) sum += fast_exp2(row[j] - mx);
+        for (int j = lane; j < blocks32 * 32; j += 32) {
+            const float p = j < n ? fast_exp2(row[j] - mx) : 0.f;
+            row[j] = p;
+            sum += p;
+        }
         sum = warp_sum(sum);
         if (lane == 0) ml[2 * h] = mx, ml[2 * h + 1] = sum;
     }
     cg::cluster_group cluster = cg::this_cluster();
     cluster.sync();
+    // what turns this block's exponentials into softmax weights, over all blocks of the cluster, in order
     for (int h = tid; h < H; h += TD_THREADS) {
-        float mx = -INFINITY, sum = 0.f;
-        for (int s = 0; s < splits; ++s) mx = fmaxf(mx, cluster.map_shared_rank(ml, s)[2 * h]);
-        for (int s = 0; s < splits; ++s) {
-            const float* o = cluster.map_shared_rank(ml, s);
-            if (o[2 * h] > -INFINITY) sum += o[2 * h + 1] * fast_exp2(o[2 * h] - mx);
+        float m[TD_MAX_SPLITS], l[TD_MAX_SPLITS], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+        for (int s = 0; s < TD_MAX_SPLITS; ++s) {  // independent loads, all in flight together
+            m[s] = -INFINITY, l[s] = 0.f;
+            if (s < splits) {
+                const float2 v = *reinterpret_cast<const float2*>(cluster.map_shared_rank(ml, s) + 2 * h);
+                m[s] = v.x, l[s] = v.y;
+            }
         }
-        ml[2 * H + 2 * h] = mx;
-        ml[2 * H + 2 * h + 1] = 1.f / sum;
+#pragma unroll
+        for (int s = 0; s < TD_MAX_SPLITS; ++s) mx = fmaxf(mx, m[s]);
+#pragma unroll
+        for (int s = 0; s < TD_MAX_SPLITS; ++s) sum += m[s] > -INFINITY ? l[s] * fast_exp2(m[s] - mx) : 0.f;
+        fac[h] = n > 0 ? fast_exp2(ml[2 * h] - mx) / sum : 0.f;
     }
     __syncthreads();
-    for (int h = warp; h < H; h += TD_WARPS) {
-        float* row = sc + (size_t)h * NS;
-        const float mx = ml[2 * H + 2 * h], inv = ml[2 * H + 2 * h + 1];
-        for (int j = lane; j < n; j += 32) row[j] = fast_exp2(row[j] - mx) * inv;
-    }
+    for (int i = tid; i < H * HP; i += TD_THREADS) tt[i] *= fac[i / HP];
     __syncthreads();
-    // The mix: a warp takes 32 keys and 8 heads at a time.
+    // The mix: a warp takes 32 keys and 8 heads at a time, float32.
     const int hb8 = HP / 8;
     for (int item = warp; item < hb8 * blocks32; item += TD_WARPS) {
         const int h0 = (item % hb8) * 8, j = (item / hb8) * 32 + lane;
@@ -167,85 +217,90 @@ talk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restr
         }
 #pragma unroll
         for (int i = 0; i < 8; ++i)
-            if (h0 + i < H) pm[(size_t)(h0 + i) * NS + j] = j < n ? acc[i] : 0.f;
+            if (h0 + i < H) pm[(size_t)(h0 + i) * NM + j] = __float2bfloat16_rn(acc[i]);
     }
     __syncthreads();
-    // Values: an item is a key/value head and up to TD_HB of its query heads; `parts` warps share an item's keys.  Lane
-    // (kl, x) of a warp holds elements 8 x .. of the row of every TD_KPW-th key.
-    const int hbs = (HG + TD_HB - 1) / TD_HB, kl = lane / TD_LPK, x8 = (lane % TD_LPK) * 8, part = warp % parts;
-    for (int item = warp / parts; item < G * hbs; item += TD_WARPS / parts) {
-        const int c = item / hbs, h0 = c * HG + (item % hbs) * TD_HB, nh = min(TD_HB, (c + 1) * HG - h0);
-        float acc[TD_HB][8];
+    // Values: an item is a key/value head and up to 16 of its query heads; `parts` warps share an item's keys, 16 at a step.
+    // Lane (r, t) holds dimensions r * TD_DPR .. of keys 4t .. 4t + 3 of a step: the operand's column r of tile j is
+    // dimension r * TD_DPR + j, its rows the keys in that order, which the weights' fragment (two 8-byte loads) takes too.
+    {
+        const int mt = (HG + 15) / 16, part = warp % parts, steps = blocks32 * 2;
+        constexpr int UN = TD_DPR <= 8 ? 2 : 1;  // steps in flight a warp
+        for (int item = warp / parts; item < G * mt; item += TD_WARPS / parts) {
+            const int c = item / mt, h0 = c * HG + (item % mt) * 16, nh = min(16, (c + 1) * HG - h0);
+            const bf16* base = cache + v_off + (size_t)c * ps * D + r * TD_DPR;
+            float acc[TD_DPR][4];
 #pragma unroll
-        for (int i = 0; i < TD_HB; ++i)
+            for (int j = 0; j < TD_DPR; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+            for (int s0 = part; s0 < steps; s0 += parts * UN) {
+                uint32_t w[UN][4][TD_DPR / 2];
 #pragma unroll
-            for (int k = 0; k < 8; ++k) acc[i][k] = 0.f;
-        constexpr int UN = 4;  // rows in flight a lane
-        for (int j0 = part * TD_KPW; j0 < n; j0 += parts * TD_KPW * UN) {
-            uint4 v[UN];
-#pragma unroll
-            for (int u = 0; u < UN; ++u) {
-                const int j = j0 + u * parts * TD_KPW + kl;
-                v[u] = make_uint4(0u, 0u, 0u, 0u);
-                if (kl < TD_KPW) {
-                    const bf16* row = key_row(j);
-                    if (row) v[u] = *reinterpret_cast<const uint4*>(row + v_off + (size_t)c * ps * D + x8);
-                }
-            }
-#pragma unroll
-            for (int u = 0; u < UN; ++u) {
-                const int j = j0 + u * parts * TD_KPW + kl;
-                if (kl < TD_KPW && j < n) {
-                    float f[8];
-                    const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&v[u]);
+                for (int u = 0; u < UN; ++u)
 #pragma unroll
                     for (int k = 0; k < 4; ++k) {
-                        const float2 z = __bfloat1622float2(b[k]);
-                        f[2 * k] = z.x;
-                        f[2 * k + 1] = z.y;
+                        const int st = s0 + u * parts;
+                        const long long at = st < steps ? off[st * 16 + t4 + k] : -1;
+                        if (at >= 0) {
+                            load_words(base + at, w[u][k]);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < TD_DPR / 2; ++i) w[u][k][i] = 0u;
+                        }
                     }
 #pragma unroll
-                    for (int i = 0; i < TD_HB; ++i) {
-                        if (i >= nh) continue;
-                        const float p = pm[(size_t)(h0 + i) * NS + j];
+                for (int u = 0; u < UN; ++u) {
+                    const int st = s0 + u * parts;
+                    if (st >= steps) continue;
+                    const uint2 x = r < nh ? *reinterpret_cast<const uint2*>(pm + (size_t)(h0 + r) * NM + st * 16 + t4) : make_uint2(0u, 0u);
+                    const uint2 y = r + 8 < nh ? *reinterpret_cast<const uint2*>(pm + (size_t)(h0 + r + 8) * NM + st * 16 + t4) : make_uint2(0u, 0u);
+                    const uint32_t a[4] = {x.x, y.x, x.y, y.y};
 #pragma unroll
-                        for (int k = 0; k < 8; ++k) acc[i][k] = fmaf(p, f[k], acc[i][k]);
+                    for (int j = 0; j < TD_DPR; ++j) {
+                        const uint32_t sel = j & 1 ? 0x7632u : 0x5410u;
+                        mma_bf16(acc[j], a, __byte_perm(w[u][0][j / 2], w[u][1][j / 2], sel), __byte_perm(w[u][2][j / 2], w[u][3][j / 2], sel));
                     }
                 }
             }
-        }
+            const int d0 = (lane & 3) * 2 * TD_DPR;
 #pragma unroll
-        for (int i = 0; i < TD_HB; ++i) {
-            if (i >= nh) continue;
+            for (int b = 0; b < 2; ++b) {
+                if (r + 8 * b >= nh) continue;
+                float* dst = po + ((size_t)part * H + h0 + r + 8 * b) * D + d0;
 #pragma unroll
-            for (int k = 0; k < 8; ++k) {
-                float a = acc[i][k];
-#pragma unroll
-                for (int o = 1; o < TD_KPW; ++o) a += __shfl_sync(0xffffffffu, acc[i][k], (lane + o * TD_LPK) & 31);
-                if (kl == 0) po[((size_t)part * H + h0 + i) * D + x8 + k] = a;
+                for (int j = 0; j < TD_DPR; ++j) {
+                    dst[j] = acc[j][2 * b];
+                    dst[TD_DPR + j] = acc[j][2 * b + 1];
+                }
             }
         }
     }
-    cluster.sync();
-    // the cluster's blocks share the outputs; every sum runs over the blocks in order, and over an item's warps in order
-    for (int i = split * TD_THREADS + tid; i < H * D; i += splits * TD_THREADS) {
+    __syncthreads();
+    // Block s of the cluster owns outputs s * owned ..: every block hands it its part (an item's warps in order), and the
+    // owner adds the blocks' parts up in order.
+    for (int i = tid; i < H * D; i += TD_THREADS) {
         float a = 0.f;
-        for (int s = 0; s < splits; ++s) {
-            const float* o = cluster.map_shared_rank(po, s);
-            for (int p = 0; p < parts; ++p) a += o[(size_t)p * H * D + i];
-        }
-        out[(size_t)e * H * D + i] = __float2bfloat16_rn(a);
+        for (int p = 0; p < parts; ++p) a += po[(size_t)p * H * D + i];
+        const int owner = i / owned;
+        cluster.map_shared_rank(recv, owner)[(size_t)split * owned + (i - owner * owned)] = a;
     }
-    cluster.sync();  // nobody leaves while its shared memory may still be read
+    cluster.sync();
+    for (int i = tid; i < owned && split * owned + i < H * D; i += TD_THREADS) {
+        float a = 0.f;
+        for (int s = 0; s < splits; ++s) a += recv[(size_t)s * owned + i];
+        out[(size_t)e * H * D + split * owned + i] = __float2bfloat16_rn(a);
+    }
 }
 
 // The fewest blocks a request's keys (at most max_keys of them) can be shared by, at most TD_MAX_SPLITS; 0: they do not fit.
 extern "C" int attn_talk_decode_min_splits(int nq, int nkv, int max_keys) {
     if (nkv <= 0 || nq % nkv) return 0;
     for (int s = 1; s <= TD_MAX_SPLITS; ++s)
-        if (td_smem(nq, nkv, ((max_keys + s - 1) / s + 7) / 8 * 8) <= 200 * 1024) return s;
+        if (td_smem(nq, nkv, ((max_keys + s - 1) / s + 7) / 8 * 8, s) <= 200 * 1024) return s;
     return 0;
 }
+
+// How many decode blocks a multiprocessor holds by threads and registers; the host sizes the splits by it.
+extern "C" int attn_talk_decode_blocks_per_sm() { return D <= 64 ? 1 : 2; }
 
 extern "C" int attn_talk_decode(const void* q, int q_stride, const void* cache, const int* meta, int group, const int* positions, void* out,
                                 int S, int nq, int nkv, int page_size, int num_pages, int chunk, float scale, const float* talk, int splits,
@@ -254,7 +309,7 @@ extern "C" int attn_talk_decode(const void* q, int q_stride, const void* cache, 
     if (nkv <= 0 || nq % nkv || splits < 1 || splits > TD_MAX_SPLITS || q_stride % 8 || ((uintptr_t)q & 15)) return (int)cudaErrorInvalidValue;
     const int seen = chunk > 0 && chunk < max_context ? chunk : max_context;
     const int max_keys = ((seen + splits - 1) / splits + 7) / 8 * 8;
-    const size_t smem = td_smem(nq, nkv, max_keys);
+    const size_t smem = td_smem(nq, nkv, max_keys, splits);
     if (smem > 220 * 1024) return (int)cudaErrorInvalidValue;
     static size_t configured = 0;  // grows only, and is not set again inside a stream capture once large enough
     if (smem > 48 * 1024 && smem > configured) {

@@ -118,33 +118,39 @@ extern "C" int memory_gates(const float* logits, const float* bias, float cap, f
 // ----------------------------------------------------------------------------- norm per head, a weight per channel, gate
 // out[t, h, :] = v / sqrt(mean(v^2) + eps) * w[h, :] * gate_fn(g[t, h, :]) with v = o[t, h, :], or, with `nq` and `floor_in`
 // (float32 [T, heads]), v = o[t, h, :] / (max(|nq|, floor) + 1e-6).  o float32 [T, heads * P], g a slice of wider rows, w float32
-// [heads * P]; kind 0: sigmoid(g), 1: g * sigmoid(g).  A warp a (token, head).
+// [heads * P]; kind 0: sigmoid(g), 1: g * sigmoid(g).  LPH lanes (a power of two) a (token, head).
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 head_weight_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ nq, const float* __restrict__ floor_in,
                              const T* __restrict__ g, long long g_stride, const float* __restrict__ w, float eps, int kind,
-                             T* __restrict__ out, const int* __restrict__ meta, int heads, int P, int vec4) {
+                             T* __restrict__ out, const int* __restrict__ meta, int heads, int P, int vec4, int LPH) {
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (t >= meta[META_NUM_TOKENS] || h >= heads) return;
-    const size_t at = ((size_t)t * heads + h) * P;
+    const int t = blockIdx.x, lane = threadIdx.x % LPH, h = blockIdx.y * (blockDim.x / LPH) + threadIdx.x / LPH;
+    if (t >= meta[META_NUM_TOKENS]) return;
+    const bool live = h < heads;  // (lanes without a head still take part in their warp's sums)
+    const size_t at = ((size_t)t * heads + (live ? h : 0)) * P;
     const float* row = o + at;
-    const T* gate = g + (size_t)t * g_stride + (size_t)h * P;
-    const float* wr = w + (size_t)h * P;
+    const T* gate = g + (size_t)t * g_stride + (size_t)(live ? h : 0) * P;
+    const float* wr = w + (size_t)(live ? h : 0) * P;
     float c = 1.f;
-    if (nq) c = 1.f / (fmaxf(fabsf(nq[(size_t)t * heads + h]), floor_in[(size_t)t * heads + h]) + 1e-6f);
+    if (nq && live) c = 1.f / (fmaxf(fabsf(nq[(size_t)t * heads + h]), floor_in[(size_t)t * heads + h]) + 1e-6f);
+    auto group_sum = [&](float v) {
+        for (int s = LPH >> 1; s > 0; s >>= 1) v += __shfl_xor_sync(0xffffffffu, v, s);
+        return v;
+    };
     float ss = 0.f;
     if (vec4) {
-        for (int i = lane * 4; i < P; i += 128) {
+        const int step = LPH * 4;
+        for (int i = lane * 4; i < P; i += step) {
             float v[4];
             load4(row + i, v);
 #pragma unroll
             for (int k = 0; k < 4; ++k) { v[k] *= c; ss = fmaf(v[k], v[k], ss); }
         }
-        ss = warp_sum(ss);
-        const float inv = rsqrtf(ss / (float)P + eps);
-        for (int i = lane * 4; i < P; i += 128) {
+        const float inv = rsqrtf(group_sum(ss) / (float)P + eps);
+        if (!live) return;
+        for (int i = lane * 4; i < P; i += step) {
             float v[4], gv[4], wv[4];
             load4(row + i, v);
             load4(gate + i, gv);
@@ -158,10 +164,10 @@ head_weight_norm_gate_kernel(const float* __restrict__ o, const float* __restric
         }
         return;
     }
-    for (int i = lane; i < P; i += 32) { const float v = row[i] * c; ss = fmaf(v, v, ss); }
-    ss = warp_sum(ss);
-    const float inv = rsqrtf(ss / (float)P + eps);
-    for (int i = lane; i < P; i += 32) {
+    for (int i = lane; i < P; i += LPH) { const float v = row[i] * c; ss = fmaf(v, v, ss); }
+    const float inv = rsqrtf(group_sum(ss) / (float)P + eps);
+    if (!live) return;
+    for (int i = lane; i < P; i += LPH) {
         const float gv = to_float(gate[i]), s = sigmoid_f(gv);
         out[at + i] = from_float<T>(row[i] * c * inv * wr[i] * (kind == 1 ? gv * s : s));
     }
@@ -171,12 +177,15 @@ extern "C" int head_weight_norm_gate(const float* o, const float* nq, const floa
                                      const float* w, float eps, int kind, void* out, const int* meta, int T, int heads, int P,
                                      cudaStream_t stream) {
     if (T <= 0) return 0;
-    const dim3 grid(T, (heads + 3) / 4);
     const int esz = dtype == DT_F32 ? 4 : 2;
     const int vec4 = P % 4 == 0 && g_stride % 4 == 0 && (((uintptr_t)o | (uintptr_t)w) & 15) == 0 && (((uintptr_t)g | (uintptr_t)out) % (4 * esz)) == 0;
+    int LPH = 1;
+    while (LPH < 32 && LPH * (vec4 ? 4 : 1) < P) LPH *= 2;
+    const int threads = heads * LPH > 128 ? 256 : 128;
+    const dim3 grid(T, (heads + threads / LPH - 1) / (threads / LPH));
     if (dtype == DT_F32)
-        return (int)launch_kernel(head_weight_norm_gate_kernel<float>, grid, 128, 0, stream, o, nq, floor_in, (const float*)g, g_stride, w, eps,
-                                  kind, (float*)out, meta, heads, P, vec4);
-    return (int)launch_kernel(head_weight_norm_gate_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, nq, floor_in, (const __nv_bfloat16*)g,
-                              g_stride, w, eps, kind, (__nv_bfloat16*)out, meta, heads, P, vec4);
+        return (int)launch_kernel(head_weight_norm_gate_kernel<float>, grid, threads, 0, stream, o, nq, floor_in, (const float*)g, g_stride, w, eps,
+                                  kind, (float*)out, meta, heads, P, vec4, LPH);
+    return (int)launch_kernel(head_weight_norm_gate_kernel<__nv_bfloat16>, grid, threads, 0, stream, o, nq, floor_in, (const __nv_bfloat16*)g,
+                              g_stride, w, eps, kind, (__nv_bfloat16*)out, meta, heads, P, vec4, LPH);
 }

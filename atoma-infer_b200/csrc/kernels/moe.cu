@@ -104,46 +104,64 @@ extern "C" int moe_route_biased(const void* h, int dtype, const float* w, const 
 // h) (float32, the logits as above), choice score c_e = s_e + correction[e].  With groups > 1 the experts form that many equal
 // groups of neighbours; a group's score is the sum of its two largest choice scores (its only one in groups of one), and only
 // experts of the `keep` best groups can be chosen.  The `top` largest choice scores choose (ties to the lower index, for
-// groups too); the weights are the chosen experts' s as they are.  The choice runs on the first warp.
-template <typename T>
-__global__ void __launch_bounds__(256)
+// groups too); the weights are the chosen experts' s as they are.
+// A block takes TOK tokens: a router row is read once for all of them, and a warp a token chooses.
+template <typename T, int TOK>
+__global__ void __launch_bounds__(512)
 moe_route_sigmoid_kernel(const T* __restrict__ h, const float* __restrict__ w, const float* __restrict__ correction,
                          int* __restrict__ ids, float* __restrict__ wts, const int* __restrict__ meta, int H, int E, int top, int groups,
                          int keep) {
-    extern __shared__ float z[];  // E scores, E choice scores, `groups` group scores, `groups` marks
+    extern __shared__ float sh[];  // per token: E scores, E choice scores, `groups` group scores, `groups` marks
     pdl_wait();
     pdl_launch_dependents();
-    const int t = blockIdx.x;
-    if (t >= meta[META_NUM_TOKENS]) return;
+    const int t0 = blockIdx.x * TOK, tokens = min(TOK, meta[META_NUM_TOKENS] - t0);
+    if (tokens <= 0) return;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-    const T* x = h + (size_t)t * H;
+    const int stride = 2 * E + (groups > 1 ? 2 * groups : 0);
+    const T* x = h + (size_t)t0 * H;
     const bool vec = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
-    float *c = z + E, *gs = c + E;
     for (int e = warp; e < E; e += nwarps) {
         const float* we = w + (size_t)e * H;
-        float acc = 0.f;
-        if (vec) {
-            float part[4] = {0.f, 0.f, 0.f, 0.f};
+        float acc[TOK];
+        if (vec) {  // four columns a lane and step; the order of a logit's sum depends on H alone
+            float part[TOK][4];
+#pragma unroll
+            for (int q = 0; q < TOK; ++q) part[q][0] = part[q][1] = part[q][2] = part[q][3] = 0.f;
+#pragma unroll 4
             for (int k = lane * 4; k < H; k += 128) {
-                float xv[4], wv[4];
-                load4(x + k, xv);
+                float wv[4];
                 load4(we + k, wv);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) part[i] = fmaf(xv[i], wv[i], part[i]);
+                for (int q = 0; q < TOK; ++q) {
+                    float xv[4];
+                    load4(x + (size_t)(q < tokens ? q : 0) * H + k, xv);
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) part[q][i] = fmaf(xv[i], wv[i], part[q][i]);
+                }
             }
-            acc = (part[0] + part[1]) + (part[2] + part[3]);
+#pragma unroll
+            for (int q = 0; q < TOK; ++q) acc[q] = (part[q][0] + part[q][1]) + (part[q][2] + part[q][3]);
         } else {
-            for (int k = lane; k < H; k += 32) acc = fmaf(to_float(x[k]), we[k], acc);
+#pragma unroll
+            for (int q = 0; q < TOK; ++q) {
+                acc[q] = 0.f;
+                for (int k = lane; k < H; k += 32) acc[q] = fmaf(to_float(x[(size_t)(q < tokens ? q : 0) * H + k]), we[k], acc[q]);
+            }
         }
-        acc = warp_sum(acc);
-        if (lane == 0) {
-            const float s = 1.f / (1.f + expf(-acc));
-            z[e] = s;
-            c[e] = s + correction[e];
+#pragma unroll
+        for (int q = 0; q < TOK; ++q) {
+            const float z = warp_sum(acc[q]);
+            if (lane == 0 && q < tokens) {
+                const float s = 1.f / (1.f + expf(-z));
+                sh[q * stride + e] = s;
+                sh[q * stride + E + e] = s + correction[e];
+            }
         }
     }
     __syncthreads();
-    if (warp != 0) return;
+    if (warp >= tokens) return;
+    const int t = t0 + warp;
+    float *z = sh + warp * stride, *c = z + E, *gs = c + E;
     // the largest of n values in shared memory, ties to the lower index; the winner is struck out
     auto take_best = [&](float* v, int n) {
         float bv = -INFINITY;
@@ -196,14 +214,21 @@ moe_route_sigmoid_kernel(const T* __restrict__ h, const float* __restrict__ w, c
 extern "C" int moe_route_sigmoid(const void* h, int dtype, const float* w, const float* correction, int* ids, float* wts, const int* meta,
                                  int T, int H, int E, int top, int groups, int keep, cudaStream_t stream) {
     if (T <= 0) return 0;
-    const size_t smem = ((size_t)2 * E + (groups > 1 ? 2 * groups : 0)) * sizeof(float);
-    if (smem > 48 * 1024 || top > E || groups < 1 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < top)
-        return (int)cudaErrorInvalidValue;
-    if (dtype == DT_F32)
-        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, moe_route_sigmoid_kernel<float>, T, 256, smem, stream, (const float*)h, w,
-                                      correction, ids, wts, meta, H, E, top, groups, keep);
-    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, moe_route_sigmoid_kernel<__nv_bfloat16>, T, 256, smem, stream,
-                                  (const __nv_bfloat16*)h, w, correction, ids, wts, meta, H, E, top, groups, keep);
+    if (top > E || groups < 1 || E % groups || keep < 1 || keep > groups || keep * (E / groups) < top) return (int)cudaErrorInvalidValue;
+    const size_t per = ((size_t)2 * E + (groups > 1 ? 2 * groups : 0)) * sizeof(float);
+    const int tok = T > 64 && 4 * per <= 48 * 1024 ? 4 : 1;  // few tokens: a block each
+    if (tok * per > 48 * 1024) return (int)cudaErrorInvalidValue;
+    const int threads = tok == 1 ? (E >= 16 ? 512 : 256) : 256, blocks = (T + tok - 1) / tok;
+#define ROUTE_CASE(TT, TOK)                                                                                                \
+    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, moe_route_sigmoid_kernel<TT, TOK>, blocks, threads, tok * per, stream, (const TT*)h, w, \
+                                  correction, ids, wts, meta, H, E, top, groups, keep)
+    if (dtype == DT_F32) {
+        if (tok == 4) ROUTE_CASE(float, 4);
+        ROUTE_CASE(float, 1);
+    }
+    if (tok == 4) ROUTE_CASE(__nv_bfloat16, 4);
+    ROUTE_CASE(__nv_bfloat16, 1);
+#undef ROUTE_CASE
 }
 
 // ----------------------------------------------------------------------------- pairs sorted by expert

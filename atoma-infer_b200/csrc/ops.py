@@ -1013,8 +1013,8 @@ class CudaOps:
                 seen = min(ctx.max_context, chunk) if chunk else ctx.max_context
                 least = lib.attn_talk_decode_min_splits(nq, nkv, seen)
                 if least:
-                    # about two blocks a multiprocessor, but no block of fewer than 64 keys; a request's blocks are one cluster
-                    splits = max(least, min(8, 2 * self.num_sms // max(ctx.S, 1), -(-seen // 64)), 1)
+                    # as many blocks as are resident at once, but none of fewer than 64 keys; a request's blocks are one cluster
+                    splits = max(least, min(8, lib.attn_talk_decode_blocks_per_sm() * self.num_sms // max(ctx.S, 1), -(-seen // 64)), 1)
                     if ctx.S <= SKINNY_MAX_ROWS:
                         self._prefetch_next_weight(ctx.S)
                     self._check(lib.attn_talk_decode(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.positions), _p(out),
