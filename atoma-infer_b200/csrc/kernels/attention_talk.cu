@@ -338,12 +338,12 @@ extern "C" int attn_talk_decode(const void* q, int q_stride, const void* cache, 
 
 // ----------------------------------------------------------------------------- prefill (and mixed steps)
 namespace {
-constexpr int TP_WARPS = 8, TP_THREADS = TP_WARPS * 32;
+constexpr int TP_WARPS = D <= 64 ? 16 : 8, TP_THREADS = TP_WARPS * 32;  // (wider heads need the registers)
 constexpr int TP_TOK = 16;  // tokens of a block
 
-// Heads whose outputs a warp keeps in registers, for H heads (more heads than 8 times this: blocks share them).
+// Heads whose outputs a warp keeps in registers, for H heads (more heads than a block's warps keep: blocks share them).
 inline int tp_heads_per_warp(int H) {
-    const int most = D <= 64 ? 4 : (D <= 128 ? 2 : 1);
+    const int most = D <= 128 ? 2 : 1;
     int n = 1;
     while (n < most && n * TP_WARPS < H) n *= 2;
     return n;
@@ -676,7 +676,6 @@ extern "C" int attn_talk_prefill(const void* q, int q_stride, const void* cache,
     } while (0)
     if (hpw == 1) TALK_PREFILL_TILE(1);
     if constexpr (D <= 128) if (hpw == 2) TALK_PREFILL_TILE(2);
-    if constexpr (D <= 64) if (hpw == 4) TALK_PREFILL_TILE(4);
     return (int)cudaErrorInvalidValue;
 #undef TALK_PREFILL_TILE
 #undef TALK_PREFILL_CASE
