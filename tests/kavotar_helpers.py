@@ -83,11 +83,32 @@ SCALES = {".mu.": 10.0, ".w0": 25.0, "right.w1": 4.0, "right.w2": 6.0, ".u": 12.
 
 
 def make_model(path: str, name: str, seed: int = 0, decisive: bool = False) -> str:
-    """``decisive``: corrections far apart, so that few choices hang on a lead that rounding to bfloat16 can turn (the choice
-    still depends on the token where two corrections lie close)."""
+    """What reads a matrix state (q of a memory, r of a token mixing) is drawn near what was written to it (k), and the bonus
+    is positive: a token finds itself, so no head's output is a near cancellation that its norm would blow up, whatever the
+    number format.  ``decisive``: corrections so far apart that the same experts of every layer run for every token: no choice
+    hangs on a lead that rounding to bfloat16 can turn (how choices follow the tokens is tested in float32)."""
+    import os
+
+    from atoma_infer_b200.weights.safetensors_io import write_safetensors
+
     cfg, _ = CONFIGS[name]
-    scales = dict(SCALES, correction=12.0) if decisive else SCALES
-    return helpers.make_model(path, cfg, seed=seed, scales=scales, norm_jitter=0.2)
+    d = helpers.make_model(path, cfg, seed=seed, scales=SCALES, norm_jitter=0.2)
+    w = helpers.read_weights(d)
+    for i, ly in enumerate(cfg["layers"]):
+        read, written = (f"l{i}.mix.q", f"l{i}.mix.k") if ly["type"] == "mlstm" else (f"l{i}.mix.right.r", f"l{i}.mix.right.k")
+        w[read] = w[written] + 0.4 * w[read]
+        if ly["type"] == "parallel":  # (both read nearly the same row too)
+            w[f"l{i}.mix.right.mu.r"] = w[f"l{i}.mix.right.mu.k"] + 0.3 * w[f"l{i}.mix.right.mu.r"]
+            w[f"l{i}.mix.right.u"] = w[f"l{i}.mix.right.u"].abs() + 0.3
+        if decisive and ly.get("mlp"):
+            r = ly["mlp"]["router"]
+            n = r.get("groups", {}).get("count", 1)
+            order = torch.randperm(n, generator=torch.Generator().manual_seed(seed + i))
+            per = r["experts"] // n
+            inside = torch.stack([torch.randperm(per, generator=torch.Generator().manual_seed(100 * seed + 10 * i + g)) for g in range(n)])
+            w[f"l{i}.mlp.correction"] = (1.25 * (order[:, None] * per + inside) - 4.0).reshape(-1)
+    write_safetensors(os.path.join(d, "model.safetensors"), {k: v.to(torch.bfloat16) for k, v in w.items()}, {})
+    return d
 
 
 def plain_logits(model_dir: str, cfg: dict, seqs: Dict[str, List[int]]) -> Dict[str, torch.Tensor]:
@@ -105,7 +126,7 @@ def plain_greedy(model_dir: str, cfg: dict, prompt: List[int], n: int) -> List[i
     return out
 
 
-def first_close_call(model_dir: str, cfg: dict, seqs: Dict[str, List[int]], lead: float = 0.004) -> Dict[str, int]:
+def first_close_call(model_dir: str, cfg: dict, seqs: Dict[str, List[int]], lead: float = 0.02) -> Dict[str, int]:
     """Per request the first position at which a router's choice (of experts or of groups) hangs on a lead of less than
     ``lead`` (the length of the request if there is none).  From there on a reduced-precision engine may rightly choose
     another expert, and every later position of the request reads what that choice left in the caches."""
@@ -120,10 +141,14 @@ def first_close_call(model_dir: str, cfg: dict, seqs: Dict[str, List[int]], lead
     return out
 
 
-def rounding_errors(model_dir: str, cfg: dict, seqs: Dict[str, List[int]], ref: Dict[str, torch.Tensor]) -> Dict[str, torch.Tensor]:
+def rounding_errors(model_dir: str, cfg: dict, seqs: Dict[str, List[int]], ref: Dict[str, torch.Tensor],
+                    dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
     """Per position, how far the plain implementation itself moves (largest logit difference over the largest logit of
-    the sequence) when what its matrix products read and write is rounded to bfloat16: the measure of how much a
-    position amplifies roundings that no implementation in that type can avoid."""
+    the sequence, the largest of three draws of the roundings) when what its matrix products read and write is rounded to
+    ``dtype``: the measure of how much a position amplifies roundings that no implementation in that type can avoid.
+    (float32: twice that, since a product's sum is then rounded at every step and not once.)"""
     w = helpers.read_weights(model_dir)
-    return {k: (PV.forward(cfg, w, v, round_to=torch.bfloat16) - ref[k]).abs().max(-1).values / ref[k].abs().max()
-            for k, v in seqs.items()}
+    f = 2.0 if dtype == torch.float32 else 1.0
+    worst = lambda k, v: torch.stack([(PV.forward(cfg, w, v, round_to=dtype, dither=s) - ref[k]).abs().max(-1).values  # noqa: E731
+                                      for s in (None, 1, 2)]).max(0).values
+    return {k: f * worst(k, v) / ref[k].abs().max() for k, v in seqs.items()}

@@ -15,23 +15,30 @@ import torch
 
 F = torch.float64
 
-_ROUND = None  # a storage type that matrix products read and write through (None: exact), see ``forward``
+_ROUND = None   # a storage type that matrix products read and write through (None: exact), see ``forward``
+_DITHER = None  # a generator that moves every value by up to half a unit of that type before it is rounded
 
 
 def t64(x):
     return x.to(F)
 
 
+def _rounded(x):
+    if _DITHER is not None:
+        x = x * (1.0 + torch.finfo(_ROUND).eps * (torch.rand(x.shape, generator=_DITHER, dtype=F) - 0.5))
+    return x.to(_ROUND).to(F)
+
+
 def lin(x, w):
     """x W^T; with a storage type set, what the product reads and what it writes is rounded to that type first."""
     if _ROUND is None:
         return x @ t64(w).T
-    return (x.to(_ROUND).to(F) @ t64(w).T).to(_ROUND).to(F)
+    return _rounded(_rounded(x) @ t64(w).T)
 
 
 def lin_wide(x, w):
     """Like ``lin``, with a result that is not rounded (what enters a recurrence's gates, a router)."""
-    return (x if _ROUND is None else x.to(_ROUND).to(F)) @ t64(w).T
+    return (x if _ROUND is None else _rounded(x)) @ t64(w).T
 
 
 def layer_norm(x, w, eps):
@@ -102,7 +109,7 @@ def attention(m, w, pre, x, eps):
     if rot:
         q, k = rotate_halves(q, rot["dims"], rot["base"]), rotate_halves(k, rot["dims"], rot["base"])
     if _ROUND is not None:
-        q, k = q.to(_ROUND).to(F), k.to(_ROUND).to(F)
+        q, k = _rounded(q), _rounded(k)
     mask = m.get("mask")
     p = head_weights(q, k, m["scale"], t64(w[pre + "temp"]), visible(T, mask["size"] if mask else None))
     o = weighted_values(mix_heads(p, w[pre + "talk"]), v)
@@ -225,16 +232,17 @@ def experts(f, w, pre, x, margins=None):
 
 
 # ---------------------------------------------------------------------------------------------- the model
-def forward(cfg, w, tokens, layers_out=None, margins=None, round_to=None):
+def forward(cfg, w, tokens, layers_out=None, margins=None, round_to=None, dither=None):
     """``layers_out``: a list that receives the stream after every layer; ``margins``: a list that receives, per routed
     layer, by how much every position's choice of experts (and of groups) leads what was not chosen; ``round_to``: a
-    storage type through which every matrix product reads and writes (to see how far rounding alone moves a position)."""
-    global _ROUND
-    _ROUND = round_to
+    storage type through which every matrix product reads and writes (to see how far rounding alone moves a position);
+    ``dither``: a seed; every value is moved by up to half a unit of that type first, another draw of the same roundings."""
+    global _ROUND, _DITHER
+    _ROUND, _DITHER = round_to, torch.Generator().manual_seed(dither) if dither is not None else None
     try:
         return _forward(cfg, w, tokens, layers_out, margins)
     finally:
-        _ROUND = None
+        _ROUND = _DITHER = None
 
 
 def _forward(cfg, w, tokens, layers_out, margins):
