@@ -351,14 +351,15 @@ inline int tp_heads_per_warp(int H) {
 inline int pad16(int n) { return (n + 15) / 16 * 16; }
 inline size_t tp_smem(int H, int G, int KT, int stages, int bt_cap) {
     return ((size_t)H * TP_TOK * LDS + (size_t)(stages + 1) * G * KT * LDS + (size_t)pad16(H) * TP_TOK * KT + (size_t)pad16(H) * (pad16(H) + 8)) * sizeof(bf16) +
-           (size_t)2 * H * TP_TOK * sizeof(float) + (size_t)bt_cap * sizeof(int);
+           (size_t)H * TP_TOK * sizeof(float) + (size_t)(bt_cap + H) * sizeof(int);
 }
 }  // namespace
 
 // Shared memory of the weights: head g's 16 x KT tile as 16-byte pieces of 8 keys, piece n * 16 + row at place (n * 16 + row) ^
 // (g & 7), so that the pieces of 8 neighbouring rows, and those of one row of 8 neighbouring heads, lie in different banks.
-template <int KT>
-__device__ __forceinline__ bf16* tp_piece(bf16* p, int g, int piece) { return p + (size_t)g * TP_TOK * KT + (size_t)((piece ^ (g & 7)) * 8); }
+// (The exclusive or stays inside groups of 8 pieces: n * 16 + 8 * (row / 8) + ((row % 8) ^ (g & 7)).)
+constexpr int TP_STATS = D <= 64 ? 2 : 4;  // heads a warp takes at a time in the first walk
+constexpr bool TP_Q_KEPT = D <= 64;        // ... with their queries' fragments in registers
 
 template <int KT, int HPW>
 __global__ void __launch_bounds__(TP_THREADS)
@@ -366,17 +367,17 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                     int group, const int* __restrict__ cu_tokens, const int* __restrict__ ctx_lens, bf16* __restrict__ out, int H,
                     int chunk, float scale_log2, const float* __restrict__ talk, int num_pages, int bt_cap, int stages,
                     int* __restrict__ status) {
-    constexpr int NK = KT / 8, MT = TP_WARPS * HPW > 16 ? TP_WARPS * HPW / 16 : 1;
+    constexpr int NK = KT / 8, MT = TP_WARPS * HPW > 16 ? TP_WARPS * HPW / 16 : 1, PH = TP_TOK * KT;  // PH: a head's weights
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int G = L.num_kv_heads, HG = H / G, HP = (H + 15) / 16 * 16, TS = HP + 8, ps = L.page_size;
     bf16* qt = reinterpret_cast<bf16*>(smem_raw);             // [H][16][LDS]
     bf16* kt = qt + (size_t)H * TP_TOK * LDS;                 // [stages][G][KT][LDS]
     bf16* vt = kt + (size_t)stages * G * KT * LDS;            // [G][KT][LDS]
-    bf16* pt = vt + (size_t)G * KT * LDS;                     // [HP][16 * KT], see tp_piece
-    bf16* tk = pt + (size_t)HP * TP_TOK * KT;                 // [HP][TS]: talk
-    float* ms = reinterpret_cast<float*>(tk + (size_t)HP * TS);  // [H][16]: a row's maximum
-    float* ls = ms + (size_t)H * TP_TOK;                      // [H][16]: its sum, then one over it
-    int* bt_s = reinterpret_cast<int*>(ls + (size_t)H * TP_TOK);
+    bf16* pt = vt + (size_t)G * KT * LDS;                     // [HP][PH]
+    bf16* tk = pt + (size_t)HP * PH;                          // [HP][TS]: talk
+    float* lse = reinterpret_cast<float*>(tk + (size_t)HP * TS);  // [H][16]: base-2 logarithm of a row's sum of exponentials
+    int* kv_of = reinterpret_cast<int*>(lse + (size_t)H * TP_TOK);  // [H]: where a head's keys and values start in a tile
+    int* bt_s = kv_of + H;
     pdl_launch_dependents();
     pdl_wait();
     // late query tiles see the most keys: they go first
@@ -408,110 +409,155 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
         const int h = idx / HP, g = idx % HP;
         tk[h * TS + g] = __float2bfloat16_rn(h < H && g < H ? talk[(size_t)h * H + g] : 0.f);
     }
-    for (int idx = tid; idx < (HP - H) * TP_TOK * KT; idx += TP_THREADS) pt[(size_t)H * TP_TOK * KT + idx] = __float2bfloat16_rn(0.f);
-    for (int i = tid; i < H * TP_TOK; i += TP_THREADS) ms[i] = -INFINITY, ls[i] = 0.f;
-    // keys (kv = 0) or values (kv = 1) of a tile for every head; positions outside [kbeg, kend_s) as zeros
+    for (int idx = tid; idx < (HP - H) * PH; idx += TP_THREADS) pt[(size_t)H * PH + idx] = __float2bfloat16_rn(0.f);
+    for (int h = tid; h < H; h += TP_THREADS) kv_of[h] = (h / HG) * KT * LDS;
+    // Keys (kv = 0) or values (kv = 1) of a tile for every head; positions outside [kbeg, kend_s) as zeros.  A thread copies
+    // 16 dimensions of the same rows of every few heads, so a row's page is looked up once.
+    constexpr int PAIRS = D / 16, PP = PAIRS <= 1 ? 1 : PAIRS <= 2 ? 2 : PAIRS <= 4 ? 4 : PAIRS <= 8 ? 8 : 16;
+    constexpr int RS = TP_THREADS / PP < KT ? TP_THREADS / PP : KT, CS = TP_THREADS / (PP * RS);
+    const int c16 = (tid % PP) * 16, rr0 = (tid / PP) % RS, cc0 = tid / (PP * RS);
     auto load_tile = [&](bf16* dst, int t, int kv) {
-        constexpr int PAIRS = D / 16;
-        for (int idx = tid; idx < G * KT * PAIRS; idx += TP_THREADS) {
-            const int c16 = (idx % PAIRS) * 16, rr = (idx / PAIRS) % KT, c = idx / PAIRS / KT, at = kbeg + t * KT + rr;
-            bf16* base = dst + (size_t)c * KT * LDS;
-            bf16 *d0 = base + toff(rr, c16), *d1 = base + toff(rr, c16 + 8);
+        if (c16 >= D) return;
+        for (int rr = rr0; rr < KT; rr += RS) {
+            const int at = kbeg + t * KT + rr;
             int page = -1, slot = 0;
             if (at < kend_s) {
                 const int pi = ps_shift >= 0 ? at >> ps_shift : at / ps;
                 slot = at - pi * ps;
                 page = bt_s[pi - page_lo];
             }
+            bf16 *d0 = dst + (size_t)cc0 * KT * LDS + toff(rr, c16), *d1 = dst + (size_t)cc0 * KT * LDS + toff(rr, c16 + 8);
             if (page > 0) {
-                const bf16* src = cache + (size_t)page * page_stride + (kv ? v_off : 0) + (size_t)(c * ps + slot) * D + c16;
-                cp_async_16(d0, src);
-                cp_async_16(d1, src + 8);
+                const bf16* src = cache + (size_t)page * page_stride + (kv ? v_off : 0) + (size_t)(cc0 * ps + slot) * D + c16;
+                for (int c = cc0; c < G; c += CS) {
+                    cp_async_16(d0, src);
+                    cp_async_16(d1, src + 8);
+                    d0 += CS * KT * LDS, d1 += CS * KT * LDS, src += (size_t)CS * ps * D;
+                }
             } else {
                 const uint4 z = make_uint4(0u, 0u, 0u, 0u);
-                *reinterpret_cast<uint4*>(d0) = z;
-                *reinterpret_cast<uint4*>(d1) = z;
+                for (int c = cc0; c < G; c += CS) {
+                    *reinterpret_cast<uint4*>(d0) = z;
+                    *reinterpret_cast<uint4*>(d1) = z;
+                    d0 += CS * KT * LDS, d1 += CS * KT * LDS;
+                }
             }
         }
     };
     auto k_stage = [&](int t) { return kt + (size_t)(stages == 2 ? t & 1 : 0) * G * KT * LDS; };
-    const int g4 = lane >> 2, pa = g4 < nt ? p_first + g4 : -1, pb = g4 + 8 < nt ? p_first + g4 + 8 : -1;
+    const int g4 = lane >> 2, tig = lane & 3, j8 = lane >> 3, l7 = lane & 7;
+    const int pa = g4 < nt ? p_first + g4 : -1, pb = g4 + 8 < nt ? p_first + g4 + 8 : -1;
     const int ca = chunk > 0 && pa >= 0 ? pa - pa % chunk : 0, cb = chunk > 0 && pb >= 0 ? pb - pb % chunk : 0;
     const int c_last = chunk > 0 ? p_last - p_last % chunk : 0;
-    // the scores of a head's 16 tokens against a tile, in base 2, masked
-    auto score = [&](int h, int t, float (&s)[NK][4]) {
-        uint32_t qf[Q_IN_REGS ? KSTEPS : 1][4];
+    // where a lane reads its share of a key fragment inside a tile (both halves of a k-step's 16 dimensions lie in one piece
+    // pair, so only the k-step moves it)
+    const int k_row = l7 + (j8 >> 1) * 8, k_col = (j8 & 1) * 8, q_row = l7 + (j8 & 1) * 8, q_col = (j8 >> 1) * 8;
+    // the products of a head's 16 tokens with a tile's keys, unscaled; -inf where a token does not see a key
+    auto score = [&](int h, const uint32_t (*qf)[4], const bf16* keys, int k0, bool whole, float (&s)[NK][4]) {
         const bf16* qh = qt + (size_t)h * TP_TOK * LDS;
-        if (Q_IN_REGS) {
+        const bf16* kh = keys + kv_of[h];
 #pragma unroll
-            for (int ks = 0; ks < KSTEPS; ++ks) load_a_frag(qf[ks], qh, ks, lane);
+        for (int n = 0; n < NK; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+#pragma unroll
+        for (int ks = 0; ks < KSTEPS; ++ks) {
+            uint32_t a[4];
+            if (qf) { a[0] = qf[ks][0]; a[1] = qf[ks][1]; a[2] = qf[ks][2]; a[3] = qf[ks][3]; }
+            else ldmatrix_x4(a, qh + toff(q_row, ks * 16 + q_col));
+#pragma unroll
+            for (int np = 0; np < NK / 2; ++np) {
+                uint32_t b[4];
+                ldmatrix_x4(b, kh + toff(np * 16 + k_row, ks * 16 + k_col));
+                mma_bf16(s[2 * np], a, b[0], b[1]);
+                mma_bf16(s[2 * np + 1], a, b[2], b[3]);
+            }
         }
-        qk_tile<NK>(s, qf, qh, k_stage(t) + (size_t)(h / HG) * KT * LDS, lane);
-        const int k0 = kbeg + t * KT;
-        if (nt == TP_TOK && k0 + KT - 1 <= p_first && k0 >= c_last) {  // a tile that every token sees whole
-#pragma unroll
-            for (int n = 0; n < NK; ++n)
-#pragma unroll
-                for (int c = 0; c < 4; ++c) s[n][c] *= scale_log2;
-            return;
-        }
+        if (whole) return;
 #pragma unroll
         for (int n = 0; n < NK; ++n)
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
-                const int key = k0 + n * 8 + (lane & 3) * 2 + (c & 1);
-                s[n][c] = (c < 2 ? key <= pa && key >= ca : key <= pb && key >= cb) ? s[n][c] * scale_log2 : -INFINITY;
+                const int key = k0 + n * 8 + tig * 2 + (c & 1);
+                if (!(c < 2 ? key <= pa && key >= ca : key <= pb && key >= cb)) s[n][c] = -INFINITY;
             }
     };
+    // a tile that every token sees whole
+    auto whole_tile = [&](int k0) { return nt == TP_TOK && k0 + KT - 1 <= p_first && k0 >= c_last; };
     __syncthreads();  // the table slice is written
-    // ---- first walk: every row's maximum and sum, for every head
-    load_tile(k_stage(0), 0, 0);
-    cp_async_commit();
-    for (int t = 0; t < ntiles; ++t) {
-        if (stages == 2 && t + 1 < ntiles) {
-            load_tile(k_stage(t + 1), t + 1, 0);
-            cp_async_commit();
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
+    // ---- first walk: every row's maximum and sum, for every head.  A lane keeps them for its own columns; the quad's four
+    // lanes are put together at the end.
+    for (int h0 = warp; h0 < H + warp; h0 += TP_WARPS * TP_STATS) {  // (all warps walk alike)
+        float m[TP_STATS][2], l[TP_STATS][2];
+#pragma unroll
+        for (int i = 0; i < TP_STATS; ++i) m[i][0] = m[i][1] = -INFINITY, l[i][0] = l[i][1] = 0.f;
+        uint32_t qf[TP_STATS][TP_Q_KEPT ? KSTEPS : 1][4];
+        if constexpr (TP_Q_KEPT) {
+#pragma unroll
+            for (int i = 0; i < TP_STATS; ++i)
+#pragma unroll
+                for (int ks = 0; ks < KSTEPS; ++ks)
+                    ldmatrix_x4(qf[i][ks], qt + (size_t)min(h0 + i * TP_WARPS, H - 1) * TP_TOK * LDS + toff(q_row, ks * 16 + q_col));
         }
-        __syncthreads();
-        for (int h = warp; h < H; h += TP_WARPS) {
-            float s[NK][4];
-            score(h, t, s);
+        load_tile(k_stage(0), 0, 0);
+        cp_async_commit();
+        for (int t = 0; t < ntiles; ++t) {
+            if (stages == 2 && t + 1 < ntiles) {
+                load_tile(k_stage(t + 1), t + 1, 0);
+                cp_async_commit();
+                cp_async_wait<1>();
+            } else {
+                cp_async_wait<0>();
+            }
+            __syncthreads();
+            const int k0 = kbeg + t * KT;
+            const bool whole = whole_tile(k0);
 #pragma unroll
-            for (int b = 0; b < 2; ++b) {
-                float mx = -INFINITY, sum = 0.f;
+            for (int i = 0; i < TP_STATS; ++i) {
+                const int h = h0 + i * TP_WARPS;
+                if (h >= H) continue;
+                float s[NK][4];
+                score(h, TP_Q_KEPT ? qf[i] : nullptr, k_stage(t), k0, whole, s);
 #pragma unroll
-                for (int n = 0; n < NK; ++n) mx = fmaxf(mx, fmaxf(s[n][2 * b], s[n][2 * b + 1]));
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-                mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-                const int at = h * TP_TOK + g4 + 8 * b;
-                const float old = ms[at], m_new = fmaxf(old, mx), base = m_new == -INFINITY ? 0.f : m_new;
+                for (int b = 0; b < 2; ++b) {
+                    float mx = fmaxf(s[0][2 * b], s[0][2 * b + 1]);
 #pragma unroll
-                for (int n = 0; n < NK; ++n) sum += fast_exp2(s[n][2 * b] - base) + fast_exp2(s[n][2 * b + 1] - base);
-                sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-                sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-                __syncwarp();  // every lane of the quad has read the old maximum
-                if ((lane & 3) == 0) {
-                    ls[at] = ls[at] * fast_exp2(old - base) + sum;
-                    ms[at] = m_new;
+                    for (int n = 1; n < NK; ++n) mx = fmaxf(mx, fmaxf(s[n][2 * b], s[n][2 * b + 1]));
+                    const float m_new = fmaxf(m[i][b], mx), base = m_new == -INFINITY ? 0.f : m_new, off = base * scale_log2;
+                    float sum = l[i][b] * fast_exp2(m[i][b] * scale_log2 - off);
+#pragma unroll
+                    for (int n = 0; n < NK; ++n)
+                        sum += fast_exp2(fmaf(s[n][2 * b], scale_log2, -off)) + fast_exp2(fmaf(s[n][2 * b + 1], scale_log2, -off));
+                    l[i][b] = sum;
+                    m[i][b] = m_new;
                 }
-                __syncwarp();
+            }
+            __syncthreads();  // the stage may be overwritten
+            if (stages == 1 && t + 1 < ntiles) {
+                load_tile(k_stage(t + 1), t + 1, 0);
+                cp_async_commit();
             }
         }
-        __syncthreads();  // the stage may be overwritten
-        if (stages == 1 && t + 1 < ntiles) {
-            load_tile(k_stage(t + 1), t + 1, 0);
-            cp_async_commit();
+#pragma unroll
+        for (int i = 0; i < TP_STATS; ++i) {
+            const int h = h0 + i * TP_WARPS;
+            if (h >= H) continue;
+#pragma unroll
+            for (int b = 0; b < 2; ++b) {
+                float mm = m[i][b], ll = l[i][b];
+#pragma unroll
+                for (int o = 1; o < 4; o <<= 1) {
+                    const float om = __shfl_xor_sync(0xffffffffu, mm, o), ol = __shfl_xor_sync(0xffffffffu, ll, o), mn = fmaxf(mm, om);
+                    const float base = mn == -INFINITY ? 0.f : mn;
+                    ll = ll * fast_exp2((mm - base) * scale_log2) + ol * fast_exp2((om - base) * scale_log2);
+                    mm = mn;
+                }
+                // (a padding row sees nothing: every weight becomes zero)
+                if (tig == 0) lse[h * TP_TOK + g4 + 8 * b] = ll > 0.f ? fmaf(mm, scale_log2, log2f(ll)) : INFINITY;
+            }
         }
-    }
-    for (int i = tid; i < H * TP_TOK; i += TP_THREADS) {
-        ls[i] = ls[i] > 0.f ? 1.f / ls[i] : 0.f;
-        if (ms[i] == -INFINITY) ms[i] = 0.f;  // (a padding row: every weight becomes zero)
     }
     // ---- second walk: weights, mix, values
     const int h_lo = hpart * TP_WARPS * HPW, h_hi = min(H, h_lo + TP_WARPS * HPW);  // the heads whose outputs this block makes
+    const int m0 = h_lo / 16 * 16;                                                 // first head of its tiles of 16
     float o[HPW][DTILES][4];
 #pragma unroll
     for (int i = 0; i < HPW; ++i)
@@ -529,49 +575,58 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
             load_tile(k_stage(t + 1), t + 1, 0);
             cp_async_commit();
         }
+        const int k0 = kbeg + t * KT;
+        const bool whole = whole_tile(k0);
         for (int h = warp; h < H; h += TP_WARPS) {
             float s[NK][4];
-            score(h, t, s);
-            const float m0 = ms[h * TP_TOK + g4], m1 = ms[h * TP_TOK + g4 + 8], l0 = ls[h * TP_TOK + g4], l1 = ls[h * TP_TOK + g4 + 8];
+            score(h, nullptr, k_stage(t), k0, whole, s);
+            const float s0 = lse[h * TP_TOK + g4], s1 = lse[h * TP_TOK + g4 + 8];
+            bf16* dst = pt + (size_t)h * PH + (g4 ^ (h & 7)) * 8 + tig * 2;
 #pragma unroll
             for (int n = 0; n < NK; ++n) {
-                *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, h, n * 16 + g4) + (lane & 3) * 2) =
-                    pack_bf16(fast_exp2(s[n][0] - m0) * l0, fast_exp2(s[n][1] - m0) * l0);
-                *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, h, n * 16 + g4 + 8) + (lane & 3) * 2) =
-                    pack_bf16(fast_exp2(s[n][2] - m1) * l1, fast_exp2(s[n][3] - m1) * l1);
+                *reinterpret_cast<uint32_t*>(dst + n * 128) =
+                    pack_bf16(fast_exp2(fmaf(s[n][0], scale_log2, -s0)), fast_exp2(fmaf(s[n][1], scale_log2, -s0)));
+                *reinterpret_cast<uint32_t*>(dst + n * 128 + 64) =
+                    pack_bf16(fast_exp2(fmaf(s[n][2], scale_log2, -s1)), fast_exp2(fmaf(s[n][3], scale_log2, -s1)));
             }
         }
         __syncthreads();
         // The mix, in place: a warp owns two pieces (16 positions) at a time of all heads, reads them and writes the heads of
-        // its block's one or two tiles of 16 (a padding head's row and column of the mixing weights are zero).
-        for (int pc = warp * 2; pc < TP_TOK * NK; pc += TP_WARPS * 2) {
-            const int m0 = h_lo / 16 * 16;
-            float acc[MT][2][4];
+        // its block's tiles of 16 (a padding head's row and column of the mixing weights are zero).
+        {
+            const int pc = warp * 2;  // a round moves the pieces by whole groups of 8
+            const bf16* src = pt + (size_t)(l7 + (j8 & 1) * 8) * PH + ((pc & ~7) + (((pc + (j8 >> 1)) & 7) ^ l7)) * 8;
+            bf16* dst = pt + (size_t)(m0 + g4) * PH + tig * 2;
+            const bf16* ta = tk + (size_t)(m0 + q_row) * TS + q_col;
 #pragma unroll
-            for (int i = 0; i < MT; ++i)
+            for (int round = 0; round < TP_TOK * NK / (TP_WARPS * 2); ++round) {
+                float acc[MT][2][4];
 #pragma unroll
-                for (int b = 0; b < 2; ++b) acc[i][b][0] = acc[i][b][1] = acc[i][b][2] = acc[i][b][3] = 0.f;
-            for (int g0 = 0; g0 < HP; g0 += 16) {
-                uint32_t b[4];
-                const int j = lane >> 3, g = g0 + (lane & 7) + (j & 1) * 8;
-                ldmatrix_x4_trans(b, tp_piece<KT>(pt, g, pc + (j >> 1)));
+                for (int i = 0; i < MT; ++i)
 #pragma unroll
-                for (int i = 0; i < MT; ++i) {
-                    if (m0 + i * 16 >= h_hi) continue;
-                    uint32_t a[4];
-                    ldmatrix_x4(a, tk + (size_t)(m0 + i * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * TS + g0 + (lane >> 4) * 8);
-                    mma_bf16(acc[i][0], a, b[0], b[1]);
-                    mma_bf16(acc[i][1], a, b[2], b[3]);
+                    for (int b = 0; b < 2; ++b) acc[i][b][0] = acc[i][b][1] = acc[i][b][2] = acc[i][b][3] = 0.f;
+                for (int g0 = 0; g0 < HP; g0 += 16) {
+                    uint32_t b[4];
+                    ldmatrix_x4_trans(b, src + (size_t)g0 * PH + round * TP_WARPS * 16);
+#pragma unroll
+                    for (int i = 0; i < MT; ++i) {
+                        if (m0 + i * 16 >= h_hi) continue;
+                        uint32_t a[4];
+                        ldmatrix_x4(a, ta + i * 16 * TS + g0);
+                        mma_bf16(acc[i][0], a, b[0], b[1]);
+                        mma_bf16(acc[i][1], a, b[2], b[3]);
+                    }
                 }
-            }
-            __syncwarp();  // the warp has read its pieces
-#pragma unroll
-            for (int i = 0; i < MT; ++i) {
-                if (m0 + i * 16 >= h_hi) continue;
+                __syncwarp();  // the warp has read its pieces
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
-                    *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, m0 + i * 16 + g4, pc + b) + (lane & 3) * 2) = pack_bf16(acc[i][b][0], acc[i][b][1]);
-                    *reinterpret_cast<uint32_t*>(tp_piece<KT>(pt, m0 + i * 16 + g4 + 8, pc + b) + (lane & 3) * 2) = pack_bf16(acc[i][b][2], acc[i][b][3]);
+                    bf16* place = dst + ((pc & ~7) + (((pc + b) & 7) ^ g4)) * 8 + round * TP_WARPS * 16;
+#pragma unroll
+                    for (int i = 0; i < MT; ++i) {
+                        if (m0 + i * 16 >= h_hi) continue;
+                        *reinterpret_cast<uint32_t*>(place + i * 16 * PH) = pack_bf16(acc[i][b][0], acc[i][b][1]);
+                        *reinterpret_cast<uint32_t*>(place + (i * 16 + 8) * PH) = pack_bf16(acc[i][b][2], acc[i][b][3]);
+                    }
                 }
             }
         }
@@ -586,16 +641,16 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
         for (int i = 0; i < HPW; ++i) {
             const int h = h_lo + warp + i * TP_WARPS;
             if (h < h_hi) {
-                const bf16* v = vt + (size_t)(h / HG) * KT * LDS;
+                const bf16* v = vt + kv_of[h];
+                const bf16* p = pt + (size_t)h * PH + ((j8 >> 1) * 16 + (l7 ^ (h & 7)) + (j8 & 1) * 8) * 8;
 #pragma unroll
                 for (int ks = 0; ks < NK / 2; ++ks) {
                     uint32_t a[4];
-                    const int j = lane >> 3;
-                    ldmatrix_x4(a, tp_piece<KT>(pt, h, (2 * ks + (j >> 1)) * 16 + (lane & 7) + (j & 1) * 8));
+                    ldmatrix_x4(a, p + ks * 256);
 #pragma unroll
                     for (int dp = 0; dp < DTILES / 2; ++dp) {
                         uint32_t b[4];
-                        ldmatrix_x4_trans(b, v + toff(ks * 16 + (lane & 7) + (j & 1) * 8, dp * 16 + (j >> 1) * 8));
+                        ldmatrix_x4_trans(b, v + toff(ks * 16 + q_row, dp * 16 + q_col));
                         mma_bf16(o[i][2 * dp], a, b[0], b[1]);
                         mma_bf16(o[i][2 * dp + 1], a, b[2], b[3]);
                     }
@@ -614,7 +669,7 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
             bf16* orow = out + ((size_t)(row0 + t0 + tok) * H + h) * D;
 #pragma unroll
             for (int dt = 0; dt < DTILES; ++dt)
-                *reinterpret_cast<__nv_bfloat162*>(orow + dt * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(o[i][dt][2 * b], o[i][dt][2 * b + 1]);
+                *reinterpret_cast<__nv_bfloat162*>(orow + dt * 8 + tig * 2) = __floats2bfloat162_rn(o[i][dt][2 * b], o[i][dt][2 * b + 1]);
         }
     }
 }
@@ -649,7 +704,7 @@ extern "C" int attn_talk_prefill(const void* q, int q_stride, const void* cache,
                                  const int* ctx_lens, void* out, int S, int max_q_len, int nq, int nkv, int page_size, int num_pages,
                                  int chunk, float scale, const float* talk, int max_context, int* status, cudaStream_t stream) {
     if (S <= 0 || max_q_len <= 0) return 0;
-    if (nkv <= 0 || nq % nkv || q_stride % 8 || ((uintptr_t)q & 15)) return (int)cudaErrorInvalidValue;
+    if (nkv <= 0 || nq % nkv || q_stride % 8 || ((uintptr_t)q & 15) || scale <= 0.f) return (int)cudaErrorInvalidValue;
     const int bt_cap = tp_table_slice(chunk, max_context, page_size);
     int KT = 0, stages = 0;
     size_t smem = 0;

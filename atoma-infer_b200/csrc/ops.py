@@ -1021,7 +1021,7 @@ class CudaOps:
                                                      ctx.S, nq, nkv, page_size, num_pages, int(chunk), ctypes.c_float(scale), _p(talk),
                                                      splits, ctx.max_context, _p(self.status), self._stream()), "attn_talk_decode")
                     return
-            elif lib.attn_talk_prefill_supports(nq, nkv, int(chunk), ctx.max_context, page_size):
+            elif scale > 0 and lib.attn_talk_prefill_supports(nq, nkv, int(chunk), ctx.max_context, page_size):
                 self._check(lib.attn_talk_prefill(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.cu_tokens),
                                                   _p(ctx.context_lens), _p(out), ctx.S, ctx.max_tokens_per_entry, nq, nkv, page_size,
                                                   num_pages, int(chunk), ctypes.c_float(scale), _p(talk), ctx.max_context,
