@@ -361,6 +361,100 @@ inline size_t tp_smem(int H, int G, int KT, int stages, int bt_cap) {
 constexpr int TP_STATS = D <= 64 ? 2 : 4;  // heads a warp takes at a time in the first walk
 constexpr bool TP_Q_KEPT = D <= 64;        // ... with their queries' fragments in registers
 
+// Shared memory by 32-bit address: the loops below compute an address per fragment, and generic pointers would cost three
+// times the instructions.
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t a) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], uint32_t a) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void sts_u32(uint32_t a, uint32_t v) { asm volatile("st.shared.b32 [%0], %1;\n" ::"r"(a), "r"(v) : "memory"); }
+__device__ __forceinline__ void cp_async_16_to(uint32_t a, const void* gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(a), "l"(gmem) : "memory");
+}
+// Bytes of (row, col) in a tile (toff in bytes), and the place of the fragment `step` steps of 16 columns behind one at `at`: in
+// swizzled tiles a step of 16 columns is an exclusive or of the two piece bits above the first (a row's pieces of 128 bytes
+// start on 128 bytes), in padded ones an addition.
+__device__ __forceinline__ uint32_t tile_bytes(int row, int col) { return (uint32_t)toff(row, col) * 2u; }
+__device__ __forceinline__ uint32_t step16(uint32_t at, int step) {
+    if constexpr (SWZ) return (at ^ ((uint32_t)(step & 3) << 5)) + (uint32_t)(step >> 2) * 128u;
+    return at + (uint32_t)step * 32u;
+}
+constexpr uint32_t ROW_BYTES = LDS * 2;
+
+// What a lane needs to know of its two rows (g4 and g4 + 8 of the 16 tokens) and of where it reads fragments in a tile.
+struct TalkLane {
+    uint32_t q_at, k_at;  // bytes from the start of a head's queries, of a key tile
+    int tig;
+    int pa, pb, ca, cb;   // the rows' positions (-1: a padding row) and their chunks' starts
+};
+
+// The products of a head's 16 tokens with a tile's keys, unscaled; unless every token sees the tile WHOLE, -inf where a token
+// does not see a key.  KEPT: the queries' fragments come from registers.
+template <bool WHOLE, bool KEPT, int NK>
+__device__ __forceinline__ void talk_scores(float (&s)[NK][4], const TalkLane& w, uint32_t qh, const uint32_t (*qf)[4], uint32_t kh, int k0) {
+#pragma unroll
+    for (int n = 0; n < NK; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+    const uint32_t q_at = qh + w.q_at, k_at = kh + w.k_at;
+#pragma unroll
+    for (int ks = 0; ks < KSTEPS; ++ks) {
+        uint32_t a[4];
+        if constexpr (KEPT) { a[0] = qf[ks][0]; a[1] = qf[ks][1]; a[2] = qf[ks][2]; a[3] = qf[ks][3]; }
+        else ldsm_x4(a, step16(q_at, ks));
+#pragma unroll
+        for (int np = 0; np < NK / 2; ++np) {
+            uint32_t b[4];
+            ldsm_x4(b, step16(k_at, ks) + np * 16 * ROW_BYTES);
+            mma_bf16(s[2 * np], a, b[0], b[1]);
+            mma_bf16(s[2 * np + 1], a, b[2], b[3]);
+        }
+    }
+    if constexpr (!WHOLE) {
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const int key = k0 + n * 8 + w.tig * 2 + (c & 1);
+                const bool sees = c < 2 ? (key <= w.pa) & (key >= w.ca) : (key <= w.pb) & (key >= w.cb);
+                s[n][c] = sees ? s[n][c] : -INFINITY;
+            }
+    }
+}
+
+// First walk, one tile and head: the lane's running maxima and sums over its own columns of its two rows.
+template <bool WHOLE, bool KEPT, int NK>
+__device__ __forceinline__ void talk_stats(float (&m)[2], float (&l)[2], const TalkLane& w, uint32_t qh, const uint32_t (*qf)[4],
+                                           uint32_t kh, int k0, float scale_log2) {
+    float s[NK][4];
+    talk_scores<WHOLE, KEPT, NK>(s, w, qh, qf, kh, k0);
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+        float mx = fmaxf(s[0][2 * b], s[0][2 * b + 1]);
+#pragma unroll
+        for (int n = 1; n < NK; ++n) mx = fmaxf(mx, fmaxf(s[n][2 * b], s[n][2 * b + 1]));
+        const float m_new = fmaxf(m[b], mx), base = m_new == -INFINITY ? 0.f : m_new, off = base * scale_log2;
+        float sum = l[b] * fast_exp2(m[b] * scale_log2 - off);
+#pragma unroll
+        for (int n = 0; n < NK; ++n)
+            sum += fast_exp2(fmaf(s[n][2 * b], scale_log2, -off)) + fast_exp2(fmaf(s[n][2 * b + 1], scale_log2, -off));
+        l[b] = sum;
+        m[b] = m_new;
+    }
+}
+
+// Second walk, one tile and head: the finished weights, to the head's pieces in shared memory.
+template <bool WHOLE, int NK>
+__device__ __forceinline__ void talk_weights(uint32_t dst, const TalkLane& w, uint32_t qh, uint32_t kh, int k0, float scale_log2, float s0, float s1) {
+    float s[NK][4];
+    talk_scores<WHOLE, false, NK>(s, w, qh, nullptr, kh, k0);
+#pragma unroll
+    for (int n = 0; n < NK; ++n) {
+        sts_u32(dst + n * 256, pack_bf16(fast_exp2(fmaf(s[n][0], scale_log2, -s0)), fast_exp2(fmaf(s[n][1], scale_log2, -s0))));
+        sts_u32(dst + n * 256 + 128, pack_bf16(fast_exp2(fmaf(s[n][2], scale_log2, -s1)), fast_exp2(fmaf(s[n][3], scale_log2, -s1))));
+    }
+}
+
 template <int KT, int HPW>
 __global__ void __launch_bounds__(TP_THREADS)
 talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ cache, CacheLayout L, const int* __restrict__ meta,
@@ -368,7 +462,7 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                     int chunk, float scale_log2, const float* __restrict__ talk, int num_pages, int bt_cap, int stages,
                     int* __restrict__ status) {
     constexpr int NK = KT / 8, MT = TP_WARPS * HPW > 16 ? TP_WARPS * HPW / 16 : 1, PH = TP_TOK * KT;  // PH: a head's weights
-    extern __shared__ __align__(16) unsigned char smem_raw[];
+    extern __shared__ __align__(1024) unsigned char smem_raw[];
     const int G = L.num_kv_heads, HG = H / G, HP = (H + 15) / 16 * 16, TS = HP + 8, ps = L.page_size;
     bf16* qt = reinterpret_cast<bf16*>(smem_raw);             // [H][16][LDS]
     bf16* kt = qt + (size_t)H * TP_TOK * LDS;                 // [stages][G][KT][LDS]
@@ -410,13 +504,15 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
         tk[h * TS + g] = __float2bfloat16_rn(h < H && g < H ? talk[(size_t)h * H + g] : 0.f);
     }
     for (int idx = tid; idx < (HP - H) * PH; idx += TP_THREADS) pt[(size_t)H * PH + idx] = __float2bfloat16_rn(0.f);
-    for (int h = tid; h < H; h += TP_THREADS) kv_of[h] = (h / HG) * KT * LDS;
+    for (int h = tid; h < H; h += TP_THREADS) kv_of[h] = (h / HG) * KT * LDS * 2;
+    const uint32_t qt_a = smem_u32(qt), kt_a = smem_u32(kt), vt_a = smem_u32(vt), pt_a = smem_u32(pt), tk_a = smem_u32(tk);
+    const uint32_t kv_bytes = (uint32_t)G * KT * ROW_BYTES;
     // Keys (kv = 0) or values (kv = 1) of a tile for every head; positions outside [kbeg, kend_s) as zeros.  A thread copies
     // 16 dimensions of the same rows of every few heads, so a row's page is looked up once.
     constexpr int PAIRS = D / 16, PP = PAIRS <= 1 ? 1 : PAIRS <= 2 ? 2 : PAIRS <= 4 ? 4 : PAIRS <= 8 ? 8 : 16;
     constexpr int RS = TP_THREADS / PP < KT ? TP_THREADS / PP : KT, CS = TP_THREADS / (PP * RS);
     const int c16 = (tid % PP) * 16, rr0 = (tid / PP) % RS, cc0 = tid / (PP * RS);
-    auto load_tile = [&](bf16* dst, int t, int kv) {
+    auto load_tile = [&](uint32_t dst, int t, int kv) {
         if (c16 >= D) return;
         for (int rr = rr0; rr < KT; rr += RS) {
             const int at = kbeg + t * KT + rr;
@@ -426,60 +522,32 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                 slot = at - pi * ps;
                 page = bt_s[pi - page_lo];
             }
-            bf16 *d0 = dst + (size_t)cc0 * KT * LDS + toff(rr, c16), *d1 = dst + (size_t)cc0 * KT * LDS + toff(rr, c16 + 8);
+            uint32_t d0 = dst + (uint32_t)cc0 * KT * ROW_BYTES + tile_bytes(rr, c16), d1 = dst + (uint32_t)cc0 * KT * ROW_BYTES + tile_bytes(rr, c16 + 8);
             if (page > 0) {
                 const bf16* src = cache + (size_t)page * page_stride + (kv ? v_off : 0) + (size_t)(cc0 * ps + slot) * D + c16;
                 for (int c = cc0; c < G; c += CS) {
-                    cp_async_16(d0, src);
-                    cp_async_16(d1, src + 8);
-                    d0 += CS * KT * LDS, d1 += CS * KT * LDS, src += (size_t)CS * ps * D;
+                    cp_async_16_to(d0, src);
+                    cp_async_16_to(d1, src + 8);
+                    d0 += CS * KT * ROW_BYTES, d1 += CS * KT * ROW_BYTES, src += (size_t)CS * ps * D;
                 }
             } else {
-                const uint4 z = make_uint4(0u, 0u, 0u, 0u);
                 for (int c = cc0; c < G; c += CS) {
-                    *reinterpret_cast<uint4*>(d0) = z;
-                    *reinterpret_cast<uint4*>(d1) = z;
-                    d0 += CS * KT * LDS, d1 += CS * KT * LDS;
+                    asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};\n" ::"r"(d0), "r"(0) : "memory");
+                    asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};\n" ::"r"(d1), "r"(0) : "memory");
+                    d0 += CS * KT * ROW_BYTES, d1 += CS * KT * ROW_BYTES;
                 }
             }
         }
     };
-    auto k_stage = [&](int t) { return kt + (size_t)(stages == 2 ? t & 1 : 0) * G * KT * LDS; };
+    auto k_stage = [&](int t) { return kt_a + (stages == 2 && (t & 1) ? kv_bytes : 0u); };
     const int g4 = lane >> 2, tig = lane & 3, j8 = lane >> 3, l7 = lane & 7;
-    const int pa = g4 < nt ? p_first + g4 : -1, pb = g4 + 8 < nt ? p_first + g4 + 8 : -1;
-    const int ca = chunk > 0 && pa >= 0 ? pa - pa % chunk : 0, cb = chunk > 0 && pb >= 0 ? pb - pb % chunk : 0;
+    TalkLane w;
+    w.tig = tig;
+    const int q_row = l7 + (j8 & 1) * 8, q_col = (j8 >> 1) * 8;
+    w.q_at = tile_bytes(q_row, q_col), w.k_at = tile_bytes(l7 + (j8 >> 1) * 8, (j8 & 1) * 8);
+    w.pa = g4 < nt ? p_first + g4 : -1, w.pb = g4 + 8 < nt ? p_first + g4 + 8 : -1;
+    w.ca = chunk > 0 && w.pa >= 0 ? w.pa - w.pa % chunk : 0, w.cb = chunk > 0 && w.pb >= 0 ? w.pb - w.pb % chunk : 0;
     const int c_last = chunk > 0 ? p_last - p_last % chunk : 0;
-    // where a lane reads its share of a key fragment inside a tile (both halves of a k-step's 16 dimensions lie in one piece
-    // pair, so only the k-step moves it)
-    const int k_row = l7 + (j8 >> 1) * 8, k_col = (j8 & 1) * 8, q_row = l7 + (j8 & 1) * 8, q_col = (j8 >> 1) * 8;
-    // the products of a head's 16 tokens with a tile's keys, unscaled; -inf where a token does not see a key
-    auto score = [&](int h, const uint32_t (*qf)[4], const bf16* keys, int k0, bool whole, float (&s)[NK][4]) {
-        const bf16* qh = qt + (size_t)h * TP_TOK * LDS;
-        const bf16* kh = keys + kv_of[h];
-#pragma unroll
-        for (int n = 0; n < NK; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-#pragma unroll
-        for (int ks = 0; ks < KSTEPS; ++ks) {
-            uint32_t a[4];
-            if (qf) { a[0] = qf[ks][0]; a[1] = qf[ks][1]; a[2] = qf[ks][2]; a[3] = qf[ks][3]; }
-            else ldmatrix_x4(a, qh + toff(q_row, ks * 16 + q_col));
-#pragma unroll
-            for (int np = 0; np < NK / 2; ++np) {
-                uint32_t b[4];
-                ldmatrix_x4(b, kh + toff(np * 16 + k_row, ks * 16 + k_col));
-                mma_bf16(s[2 * np], a, b[0], b[1]);
-                mma_bf16(s[2 * np + 1], a, b[2], b[3]);
-            }
-        }
-        if (whole) return;
-#pragma unroll
-        for (int n = 0; n < NK; ++n)
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                const int key = k0 + n * 8 + tig * 2 + (c & 1);
-                if (!(c < 2 ? key <= pa && key >= ca : key <= pb && key >= cb)) s[n][c] = -INFINITY;
-            }
-    };
     // a tile that every token sees whole
     auto whole_tile = [&](int k0) { return nt == TP_TOK && k0 + KT - 1 <= p_first && k0 >= c_last; };
     __syncthreads();  // the table slice is written
@@ -495,7 +563,7 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
             for (int i = 0; i < TP_STATS; ++i)
 #pragma unroll
                 for (int ks = 0; ks < KSTEPS; ++ks)
-                    ldmatrix_x4(qf[i][ks], qt + (size_t)min(h0 + i * TP_WARPS, H - 1) * TP_TOK * LDS + toff(q_row, ks * 16 + q_col));
+                    ldsm_x4(qf[i][ks], step16(qt_a + (uint32_t)min(h0 + i * TP_WARPS, H - 1) * TP_TOK * ROW_BYTES + w.q_at, ks));
         }
         load_tile(k_stage(0), 0, 0);
         cp_async_commit();
@@ -509,25 +577,18 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
             }
             __syncthreads();
             const int k0 = kbeg + t * KT;
-            const bool whole = whole_tile(k0);
+            const uint32_t keys = k_stage(t);
+            if (whole_tile(k0)) {
 #pragma unroll
-            for (int i = 0; i < TP_STATS; ++i) {
-                const int h = h0 + i * TP_WARPS;
-                if (h >= H) continue;
-                float s[NK][4];
-                score(h, TP_Q_KEPT ? qf[i] : nullptr, k_stage(t), k0, whole, s);
+                for (int i = 0; i < TP_STATS; ++i) {
+                    const int h = h0 + i * TP_WARPS;
+                    if (h < H) talk_stats<true, TP_Q_KEPT, NK>(m[i], l[i], w, qt_a + (uint32_t)h * TP_TOK * ROW_BYTES, qf[i], keys + kv_of[h], k0, scale_log2);
+                }
+            } else {
 #pragma unroll
-                for (int b = 0; b < 2; ++b) {
-                    float mx = fmaxf(s[0][2 * b], s[0][2 * b + 1]);
-#pragma unroll
-                    for (int n = 1; n < NK; ++n) mx = fmaxf(mx, fmaxf(s[n][2 * b], s[n][2 * b + 1]));
-                    const float m_new = fmaxf(m[i][b], mx), base = m_new == -INFINITY ? 0.f : m_new, off = base * scale_log2;
-                    float sum = l[i][b] * fast_exp2(m[i][b] * scale_log2 - off);
-#pragma unroll
-                    for (int n = 0; n < NK; ++n)
-                        sum += fast_exp2(fmaf(s[n][2 * b], scale_log2, -off)) + fast_exp2(fmaf(s[n][2 * b + 1], scale_log2, -off));
-                    l[i][b] = sum;
-                    m[i][b] = m_new;
+                for (int i = 0; i < TP_STATS; ++i) {
+                    const int h = h0 + i * TP_WARPS;
+                    if (h < H) talk_stats<false, TP_Q_KEPT, NK>(m[i], l[i], w, qt_a + (uint32_t)h * TP_TOK * ROW_BYTES, qf[i], keys + kv_of[h], k0, scale_log2);
                 }
             }
             __syncthreads();  // the stage may be overwritten
@@ -568,7 +629,7 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
     for (int t = 0; t < ntiles; ++t) {
         cp_async_wait<0>();
         __syncthreads();  // keys of the tile are there; values and weights of the tile before are no longer read
-        load_tile(vt, t, 1);
+        load_tile(vt_a, t, 1);
         cp_async_commit();
         const bool ahead = stages == 2 && t + 1 < ntiles;
         if (ahead) {
@@ -576,28 +637,22 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
             cp_async_commit();
         }
         const int k0 = kbeg + t * KT;
+        const uint32_t keys = k_stage(t);
         const bool whole = whole_tile(k0);
         for (int h = warp; h < H; h += TP_WARPS) {
-            float s[NK][4];
-            score(h, nullptr, k_stage(t), k0, whole, s);
             const float s0 = lse[h * TP_TOK + g4], s1 = lse[h * TP_TOK + g4 + 8];
-            bf16* dst = pt + (size_t)h * PH + (g4 ^ (h & 7)) * 8 + tig * 2;
-#pragma unroll
-            for (int n = 0; n < NK; ++n) {
-                *reinterpret_cast<uint32_t*>(dst + n * 128) =
-                    pack_bf16(fast_exp2(fmaf(s[n][0], scale_log2, -s0)), fast_exp2(fmaf(s[n][1], scale_log2, -s0)));
-                *reinterpret_cast<uint32_t*>(dst + n * 128 + 64) =
-                    pack_bf16(fast_exp2(fmaf(s[n][2], scale_log2, -s1)), fast_exp2(fmaf(s[n][3], scale_log2, -s1)));
-            }
+            const uint32_t dst = pt_a + (uint32_t)(h * PH + (g4 ^ (h & 7)) * 8 + tig * 2) * 2u;
+            if (whole) talk_weights<true, NK>(dst, w, qt_a + (uint32_t)h * TP_TOK * ROW_BYTES, keys + kv_of[h], k0, scale_log2, s0, s1);
+            else talk_weights<false, NK>(dst, w, qt_a + (uint32_t)h * TP_TOK * ROW_BYTES, keys + kv_of[h], k0, scale_log2, s0, s1);
         }
         __syncthreads();
         // The mix, in place: a warp owns two pieces (16 positions) at a time of all heads, reads them and writes the heads of
         // its block's tiles of 16 (a padding head's row and column of the mixing weights are zero).
         {
             const int pc = warp * 2;  // a round moves the pieces by whole groups of 8
-            const bf16* src = pt + (size_t)(l7 + (j8 & 1) * 8) * PH + ((pc & ~7) + (((pc + (j8 >> 1)) & 7) ^ l7)) * 8;
-            bf16* dst = pt + (size_t)(m0 + g4) * PH + tig * 2;
-            const bf16* ta = tk + (size_t)(m0 + q_row) * TS + q_col;
+            const uint32_t src = pt_a + (uint32_t)((l7 + (j8 & 1) * 8) * PH + ((pc & ~7) + (((pc + (j8 >> 1)) & 7) ^ l7)) * 8) * 2u;
+            const uint32_t dst = pt_a + (uint32_t)((m0 + g4) * PH + tig * 2) * 2u;
+            const uint32_t ta = tk_a + (uint32_t)((m0 + q_row) * TS + q_col) * 2u;
 #pragma unroll
             for (int round = 0; round < TP_TOK * NK / (TP_WARPS * 2); ++round) {
                 float acc[MT][2][4];
@@ -607,12 +662,12 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                     for (int b = 0; b < 2; ++b) acc[i][b][0] = acc[i][b][1] = acc[i][b][2] = acc[i][b][3] = 0.f;
                 for (int g0 = 0; g0 < HP; g0 += 16) {
                     uint32_t b[4];
-                    ldmatrix_x4_trans(b, src + (size_t)g0 * PH + round * TP_WARPS * 16);
+                    ldsm_x4_trans(b, src + (uint32_t)g0 * PH * 2u + round * TP_WARPS * 32);
 #pragma unroll
                     for (int i = 0; i < MT; ++i) {
                         if (m0 + i * 16 >= h_hi) continue;
                         uint32_t a[4];
-                        ldmatrix_x4(a, ta + i * 16 * TS + g0);
+                        ldsm_x4(a, ta + (uint32_t)(i * 16 * TS + g0) * 2u);
                         mma_bf16(acc[i][0], a, b[0], b[1]);
                         mma_bf16(acc[i][1], a, b[2], b[3]);
                     }
@@ -620,12 +675,12 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                 __syncwarp();  // the warp has read its pieces
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
-                    bf16* place = dst + ((pc & ~7) + (((pc + b) & 7) ^ g4)) * 8 + round * TP_WARPS * 16;
+                    const uint32_t place = dst + (uint32_t)((pc & ~7) + (((pc + b) & 7) ^ g4)) * 16u + round * TP_WARPS * 32;
 #pragma unroll
                     for (int i = 0; i < MT; ++i) {
                         if (m0 + i * 16 >= h_hi) continue;
-                        *reinterpret_cast<uint32_t*>(place + i * 16 * PH) = pack_bf16(acc[i][b][0], acc[i][b][1]);
-                        *reinterpret_cast<uint32_t*>(place + (i * 16 + 8) * PH) = pack_bf16(acc[i][b][2], acc[i][b][3]);
+                        sts_u32(place + i * 16 * PH * 2, pack_bf16(acc[i][b][0], acc[i][b][1]));
+                        sts_u32(place + (i * 16 + 8) * PH * 2, pack_bf16(acc[i][b][2], acc[i][b][3]));
                     }
                 }
             }
@@ -641,16 +696,16 @@ talk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
         for (int i = 0; i < HPW; ++i) {
             const int h = h_lo + warp + i * TP_WARPS;
             if (h < h_hi) {
-                const bf16* v = vt + kv_of[h];
-                const bf16* p = pt + (size_t)h * PH + ((j8 >> 1) * 16 + (l7 ^ (h & 7)) + (j8 & 1) * 8) * 8;
+                const uint32_t v = vt_a + kv_of[h] + w.q_at;
+                const uint32_t p = pt_a + (uint32_t)(h * PH + ((j8 >> 1) * 16 + (l7 ^ (h & 7)) + (j8 & 1) * 8) * 8) * 2u;
 #pragma unroll
                 for (int ks = 0; ks < NK / 2; ++ks) {
                     uint32_t a[4];
-                    ldmatrix_x4(a, p + ks * 256);
+                    ldsm_x4(a, p + ks * 512);
 #pragma unroll
                     for (int dp = 0; dp < DTILES / 2; ++dp) {
                         uint32_t b[4];
-                        ldmatrix_x4_trans(b, v + toff(ks * 16 + q_row, dp * 16 + q_col));
+                        ldsm_x4_trans(b, step16(v, dp) + ks * 16 * ROW_BYTES);
                         mma_bf16(o[i][2 * dp], a, b[0], b[1]);
                         mma_bf16(o[i][2 * dp + 1], a, b[2], b[3]);
                     }
