@@ -135,7 +135,7 @@ def host_library() -> ctypes.CDLL:
 
 def all_kernel_libraries():
     """(name, sources, defines) of every kernel library, for the build check."""
-    from .ops import (ATTENTION_HEAD_DIMS, ATTENTION_SOURCES, ATTENTION_TALK_SOURCES, ATTENTION_TC_HEAD_DIMS, ATTENTION_TC_SOURCES, CORE_SOURCES,
+    from .ops import (ATTENTION_HEAD_DIMS, ATTENTION_SOURCES, ATTENTION_TALK_SOURCES, ATTENTION_TALK_TC_SOURCES, ATTENTION_TC_HEAD_DIMS, ATTENTION_TC_SOURCES, CORE_SOURCES,
                       DECODE_STACK_SOURCES, GEMM_SOURCES, MATRIX_RECURRENT_SOURCES, MIXER_SOURCES, RECURRENT_SOURCES)
 
     return [("core", CORE_SOURCES, None), ("mixers", MIXER_SOURCES, None), ("recurrent", RECURRENT_SOURCES, None),
@@ -144,5 +144,6 @@ def all_kernel_libraries():
         (f"attention_d{d}", ATTENTION_SOURCES, {"HEAD_DIM": d}) for d in ATTENTION_HEAD_DIMS] + [
         (f"attention_talk_d{d}", ATTENTION_TALK_SOURCES, {"HEAD_DIM": d}) for d in ATTENTION_HEAD_DIMS] + [
         (f"attention_noalloc_d{d}", ["kernels/attention_noalloc.cu"], {"HEAD_DIM": d}) for d in (64, 128)] + [
+        (f"attention_talk_tc_d{d}", ATTENTION_TALK_TC_SOURCES, {"HEAD_DIM": d}) for d in ATTENTION_TC_HEAD_DIMS] + [
         (f"attention_tc_d{d}", ATTENTION_TC_SOURCES, {"HEAD_DIM": d}) for d in ATTENTION_TC_HEAD_DIMS] + [
         (f"decode_stack_d{d}", DECODE_STACK_SOURCES, {"HEAD_DIM": d}) for d in (64, 128)]

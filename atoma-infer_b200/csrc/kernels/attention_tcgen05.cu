@@ -26,26 +26,15 @@
 //
 // All barrier waits are bounded; on a timeout the block raises a status word, every warp leaves its
 // loop, and the block frees its tensor memory and returns.
-#include <cuda.h>
-
-#include "common.cuh"
-
-#ifndef HEAD_DIM
-#define HEAD_DIM 64
-#endif
-static_assert(HEAD_DIM == 64 || HEAD_DIM == 128, "the tcgen05 attention kernel is built for head sizes 64 and 128");
+#include "attention_tc.cuh"
 
 int g_use_pdl = 0;
 extern "C" void kernels_set_pdl(int mode) { g_use_pdl = mode; }
 
 namespace {
 
-typedef __nv_bfloat16 bf16;
-constexpr int D = HEAD_DIM;
 constexpr int BQ = 128;            // query rows per block
 constexpr int BKV = 128;           // keys per tile
-constexpr int HALVES = D / 64;     // 64-column (128-byte) halves of a head
-constexpr int HALF_BYTES = 128 * 128;  // a [128 rows x 64 columns] bfloat16 sub-tile
 // Tensor memory of a block: the scores S of one tile (128 columns of float32), P (the tile's 128 keys as packed
 // bfloat16, 64 columns) and the output accumulator O (head size columns of float32), which stays there for the whole
 // key loop: P V of every tile is added to it by the tensor core itself.
@@ -57,137 +46,18 @@ constexpr float RESCALE_STEP = 8.f;
 constexpr int SOFTMAX_THREADS = 256, SOFTMAX_WARPS = 8;
 constexpr int COPY_WARP = 8, MMA_WARP = 9;
 constexpr int TC_THREADS = 384;  // three warpgroups: two of softmax warps, one with the copy and the MMA warp
-constexpr uint32_t WAIT_LIMIT = 1u << 22;
-constexpr float LOG2E = 1.4426950408889634f;
-#define STATUS_ATTN_TIMEOUT 3
-
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void mbar_init(uint64_t* bar, uint32_t count) {
-    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count));
-}
-__device__ __forceinline__ void mbar_expect_tx(uint64_t* bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(bar)), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ bool mbar_try_wait(uint64_t* bar, uint32_t parity) {
-    uint32_t ok;
-    asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-                 : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
-    return ok != 0;
-}
-__device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, int* status, volatile int* abort_flag) {
-    for (uint32_t i = 0; i < WAIT_LIMIT; ++i) {
-        if (mbar_try_wait(bar, parity)) return true;
-        if (*abort_flag) return false;
-    }
-    *abort_flag = 1;
-    atomicExch(&status[STATUS_ATTN_TIMEOUT], 1 + (int)blockIdx.y);
-    return false;
-}
-__device__ __forceinline__ void tma_load_2d(void* smem_dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-                 ::"r"(smem_u32(smem_dst)), "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-__device__ __forceinline__ void tmem_alloc(uint32_t* smem_result, uint32_t ncols) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(smem_result)), "r"(ncols));
-}
-__device__ __forceinline__ void tmem_relinquish() { asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;"); }
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t ncols) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols));
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void umma_commit(uint64_t* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-                 ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
-}
-// 32 columns of this thread's lane, written from 32 registers (used for P: two bfloat16 keys a column)
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,"
-                 "%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
-                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
-                   "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
-                   "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
-                   "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-                 : "memory");
-    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-}
-// D (tensor memory) = A (tensor memory: row = lane, two bfloat16 of K per column) * B (shared memory)
-__device__ __forceinline__ void umma_bf16_a_tmem(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
-                                                 uint32_t accumulate) {
-    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-                 ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-// Registers move between warpgroups: the copy/MMA warpgroup gives up what the softmax warpgroups take.
-template <int N> __device__ __forceinline__ void regs_release() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
-template <int N> __device__ __forceinline__ void regs_take() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
-    uint32_t r[32];
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n\ttcgen05.wait::ld.sync.aligned;"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-                 : "r"(taddr) : "memory");
-#pragma unroll
-    for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-}
-// 64 columns in two loads of 32 and one wait
-__device__ __forceinline__ void tmem_ld32x2(uint32_t taddr, float (&v)[64]) {
-    uint32_t r[64];
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%64];\n\t"
-                 "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%32,%33,%34,%35,%36,%37,%38,%39,%40,%41,%42,%43,%44,%45,%46,%47,%48,%49,%50,%51,%52,%53,%54,%55,%56,%57,%58,%59,%60,%61,%62,%63}, [%65];\n\t"
-                 "tcgen05.wait::ld.sync.aligned;"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31]), "=r"(r[32]), "=r"(r[33]), "=r"(r[34]), "=r"(r[35]), "=r"(r[36]), "=r"(r[37]), "=r"(r[38]), "=r"(r[39]), "=r"(r[40]), "=r"(r[41]), "=r"(r[42]), "=r"(r[43]), "=r"(r[44]), "=r"(r[45]), "=r"(r[46]), "=r"(r[47]), "=r"(r[48]), "=r"(r[49]), "=r"(r[50]), "=r"(r[51]), "=r"(r[52]), "=r"(r[53]), "=r"(r[54]), "=r"(r[55]), "=r"(r[56]), "=r"(r[57]), "=r"(r[58]), "=r"(r[59]), "=r"(r[60]), "=r"(r[61]), "=r"(r[62]), "=r"(r[63])
-                 : "r"(taddr), "r"(taddr + 32) : "memory");
-#pragma unroll
-    for (int i = 0; i < 64; ++i) v[i] = __uint_as_float(r[i]);
-}
-// 32 columns of this thread's lane, written from 32 float registers
-__device__ __forceinline__ void tmem_st32f(uint32_t taddr, const float (&v)[32]) {
-    uint32_t r[32];
-#pragma unroll
-    for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(v[i]);
-    tmem_st32(taddr, r);
-}
-__device__ __forceinline__ float fast_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
-// Descriptors of 128-byte-swizzled tiles whose rows are 128 bytes (64 bfloat16) and whose 8-row groups
-// are 1024 bytes apart.  K-major: the 64 contiguous elements run along the MMA's K.  MN-major: they run
-// along M or N, rows are K; `lbo` is then the distance between 64-wide halves.
-__device__ __forceinline__ uint64_t make_desc(uint32_t smem_addr, uint32_t lbo_bytes) {
-    uint64_t d = (uint64_t)((smem_addr & 0x3FFFF) >> 4);
-    d |= (uint64_t)((lbo_bytes >> 4) & 0x3FFF) << 16;
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;
-    return d;
-}
-// kind::f16 instruction descriptor: float32 accumulator, bfloat16 operands, A K-major, B K- or MN-major.
-__host__ __device__ constexpr uint32_t make_idesc(int m, int n, bool b_mn_major) {
-    return (1u << 4) | (1u << 7) | (1u << 10) | ((b_mn_major ? 1u : 0u) << 16) | ((uint32_t)(n >> 3) << 17) |
-           ((uint32_t)(m >> 4) << 24);
-}
-// byte offset of (row, 16-byte chunk c of a 64-column half) in a swizzled [rows x 64] sub-tile
-__device__ __forceinline__ uint32_t swz(int row, int c) { return (uint32_t)row * 128u + (uint32_t)((c ^ (row & 7)) << 4); }
 
 }  // namespace
 
-// CS: the instantiation that knows chunk masks and the softmax's sink (the plain one keeps its registers)
-template <bool CS>
+// CS: the instantiation that knows chunk masks and the softmax's sink (the plain one keeps its registers).  STATS: only the base-2
+// logarithm of every row's sum of exponentials is wanted (`lse` [rows, nq]); values are neither copied nor weighed.
+template <bool CS, bool STATS = false>
 __global__ void __launch_bounds__(TC_THREADS, HEAD_DIM == 64 ? 2 : 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* __restrict__ q, int q_stride,
                        CacheLayout L, const int* __restrict__ meta, int group, const int* __restrict__ cu_tokens,
                        const int* __restrict__ ctx_lens, bf16* __restrict__ out, int nq, int window, int chunk_arg, int sink_arg,
                        const float* __restrict__ sink_values, float scale_log2, int num_pages, int bt_cap,
-                       float softcap_arg, const float* __restrict__ slopes_arg, int* __restrict__ status) {
+                       float softcap_arg, const float* __restrict__ slopes_arg, int* __restrict__ status, float* __restrict__ lse) {
     const int chunk = CS ? chunk_arg : 0, sink = CS ? sink_arg : 0;
     // capped scores (s <- softcap * tanh(s / softcap)) and a bias by distance (slopes[h] * (query position - key position)
     // taken off): the scores are then turned into their final form, in base 2, before the maximum is taken
@@ -300,7 +170,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
             };
             int last_k[2] = {-1, -1}, last_v[2] = {-1, -1};  // the last tile whose copy was started into a stage
             for (int t = 0; t < 2 && t < ntiles; ++t) { issue_loads(t, 0, k_s + t * STAGE, &k_full[t]); last_k[t] = t; }
-            for (int t = 0; t < 2 && t < ntiles; ++t) { issue_loads(t, 1, v_s + t * STAGE, &v_full[t]); last_v[t] = t; }
+            for (int t = 0; !STATS && t < 2 && t < ntiles; ++t) { issue_loads(t, 1, v_s + t * STAGE, &v_full[t]); last_v[t] = t; }
             bool ok = true;
             for (int t = 0; t + 2 < ntiles; ++t) {
                 const int b = t & 1;
@@ -309,6 +179,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
                 if (!ok) break;
                 issue_loads(t + 2, 0, k_s + b * STAGE, &k_full[b]);
                 last_k[b] = t + 2;
+                if constexpr (STATS) continue;
                 ok = mbar_wait(&pv_done[b], par, status, abort_flag);  // P V of tile t is done: its V stage is free
                 if (!ok) break;
                 issue_loads(t + 2, 1, v_s + b * STAGE, &v_full[b]);
@@ -351,6 +222,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
                     issue_scores(t + 1);
                     if (!ok) break;
                 }
+                if constexpr (STATS) continue;
                 ok = mbar_wait(p_ready, (uint32_t)t & 1u, status, abort_flag);  // P(t) is in tensor memory, O is scaled
                 if (!ok) break;
                 ok = mbar_wait(&v_full[b], par, status, abort_flag);
@@ -451,7 +323,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
             }
             l_run = l_run * corr + (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]);
             // ---- the product of the tile before must be complete before P is overwritten and before O is touched
-            if (t >= 1) {
+            if (!STATS && t >= 1) {
                 if (!mbar_wait(&pv_done[b ^ 1], (uint32_t)((t - 1) >> 1) & 1u, status, abort_flag)) ok = false;
                 tc_fence_after();
                 // O (my half of the row) times the correction, if any row of this warp moved its base
@@ -467,6 +339,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
                     }
                 }
             }
+            if constexpr (STATS) continue;
             tmem_st32(tmem_row + P_COL + half * 32, pk);
 
             // ---- V rows that no page delivered, or that lie beyond the last key, must be zero (0 * NaN would
@@ -488,7 +361,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
             __syncwarp();
             if (lane == 0) mbar_arrive(p_ready);
         }
-        if (ntiles > 0) {
+        if (!STATS && ntiles > 0) {
             if (!mbar_wait(&pv_done[(ntiles - 1) & 1], (uint32_t)((ntiles - 1) >> 1) & 1u, status, abort_flag)) ok = false;
             tc_fence_after();
         }
@@ -500,9 +373,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
         asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp & 3)) : "memory");
         const float l_all = slot[row] + slot[BQ + row];
         const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+        if constexpr (STATS) {
+            if (half == 0 && my_valid && ok) lse[(size_t)(row0 + t0 + my_tok) * nq + kvh * G + my_hd] = m_base + log2f(l_all);
+        }
         bf16* dst = out + ((size_t)(row0 + t0 + my_tok) * nq + kvh * G + my_hd) * D + half * DH;
 #pragma unroll
-        for (int ch = 0; ch < DH / 32; ++ch) {
+        for (int ch = 0; ch < (STATS ? 0 : DH / 32); ++ch) {
             float o[32];
             if (ntiles > 0) tmem_ld32(tmem_row + O_COL + half * DH + ch * 32, o);  // warp-wide: every lane takes part
             if (ok && my_valid) {
@@ -526,20 +402,6 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16* _
 
 // ----------------------------------------------------------------------------- host side
 namespace {
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-EncodeTiledFn encode_fn() {
-    static EncodeTiledFn fn = nullptr;
-    if (!fn) {
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &qres) == cudaSuccess &&
-            qres == cudaDriverEntryPointSuccess)
-            fn = reinterpret_cast<EncodeTiledFn>(p);
-    }
-    return fn;
-}
 constexpr size_t TC_SMEM_FIXED = (size_t)(5 * HALVES) * HALF_BYTES + 12 * 8 + 16 + 4 * BQ * 4 + 1024;  // Q, 2 K, 2 V; barriers; slots; alignment
 }  // namespace
 
@@ -575,18 +437,8 @@ extern "C" int attn_prefill_tc_scores(const void* q, int q_stride, const void* c
                                       int* status, cudaStream_t stream) {
     if (S <= 0 || max_q_len <= 0) return 0;
     if (!attn_prefill_tc_supports(page_size, nq, nkv)) return (int)cudaErrorInvalidValue;
-    EncodeTiledFn fn = encode_fn();
-    if (!fn) return (int)cudaErrorNotSupported;
-    // the layer's cache as a matrix: one row per (page, K|V, head, slot), HEAD_DIM columns
     CUtensorMap map;
-    cuuint64_t dims[2] = {(cuuint64_t)D, (cuuint64_t)num_pages * 2 * nkv * page_size};
-    cuuint64_t strides[1] = {(cuuint64_t)D * 2};
-    cuuint32_t box[2] = {64, (cuuint32_t)page_size};
-    cuuint32_t estr[2] = {1, 1};
-    if (fn(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(cache), dims, strides, box, estr,
-           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-        return (int)cudaErrorInvalidValue;
+    if (!cache_map(&map, cache, num_pages, nkv, page_size)) return (int)cudaErrorNotSupported;
     CacheLayout L{nkv, page_size, D};
     const int tpt = BQ / (nq / nkv);
     int span = window > 0 ? min(max_context, window + tpt + 2 * BKV) : max_context;
@@ -606,11 +458,38 @@ extern "C" int attn_prefill_tc_scores(const void* q, int q_stride, const void* c
     if (cs)
         attn_prefill_tc_kernel<true><<<grid, TC_THREADS, smem, stream>>>(map, (const bf16*)q, q_stride, L, meta, group, cu_tokens,
                                                                   ctx_lens, (bf16*)out, nq, window, chunk, sink, sink_values,
-                                                                  scale * LOG2E, num_pages, bt_cap, softcap, slopes, status);
+                                                                  scale * LOG2E, num_pages, bt_cap, softcap, slopes, status, nullptr);
     else
         attn_prefill_tc_kernel<false><<<grid, TC_THREADS, smem, stream>>>(map, (const bf16*)q, q_stride, L, meta, group, cu_tokens,
                                                                    ctx_lens, (bf16*)out, nq, window, 0, 0, nullptr, scale * LOG2E,
-                                                                   num_pages, bt_cap, 0.f, nullptr, status);
+                                                                   num_pages, bt_cap, 0.f, nullptr, status, nullptr);
+    LAUNCH_RETURN();
+}
+
+// lse[row, h] (float32, base 2) = log2 of the sum over the keys that query head h of the row sees of exp(score); chunk as above.
+// For kernels that need the finished softmax of every head before they weigh values.
+extern "C" int attn_prefill_tc_stats(const void* q, int q_stride, const void* cache, const int* meta, int group, const int* cu_tokens,
+                                     const int* ctx_lens, float* lse, int S, int max_q_len, int nq, int nkv, int page_size, int num_pages,
+                                     int chunk, float scale, int max_context, int* status, cudaStream_t stream) {
+    if (S <= 0 || max_q_len <= 0) return 0;
+    if (!attn_prefill_tc_supports(page_size, nq, nkv) || scale <= 0.f) return (int)cudaErrorInvalidValue;
+    CUtensorMap map;
+    if (!cache_map(&map, cache, num_pages, nkv, page_size)) return (int)cudaErrorNotSupported;
+    CacheLayout L{nkv, page_size, D};
+    const int tpt = BQ / (nq / nkv);
+    const int span = chunk > 0 ? min(max_context, chunk + tpt + 2 * BKV) : max_context;
+    const int bt_cap = span / page_size + 2 + BKV / page_size;
+    const size_t smem = TC_SMEM_FIXED + (size_t)bt_cap * sizeof(int);
+    if (smem > 227 * 1024) return (int)cudaErrorInvalidValue;
+    static size_t configured = 0;
+    if (smem > configured) {
+        cudaError_t err = cudaFuncSetAttribute(attn_prefill_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (err != cudaSuccess) return (int)err;
+        configured = smem;
+    }
+    attn_prefill_tc_kernel<true, true><<<dim3(nkv, (max_q_len + tpt - 1) / tpt, S), TC_THREADS, smem, stream>>>(
+        map, (const bf16*)q, q_stride, L, meta, group, cu_tokens, ctx_lens, nullptr, nq, 0, chunk, 0, nullptr, scale * LOG2E, num_pages,
+        bt_cap, 0.f, nullptr, status, lse);
     LAUNCH_RETURN();
 }
 

@@ -30,6 +30,7 @@ GEMM_SOURCES = ["kernels/gemm_tcgen05.cu"]
 ATTENTION_TC_SOURCES = ["kernels/attention_tcgen05.cu"]
 DECODE_STACK_SOURCES = ["kernels/decode_stack.cu"]
 ATTENTION_TALK_SOURCES = ["kernels/attention_talk.cu"]  # weights mixed across heads; one library per head size
+ATTENTION_TALK_TC_SOURCES = ["kernels/attention_talk_tcgen05.cu"]  # the same for prompts, head sizes 64 and 128
 # parallel blocks, state-space mixers, latent attention, routed experts: built when a model first uses one of them
 MIXER_SOURCES = ["kernels/stream_ops.cu", "kernels/ssm.cu", "kernels/latent.cu", "kernels/moe.cu", "kernels/gated_stream.cu",
                  "kernels/normed_stream.cu", "kernels/talking_heads.cu"]
@@ -69,7 +70,7 @@ class CudaOps:
         self.launches = 0  # own kernel launches, counted for the benchmark record
         self._attn_libs = {}
         self._attn_tc_libs = {}
-        self._talk_libs = {}
+        self._talk_libs, self._talk_tc_libs = {}, {}
         self.fast_talking_attention = True  # tensor-core kernels for weights mixed across heads (False: the plain one; a test lever)
         # levers for the kernel tests (each kernel is compared with the one it stands in for)
         self.tc_attention = True    # tcgen05 prefill attention where the geometry allows
@@ -1021,6 +1022,8 @@ class CudaOps:
                                                      ctx.S, nq, nkv, page_size, num_pages, int(chunk), ctypes.c_float(scale), _p(talk),
                                                      splits, ctx.max_context, _p(self.status), self._stream()), "attn_talk_decode")
                     return
+            elif self._talk_prefill_tc(q, q_stride, cache_layer, ctx, group, out, nq, nkv, d, page_size, num_pages, scale, talk, int(chunk)):
+                return
             elif scale > 0 and lib.attn_talk_prefill_supports(nq, nkv, int(chunk), ctx.max_context, page_size):
                 self._check(lib.attn_talk_prefill(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.cu_tokens),
                                                   _p(ctx.context_lens), _p(out), ctx.S, ctx.max_tokens_per_entry, nq, nkv, page_size,
@@ -1030,6 +1033,35 @@ class CudaOps:
         self._check(self._mixers().talk_attn_plain(_p(q), q_stride, _p(cache_layer), _code(q), _p(ctx.meta), group, _p(ctx.token_entry),
                                                    _p(ctx.positions), _p(out), ctx.T, nq, nkv, d, page_size, num_pages, int(chunk),
                                                    ctypes.c_float(scale), _p(talk), _p(self.status), self._stream()), "talk_attn_plain")
+
+    TALK_TC_FROM = 64  # tokens of the step's longest entry from which on a prompt runs on the tcgen05 kernels (a test lever too)
+
+    def _talk_prefill_tc(self, q, q_stride, cache_layer, ctx, group, out, nq, nkv, d, page_size, num_pages, scale, talk, chunk) -> bool:
+        """Prompts with head size 64 or 128 and up to 32 head slots: one kernel leaves every row's logarithm of its sum of
+        exponentials, the other finishes, mixes and weighs.  False: not this geometry, nothing has run."""
+        if d not in ATTENTION_TC_HEAD_DIMS or ctx.max_tokens_per_entry < self.TALK_TC_FROM or scale <= 0:
+            return False
+        stats = self._prefill_tc(d, page_size, nq, nkv)
+        if stats is None:
+            return False
+        lib = self._talk_tc_libs.get(d)
+        if lib is None:
+            lib = self._talk_tc_libs[d] = build.load_library(f"attention_talk_tc_d{d}", ATTENTION_TALK_TC_SOURCES, cuda=True,
+                                                             defines={"HEAD_DIM": d})
+            if lib.attn_talk_tc_head_dim() != d:
+                raise KernelError(f"tcgen05 attention library was built for head size {lib.attn_talk_tc_head_dim()}, wanted {d}")
+        if not lib.attn_talk_prefill_tc_supports(nq, nkv, chunk, ctx.max_context, page_size):
+            return False
+        lse = torch.empty((ctx.T, nq), dtype=torch.float32, device=q.device)
+        self._check(stats.attn_prefill_tc_stats(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.cu_tokens),
+                                                _p(ctx.context_lens), _p(lse), ctx.S, ctx.max_tokens_per_entry, nq, nkv, page_size,
+                                                num_pages, chunk, ctypes.c_float(scale), ctx.max_context, _p(self.status), self._stream()),
+                    "attn_prefill_tc_stats")
+        self._check(lib.attn_talk_prefill_tc(_p(q), q_stride, _p(cache_layer), _p(ctx.meta), group, _p(ctx.cu_tokens), _p(ctx.context_lens),
+                                             _p(lse), _p(out), ctx.S, ctx.max_tokens_per_entry, nq, nkv, page_size, num_pages, chunk,
+                                             ctypes.c_float(scale), _p(talk), ctx.max_context, _p(self.status), self._stream()),
+                    "attn_talk_prefill_tc")
+        return True
 
     def _talk_library(self, d: int):
         lib = self._talk_libs.get(d)

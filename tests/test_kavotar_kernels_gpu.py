@@ -116,12 +116,13 @@ def test_weights_mixed_across_heads(rts, dtype, H, G, d, dv, page, chunk):
             rt.ops.fast_talking_attention = True
 
 
-@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("chunk,page", [(24, 16), (32, 16), (7, 4)])
-def test_a_towering_key_shows_inside_its_chunk_and_nowhere_else(rts, dtype, chunk, page):
+@pytest.mark.parametrize("dtype,first", [("float32", 64), ("bfloat16", 1 << 30), ("bfloat16", 1)])
+@pytest.mark.parametrize("chunk,page", [(24, 16), (32, 16), (7, 4), (50, 8)])
+def test_a_towering_key_shows_inside_its_chunk_and_nowhere_else(rts, monkeypatch, dtype, first, chunk, page):
     """The key at a chunk's first place dominates every query of the chunk, to its last place, and none of the next chunk; in
     prompts, in portions that start inside the chunk, and in decode steps."""
     rt, H, G, d = rts[dtype], 8, 2, 64
+    monkeypatch.setattr(rt.ops, "TALK_TC_FROM", first)
     tower = 2 * chunk
     n = 4 * chunk + 3
     dp, qs, cache, tables, num_pages, talk, scale, want = _talk_case(rt, H, G, d, d, page, chunk, (n,), seed=5, tower=tower)
@@ -138,6 +139,36 @@ def test_a_towering_key_shows_inside_its_chunk_and_nowhere_else(rts, dtype, chun
     for a in (tower - 1, tower, tower + 1, 3 * chunk - 1, 3 * chunk, n - 1):
         got = _talk_run(rt, [(0, a, 1)], *args)[0]
         assert float((got - want[0][a:a + 1]).abs().max()) <= tol * big, a
+
+
+TALK_LARGE = [  # heads, key/value heads, key and value size, page, chunk: what the tcgen05 kernels take
+    (32, 8, 64, 16, 96), (16, 8, 64, 64, None), (8, 1, 128, 16, 130), (32, 4, 128, 16, 64), (6, 3, 64, 8, 37), (12, 4, 128, 32, None),
+    (2, 2, 64, 128, 200), (40, 8, 64, 16, 90),  # (the last has more heads than slots: the kernels pass it on)
+]
+
+
+@pytest.mark.parametrize("H,G,d,page,chunk", TALK_LARGE)
+def test_weights_mixed_across_heads_in_long_prompts(rts, H, G, d, page, chunk):
+    """The tcgen05 kernels, forced for any number of tokens: prompts that end inside a tile, portions that start inside a
+    chunk, a page and a tile, steps of unequal requests; against the plain outputs and against the other prefill kernel."""
+    rt = rts["bfloat16"]
+    lens = (1, 9, 128, 333)
+    dp, qs, cache, tables, num_pages, talk, scale, want = _talk_case(rt, H, G, d, d, page, chunk, lens, seed=H + d + 1)
+    args = (qs, dp, H, G, cache, tables, num_pages, page, chunk, scale, talk)
+    big = max(float(w.abs().max()) for w in want)
+    steps = [[(k, 0, n) for k, n in enumerate(lens)], [(3, 0, 333)],
+             [(1, 3, 2), (2, 37, 91), (3, 131, 130), (0, 0, 1)], [(3, 127, 2), (2, 120, 8)], [(3, 261, 72)]]
+    before, results = rt.ops.TALK_TC_FROM, {}
+    try:
+        for first in (1, 1 << 30):
+            rt.ops.TALK_TC_FROM = first
+            results[first] = [_talk_run(rt, entries, *args) for entries in steps]
+    finally:
+        rt.ops.TALK_TC_FROM = before
+    for first, runs in results.items():
+        for entries, outs in zip(steps, runs):
+            for (k, a, n), got in zip(entries, outs):
+                assert float((got - want[k][a:a + n]).abs().max()) / big <= 0.02, (first, entries, k)
 
 
 def test_decode_steps_with_a_bound_above_the_context(rts):
