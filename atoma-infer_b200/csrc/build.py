@@ -136,10 +136,10 @@ def host_library() -> ctypes.CDLL:
 def all_kernel_libraries():
     """(name, sources, defines) of every kernel library, for the build check."""
     from .ops import (ATTENTION_HEAD_DIMS, ATTENTION_SOURCES, ATTENTION_TALK_SOURCES, ATTENTION_TALK_TC_SOURCES, ATTENTION_TC_HEAD_DIMS, ATTENTION_TC_SOURCES, CORE_SOURCES,
-                      DECODE_STACK_SOURCES, GEMM_SOURCES, MATRIX_RECURRENT_SOURCES, MIXER_SOURCES, RECURRENT_SOURCES)
+                      DECODE_STACK_SOURCES, GEMM_SOURCES, MATRIX_RECURRENT_SOURCES, MIXER_SOURCES, RECURRENT_SOURCES, STREAMS_SOURCES)
 
     return [("core", CORE_SOURCES, None), ("mixers", MIXER_SOURCES, None), ("recurrent", RECURRENT_SOURCES, None),
-            ("matrix_recurrent", MATRIX_RECURRENT_SOURCES, None),
+            ("matrix_recurrent", MATRIX_RECURRENT_SOURCES, None), ("streams", STREAMS_SOURCES, None),
             ("gemm_tcgen05", GEMM_SOURCES, None)] + [
         (f"attention_d{d}", ATTENTION_SOURCES, {"HEAD_DIM": d}) for d in ATTENTION_HEAD_DIMS] + [
         (f"attention_talk_d{d}", ATTENTION_TALK_SOURCES, {"HEAD_DIM": d}) for d in ATTENTION_HEAD_DIMS] + [

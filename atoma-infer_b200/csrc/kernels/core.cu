@@ -16,12 +16,13 @@ int g_use_pdl = 1;
 extern "C" void kernels_set_pdl(int mode) { g_use_pdl = mode; }
 
 // ----------------------------------------------------------------------------- embedding
-// resid[t, :] = scale * table[tokens[t], :], widened to float32 (the residual stream is float32).
+// resid[t, c, :] = scale * table[tokens[t], :] for c < copies, widened to float32 (the residual stream is float32; models with
+// several streams side by side start with that many copies).
 // A negative token id -1 - s stands for "the token last sampled into slot s" (last_tokens[s]):
 // a decode step can be launched before the host has read the previous step's tokens.
 template <typename T>
 __global__ void embed_rows_kernel(const int* __restrict__ tokens, const T* __restrict__ table,
-                                  float* __restrict__ resid, const int* __restrict__ meta, int H, int V, float scale,
+                                  float* __restrict__ resid, const int* __restrict__ meta, int H, int V, float scale, int copies,
                                   const int* __restrict__ last_tokens, int num_slots, int* __restrict__ status) {
     pdl_launch_dependents();
     pdl_wait();
@@ -33,20 +34,23 @@ __global__ void embed_rows_kernel(const int* __restrict__ tokens, const T* __res
     bool bad = tok < 0 || tok >= V;
     if (bad && threadIdx.x == 0) atomicExch(&status[STATUS_BAD_TOKEN], 1 + t);
     const T* row = table + (size_t)(bad ? 0 : tok) * H;
-    float* out = resid + (size_t)t * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = bad ? 0.f : scale * to_float(row[i]);
+    float* out = resid + (size_t)t * copies * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = bad ? 0.f : scale * to_float(row[i]);
+        for (int c = 0; c < copies; ++c) out[(size_t)c * H + i] = v;
+    }
 }
 
 extern "C" int embed_rows(const int* tokens, const void* table, int table_dtype, float* resid, const int* meta,
-                          int T, int H, int V, float scale, const int* last_tokens, int num_slots, int* status,
+                          int T, int H, int V, float scale, int copies, const int* last_tokens, int num_slots, int* status,
                           cudaStream_t stream) {
     if (T <= 0) return 0;
     int threads = H >= 1024 ? 256 : 128;
     if (table_dtype == DT_F32)
-        return (int)launch_kernel(embed_rows_kernel<float>, T, threads, 0, stream, tokens, (const float*)table, resid, meta, H, V, scale,
+        return (int)launch_kernel(embed_rows_kernel<float>, T, threads, 0, stream, tokens, (const float*)table, resid, meta, H, V, scale, copies,
                                   last_tokens, num_slots, status);
     return (int)launch_kernel(embed_rows_kernel<__nv_bfloat16>, T, threads, 0, stream, tokens, (const __nv_bfloat16*)table, resid,
-                              meta, H, V, scale, last_tokens, num_slots, status);
+                              meta, H, V, scale, copies, last_tokens, num_slots, status);
 }
 
 // ----------------------------------------------------------------------------- RMSNorm

@@ -40,7 +40,7 @@ extern "C" int rms_rows(const void* x, int dtype, long long x_stride, const floa
 
 // ----------------------------------------------------------------------------- a linear map per head
 // y[t, h, n] = sum_k x[t, h, k] * w[h, n, k] (optionally times sigmoid(gate[t, h, n])).  x, y and gate are slices:
-// element (t, h, i) lies at t * stride_t + h * stride_h + i.
+// element (t, h, i) lies at t * stride_t + h * stride_h + i (of a gate with one number per head: without the i).
 #define HL_TM 8
 #define HL_TN 128
 #define HL_KC 512
@@ -51,7 +51,7 @@ template <typename T>
 __global__ void __launch_bounds__(HL_TN)
 head_linear_kernel(const T* __restrict__ x, long long xs_t, long long xs_h, const T* __restrict__ w, T* __restrict__ y,
                    long long ys_t, long long ys_h, const T* __restrict__ gate, long long gs_t, long long gs_h,
-                   const int* __restrict__ meta, int K, int N, int wvec) {
+                   int gate_per_head, const int* __restrict__ meta, int K, int N, int wvec) {
     __shared__ float xs[HL_TM][HL_KC];
     pdl_launch_dependents();
     pdl_wait();
@@ -95,7 +95,7 @@ head_linear_kernel(const T* __restrict__ x, long long xs_t, long long xs_h, cons
     for (int m = 0; m < rows; ++m) {
         float v = acc[m];
         if (gate) {
-            const float g = to_float(gate[(size_t)(t0 + m) * gs_t + (size_t)h * gs_h + n]);
+            const float g = to_float(gate[(size_t)(t0 + m) * gs_t + (size_t)h * gs_h + (gate_per_head ? 0 : n)]);
             v = v / (1.f + expf(-g));
         }
         y[(size_t)(t0 + m) * ys_t + (size_t)h * ys_h + n] = from_float<T>(v);
@@ -103,8 +103,8 @@ head_linear_kernel(const T* __restrict__ x, long long xs_t, long long xs_h, cons
 }
 
 extern "C" int head_linear(const void* x, long long xs_t, long long xs_h, const void* w, void* y, long long ys_t,
-                           long long ys_h, const void* gate, long long gs_t, long long gs_h, int dtype, const int* meta, int T,
-                           int heads, int K, int N, cudaStream_t stream) {
+                           long long ys_h, const void* gate, long long gs_t, long long gs_h, int gate_per_head, int dtype, const int* meta,
+                           int T, int heads, int K, int N, cudaStream_t stream) {
     if (T <= 0) return 0;
     const int tn = N <= 32 ? 32 : (N <= 64 ? 64 : HL_TN);  // few outputs a head: smaller blocks, all of their threads at work
     dim3 grid((T + HL_TM - 1) / HL_TM, heads, (N + tn - 1) / tn);
@@ -112,10 +112,10 @@ extern "C" int head_linear(const void* x, long long xs_t, long long xs_h, const 
     const int wvec = ((size_t)K * elem) % 16 == 0 && ((uintptr_t)w & 15) == 0;
     if (dtype == DT_F32)
         return (int)launch_kernel(head_linear_kernel<float>, grid, tn, 0, stream, (const float*)x, xs_t, xs_h, (const float*)w,
-                                  (float*)y, ys_t, ys_h, (const float*)gate, gs_t, gs_h, meta, K, N, wvec);
+                                  (float*)y, ys_t, ys_h, (const float*)gate, gs_t, gs_h, gate_per_head, meta, K, N, wvec);
     return (int)launch_kernel(head_linear_kernel<__nv_bfloat16>, grid, tn, 0, stream, (const __nv_bfloat16*)x, xs_t, xs_h,
                               (const __nv_bfloat16*)w, (__nv_bfloat16*)y, ys_t, ys_h, (const __nv_bfloat16*)gate, gs_t, gs_h,
-                              meta, K, N, wvec);
+                              gate_per_head, meta, K, N, wvec);
 }
 
 // y[t, h, n] *= sigmoid(gate[t, h, n]) for a product that a library made (same slices as above).  ``vec``: every head's
@@ -169,7 +169,7 @@ extern "C" int sigmoid_gate(void* y, long long ys_t, long long ys_h, const void*
 // Per token: the cached vector [c | rotated key part | zeros] with c = dkv[:rank] * rsqrt(mean(.^2) + eps) * norm_w
 // goes to the key plane and to the value plane of the token's page (one key/value head of D elements); the queries
 // become [q_abs[h] | rotated q_rot[h] | zeros] of D elements a head.  Rotation: of the first `rot` dimensions of a
-// rotated part, 2i pairs with 2i + 1, by the angle position * inv_freq[i] (float32 product, sincosf).
+// rotated part, 2i pairs with 2i + 1 (`halves`: i with i + rot / 2), by the angle position * inv_freq[i] (float32 product, sincosf).
 // Two neighbouring elements at once (the address a multiple of two elements): a rotation's pair.
 __device__ __forceinline__ void load2(const float* p, float& a, float& b) { const float2 t = *reinterpret_cast<const float2*>(p); a = t.x; b = t.y; }
 __device__ __forceinline__ void load2(const __nv_bfloat16* p, float& a, float& b) {
@@ -179,6 +179,43 @@ __device__ __forceinline__ void load2(const __nv_bfloat16* p, float& a, float& b
 __device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
 __device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
 
+// Elements j and j + 1 (j even) of a rotated part whose element 0 is at `p`, turned if they belong to the first `rot`:
+// interleaved, 2i pairs with 2i + 1; `halves`: i pairs with i + rot / 2 (rot / 2 even, so both partners are one access).
+template <typename T>
+__device__ __forceinline__ void turned2(const T* p, int j, int rot, int halves, const float* cs, const float* sn, float& a, float& b) {
+    load2(p + j, a, b);
+    if (j >= rot) return;
+    const float a0 = a, b0 = b;
+    if (!halves) {
+        rotate_pair(a0, b0, cs[j >> 1], sn[j >> 1], a, b);
+        return;
+    }
+    const int half = rot / 2;
+    float c, d, unused;
+    if (j < half) {
+        load2(p + j + half, c, d);
+        rotate_pair(a0, c, cs[j], sn[j], a, unused);
+        rotate_pair(b0, d, cs[j + 1], sn[j + 1], b, unused);
+    } else {
+        const int f = j - half;
+        load2(p + f, c, d);
+        rotate_pair(c, a0, cs[f], sn[f], unused, a);
+        rotate_pair(d, b0, cs[f + 1], sn[f + 1], unused, b);
+    }
+}
+// One element likewise, any sizes.
+template <typename T>
+__device__ __forceinline__ float turned1(const T* p, int j, int rot, int halves, const float* cs, const float* sn) {
+    const float v = to_float(p[j]);
+    if (j >= rot) return v;
+    const int half = rot / 2, f = halves ? (j < half ? j : j - half) : j >> 1;
+    const bool low = halves ? j < half : !(j & 1);
+    const float other = to_float(p[halves ? (low ? j + half : f) : j ^ 1]);
+    float lo, hi;
+    rotate_pair(low ? v : other, low ? other : v, cs[f], sn[f], lo, hi);
+    return low ? lo : hi;
+}
+
 // A block takes one token and `hpb` of its heads + 1 jobs: job h < heads lays out query head h, job `heads` makes the
 // cached vector.  Few tokens: a job a block; many: all of a token's jobs in one block, which takes the cosines and
 // sines once.  `pairs`: sizes, strides and addresses are even, so a thread takes a rotation's pair with one access.
@@ -187,7 +224,7 @@ __global__ void __launch_bounds__(256)
 latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, const T* __restrict__ q_abs,
                    const T* __restrict__ dkv, long long dkv_stride, const float* __restrict__ norm_w, float eps,
                    const int* __restrict__ positions, const int* __restrict__ token_entry, const int* __restrict__ meta,
-                   int group, const float* __restrict__ inv_freq, int rot, T* __restrict__ q_out, T* __restrict__ cache,
+                   int group, const float* __restrict__ inv_freq, int rot, int halves, T* __restrict__ q_out, T* __restrict__ cache,
                    int heads, int rank, int rdim, int D, int page_size, int num_pages, int store, int pairs, int hpb,
                    int* __restrict__ status) {
     __shared__ float red[33];
@@ -215,12 +252,7 @@ latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, 
                 if (i < rank) {
                     load2(qa + i, a, b);
                 } else if (i < rank + rdim) {
-                    const int j = i - rank;
-                    load2(qr + j, a, b);
-                    if (j < rot) {
-                        const float a0 = a, b0 = b;
-                        rotate_pair(a0, b0, cs[j >> 1], sn[j >> 1], a, b);
-                    }
+                    turned2(qr, i - rank, rot, halves, cs, sn, a, b);
                 }
                 store2(dst + i, a, b);
             }
@@ -231,14 +263,7 @@ latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, 
             if (i < rank) {
                 v = to_float(qa[i]);
             } else if (i < rank + rdim) {
-                const int j = i - rank;
-                v = to_float(qr[j]);
-                if (j < rot) {
-                    const float other = to_float(qr[j ^ 1]);
-                    float lo, hi;
-                    if (j & 1) { rotate_pair(other, v, cs[j >> 1], sn[j >> 1], lo, hi); v = hi; }
-                    else { rotate_pair(v, other, cs[j >> 1], sn[j >> 1], lo, hi); v = lo; }
-                }
+                v = turned1(qr, i - rank, rot, halves, cs, sn);
             }
             dst[i] = from_float<T>(v);
         }
@@ -267,12 +292,7 @@ latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, 
                 a = a * inv * norm_w[i];
                 b = b * inv * norm_w[i + 1];
             } else if (i < rank + rdim) {
-                const int j = i - rank;
-                load2(kv + i, a, b);
-                if (j < rot) {
-                        const float a0 = a, b0 = b;
-                        rotate_pair(a0, b0, cs[j >> 1], sn[j >> 1], a, b);
-                    }
+                turned2(kv + rank, i - rank, rot, halves, cs, sn, a, b);
             }
             store2(kdst + i, a, b);
             store2(vdst + i, a, b);
@@ -284,14 +304,7 @@ latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, 
         if (i < rank) {
             v = to_float(kv[i]) * inv * norm_w[i];
         } else if (i < rank + rdim) {
-            const int j = i - rank;
-            v = to_float(kv[i]);
-            if (j < rot) {
-                const float other = to_float(kv[rank + (j ^ 1)]);
-                float lo, hi;
-                if (j & 1) { rotate_pair(other, v, cs[j >> 1], sn[j >> 1], lo, hi); v = hi; }
-                else { rotate_pair(v, other, cs[j >> 1], sn[j >> 1], lo, hi); v = lo; }
-            }
+            v = turned1(kv + rank, i - rank, rot, halves, cs, sn);
         }
         const T o = from_float<T>(v);
         kdst[i] = o;
@@ -301,25 +314,25 @@ latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, 
 
 extern "C" int latent_rows(const void* q_rot, long long qs_t, long long qs_h, const void* q_abs, const void* dkv,
                            long long dkv_stride, const float* norm_w, float eps, const int* positions, const int* token_entry,
-                           const int* meta, int group, const float* inv_freq, int rot, void* q_out, void* cache, int dtype,
+                           const int* meta, int group, const float* inv_freq, int rot, int halves, void* q_out, void* cache, int dtype,
                            int T, int heads, int rank, int rdim, int D, int page_size, int num_pages, int store, int* status,
                            cudaStream_t stream) {
     if (T <= 0) return 0;
     if (rot % 2 || rot > rdim || rank + rdim > D || (rot && !inv_freq)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)rot * sizeof(float);
     const int elem = dtype == DT_F32 ? 4 : 2;
-    const int pairs = rank % 2 == 0 && rdim % 2 == 0 && D % 2 == 0 && qs_t % 2 == 0 && qs_h % 2 == 0 && dkv_stride % 2 == 0 &&
+    const int pairs = rank % 2 == 0 && rdim % 2 == 0 && D % 2 == 0 && (!halves || rot % 4 == 0) && qs_t % 2 == 0 && qs_h % 2 == 0 && dkv_stride % 2 == 0 &&
                       (((uintptr_t)q_rot | (uintptr_t)q_abs | (uintptr_t)dkv | (uintptr_t)q_out | (uintptr_t)cache) % (2 * elem)) == 0;
     const int hpb = T >= 512 ? heads + 1 : 1, threads = hpb > 1 ? 256 : 128;
     const dim3 grid(T, (heads + 1 + hpb - 1) / hpb);
     if (dtype == DT_F32)
         return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<float>, grid, threads, smem, stream, (const float*)q_rot, qs_t,
                                       qs_h, (const float*)q_abs, (const float*)dkv, dkv_stride, norm_w, eps, positions, token_entry,
-                                      meta, group, inv_freq, rot, (float*)q_out, (float*)cache, heads, rank, rdim, D, page_size,
+                                      meta, group, inv_freq, rot, halves, (float*)q_out, (float*)cache, heads, rank, rdim, D, page_size,
                                       num_pages, store, pairs, hpb, status);
     return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<__nv_bfloat16>, grid, threads, smem, stream,
                                   (const __nv_bfloat16*)q_rot, qs_t, qs_h, (const __nv_bfloat16*)q_abs, (const __nv_bfloat16*)dkv,
-                                  dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq, rot,
+                                  dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq, rot, halves,
                                   (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, heads, rank, rdim, D, page_size, num_pages, store,
                                   pairs, hpb, status);
 }

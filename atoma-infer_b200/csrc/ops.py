@@ -38,6 +38,8 @@ MIXER_SOURCES = ["kernels/stream_ops.cu", "kernels/ssm.cu", "kernels/latent.cu",
 RECURRENT_SOURCES = ["kernels/recurrent.cu"]
 # recurrences whose query reads more than the decayed state (a bonus for the current token, a memory with a normalizer)
 MATRIX_RECURRENT_SOURCES = ["kernels/matrix_recurrent.cu"]
+# several residual streams side by side, attention as the difference of two maps
+STREAMS_SOURCES = ["kernels/stream_mix.cu", "kernels/differential.cu"]
 ATTENTION_TC_HEAD_DIMS = (64, 128)  # head sizes of the tcgen05 prefill attention
 ATTENTION_HEAD_DIMS = tuple(range(16, 257, 16))  # every head size the kernels take; the build check builds them all, a model only its own
 
@@ -135,7 +137,7 @@ class CudaOps:
         self.lib.kernels_set_pdl(int(on))
         for lib in list(self._attn_libs.values()) + list(self._talk_libs.values()):
             lib.kernels_set_pdl(1 if on else 0)
-        for name in ("_mixer_lib", "_recurrent_lib", "_matrix_recurrent_lib"):
+        for name in ("_mixer_lib", "_recurrent_lib", "_matrix_recurrent_lib", "_streams_lib"):
             if getattr(self, name, None) is not None:
                 getattr(self, name).kernels_set_pdl(int(on))
 
@@ -224,12 +226,12 @@ class CudaOps:
             self._side_pending = False
 
     # ------------------------------------------------------------------ kernels
-    def embed(self, tokens, table, resid, meta, T: int, scale: float = 1.0):
-        """resid[t] = scale * table[tokens[t]].  A token id -1 - s means: the token last sampled into slot s
-        (``self.last_tokens``)."""
+    def embed(self, tokens, table, resid, meta, T: int, scale: float = 1.0, copies: int = 1):
+        """resid[t] = scale * table[tokens[t]], ``copies`` times side by side.  A token id -1 - s means: the token last
+        sampled into slot s (``self.last_tokens``)."""
         H, V = table.shape[1], table.shape[0]
         self._check(self.lib.embed_rows(_p(tokens), _p(table), _code(table), _p(resid), _p(meta), T, H, V,
-                                        ctypes.c_float(scale), _p(self.last_tokens), self.last_tokens.numel(),
+                                        ctypes.c_float(scale), int(copies), _p(self.last_tokens), self.last_tokens.numel(),
                                         _p(self.status), self._stream()), "embed_rows")
 
     def add_rmsnorm(self, resid, delta, w, eps: float, out, meta, n: int, rows=None):
@@ -748,36 +750,43 @@ class CudaOps:
 
     def head_linear(self, x, w, out, meta, gate=None):
         """out[t, h] = w[h] x[t, h] (times sigmoid(gate[t, h]) if given): x [T, heads, K], out and gate [T, heads, N] slices
-        with a contiguous last axis, w [heads, N, K] contiguous."""
+        with a contiguous last axis, w [heads, N, K] contiguous.  A gate [T, heads] is one number per head."""
         heads, N, K = w.shape
         T = x.shape[0]
         lib = self._mixers()
         op, ot, oh = self._heads(out, "head_linear")
-        gp, gt, gh = self._heads(gate, "head_linear") if gate is not None else (None, ctypes.c_longlong(0), ctypes.c_longlong(0))
+        gp, gt, gh = None, ctypes.c_longlong(0), ctypes.c_longlong(0)
+        per_head = gate is not None and gate.dim() == 2
+        if per_head:
+            (gp, gt), gh = self._rows(gate, "head_linear"), ctypes.c_longlong(1)
+        elif gate is not None:
+            gp, gt, gh = self._heads(gate, "head_linear")
         if x.dtype == torch.bfloat16 and T >= self.HEAD_LINEAR_LIBRARY_ROWS:
             out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
-            if gate is not None:
+            if per_head:
+                self.head_gate(out, gate, meta)
+            elif gate is not None:
                 self._check(lib.sigmoid_gate(op, ot, oh, gp, gt, gh, _code(out), _p(meta), T, heads, N, self._stream()),
                             "sigmoid_gate")
             return
         xp, xt, xh = self._heads(x, "head_linear")
-        self._check(lib.head_linear(xp, xt, xh, _p(w), op, ot, oh, gp, gt, gh, _code(x), _p(meta), T, heads, K, N,
+        self._check(lib.head_linear(xp, xt, xh, _p(w), op, ot, oh, gp, gt, gh, int(per_head), _code(x), _p(meta), T, heads, K, N,
                                     self._stream()), "head_linear")
 
     def latent_rows(self, q_rot, q_abs, dkv, norm_w, eps: float, ctx, cache_layer, group: int, q_out, *, heads: int,
                     kv_rank: int, rot_dim: int, padded: int, page_size: int, num_pages: int, store: bool, inv_freq=None,
-                    rotary_dims: int = 0):
+                    rotary_dims: int = 0, halves: bool = False):
         """The rows of latent attention.  The cached vector [rmsnorm(dkv[:kv_rank]) * norm_w | rotated dkv[kv_rank:] |
         zeros] of ``padded`` elements goes to the key plane and the value plane of the token's page; the queries become
         [q_abs[h] | rotated q_rot[h] | zeros] in ``q_out`` [T, heads * padded].  Rotation: of the first ``rotary_dims``
-        dimensions, 2i pairs with 2i + 1, angle position * inv_freq[i]."""
+        dimensions, 2i pairs with 2i + 1 (``halves``: i with i + rotary_dims / 2), angle position * inv_freq[i]."""
         qp, qt, qh = self._heads(q_rot, "latent_rows")
         dp, ds = self._rows(dkv, "latent_rows")
         if not q_abs.is_contiguous():
             raise KernelError("latent_rows: q_abs must be contiguous")
         self._check(self._mixers().latent_rows(qp, qt, qh, _p(q_abs), dp, ds, _p(norm_w), ctypes.c_float(eps), _p(ctx.positions),
                                                _p(ctx.token_entry), _p(ctx.meta), max(group, 0), _p(inv_freq),
-                                               int(rotary_dims) if inv_freq is not None else 0, _p(q_out), _p(cache_layer),
+                                               int(rotary_dims) if inv_freq is not None else 0, int(halves), _p(q_out), _p(cache_layer),
                                                _code(q_out), ctx.T, heads, kv_rank, rot_dim, padded, page_size, num_pages,
                                                int(store), _p(self.status), self._stream()), "latent_rows")
 
@@ -788,6 +797,75 @@ class CudaOps:
         gp, gt, gh = self._heads(gate, "sigmoid_gate")
         self._check(self._mixers().sigmoid_gate(yp, yt, yh, gp, gt, gh, _code(y), _p(meta), T, heads, N, self._stream()),
                     "sigmoid_gate")
+
+    # ------------------------------------------------------------------ several streams, differential attention
+    def _streams(self):
+        lib = getattr(self, "_streams_lib", None)
+        if lib is None:
+            lib = self._streams_lib = build.load_library("streams", STREAMS_SOURCES, cuda=True)
+            lib.kernels_set_pdl(int(self.pdl))
+        return lib
+
+    def stream_mix_norm(self, resid, streams: int, pending, read, w, eps: float, out, meta, n: int, rows=None):
+        """``resid`` float32 [T, streams * H].  With ``pending`` (a ``StreamMix``): y = its result (up to four weighted terms,
+        a factor, a vector) times its scale per channel; stream k becomes sum_j mix[j, k] x_j + give[k] y.  With ``out``: out =
+        rmsnorm(sum_k read[k] x_k) * w (``read`` None: the plain sum).  With ``rows`` both are taken at those rows only and
+        ``resid`` is left as it is."""
+        H = resid.shape[-1] // streams
+        p = pending.result if pending is not None else None
+        terms = list(p.terms) if p is not None else []
+        if len(terms) > 4 or len({t.dtype for t in terms}) > 1:
+            raise KernelError("a sublayer's result has at most four terms, of one type")
+        if p is not None and (not terms or p.rows is not None or p.norms is not None):
+            raise KernelError("what enters several streams has terms, weights, a factor and a vector only")
+        for t in (pending.mix, pending.give, pending.scale) if pending is not None else ():
+            if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+                raise KernelError("the weights of the streams are contiguous float32 tensors")
+        if pending is not None and (tuple(pending.mix.shape) != (streams, streams) or pending.give.numel() != streams):
+            raise KernelError(f"{streams} streams are mixed by a matrix of that size")
+        ptrs = (ctypes.c_void_p * 4)(*[t.data_ptr() for t in terms])
+        facs = (ctypes.c_float * 4)(*(p.weights() if p is not None else ()))
+        tcode = _code(terms[0]) if terms else (_code(out) if out is not None else DT_F32)
+        self._check(self._streams().stream_mix_norm(
+            _p(resid), streams, len(terms), ptrs, facs, tcode, ctypes.c_float(p.mult if p is not None else 1.0),
+            _p(p.vector if p is not None else None), _p(pending.scale if pending is not None else None),
+            _p(pending.mix if pending is not None else None), _p(pending.give if pending is not None else None), _p(read), _p(rows),
+            _p(w), ctypes.c_float(eps), _p(out), _code(out) if out is not None else DT_F32, _p(meta), n, H, self._stream()),
+            "stream_mix_norm")
+
+    def map_rows(self, qkv, ctx, cache_layer, group: int, q_out, *, heads: int, kv_heads: int, maps: int, d: int, dv: int, dp: int,
+                 page_size: int, num_pages: int, store_kv: bool, bias=None, conv_w=None, ring=None):
+        """Rows [q: heads * maps * d | k: kv_heads * maps * d | v: kv_heads * dv] (a slice of wider rows) of attention with
+        several maps over the same values become the attention kernels' inputs: biases (float32) are added, then every
+        channel goes through a causal convolution over time (``conv_w`` float32 [taps, channels]; None: none) whose earlier
+        rows, without biases, come from ``ring`` (float32 [slots, taps - 1, channels], the row of position p at place p mod
+        (taps - 1)), terms before the request's start left out.  Query map (h, m) goes to ``q_out`` [T, heads * maps * dp] as
+        a head that holds its values at m * d and zeros elsewhere; a key head's maps side by side, and a value head, go to
+        the token's page, zeros behind them.  The ring is updated too: in decode steps by the same launch, else by a second one."""
+        taps = conv_w.shape[0] if conv_w is not None else 0
+        n = (heads + kv_heads) * maps * d + kv_heads * dv
+        if conv_w is not None and (conv_w.shape[1] != n or conv_w.dtype != torch.float32 or not conv_w.is_contiguous()):
+            raise KernelError(f"the convolution of the rows has contiguous float32 weights [taps, {n}]")
+        if bias is not None and (bias.dtype != torch.float32 or bias.numel() != n):
+            raise KernelError(f"the rows have {n} float32 biases")
+        up, us = self._rows(qkv, "map_rows")
+        saves = bool(1 < taps <= 4 and ctx.decode_only and ctx.T == ctx.S)
+        lib, stride = self._streams(), self._slot_stride(ring)
+        self._check(lib.map_rows(up, _code(qkv), us, _p(bias), _p(conv_w), taps, _p(ring), stride, _p(q_out), _p(cache_layer), _p(ctx.meta),
+                                 _p(ctx.positions), _p(ctx.token_entry), _p(ctx.cu_tokens), _p(ctx.state_slots), max(group, 0), ctx.T,
+                                 heads, kv_heads, maps, d, dv, dp, page_size, num_pages, int(store_kv), int(saves), _p(self.status),
+                                 self._stream()), "map_rows")
+        if taps > 1 and not saves:
+            self._check(lib.map_rows_save(up, _code(qkv), us, _p(ring), stride, _p(ctx.meta), _p(ctx.positions), _p(ctx.cu_tokens),
+                                          _p(ctx.state_slots), ctx.S, n, taps, self._stream()), "map_rows_save")
+
+    def map_difference(self, a, gate, lam, factor: float, eps: float, out, meta, *, heads: int, dp: int):
+        """``a`` [T, heads * 2 * dp]: per head the results of two maps, ``dv`` values each (``out`` is [T, heads * dv]); o = a_1 -
+        lam a_2 (``lam``: one float32 number on the device), out = o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate[t, h]),
+        ``gate`` [T, heads] a slice of wider rows or None."""
+        gp, gs = self._rows(gate, "map_difference") if gate is not None else (None, ctypes.c_longlong(0))
+        self._check(self._streams().map_difference(_p(a), _code(a), dp, gp, gs, _p(lam), ctypes.c_float(factor), ctypes.c_float(eps), _p(out),
+                                                   _p(meta), a.shape[0], heads, out.shape[1] // heads, self._stream()), "map_difference")
 
     # ------------------------------------------------------------------ recurrences with a decay per row
     def _recurrent(self):

@@ -51,14 +51,14 @@ def make_runtime(dtype: str, device=None, ops=None) -> Runtime:
 
 
 def step_workspace_bytes(model: DecoderModel, dtype: torch.dtype, max_batched_tokens: int, max_seqs: int) -> int:
-    """An upper estimate of what a step allocates besides the cache: per token the float32 residual stream and
+    """An upper estimate of what a step allocates besides the cache: per token the float32 residual stream(s) and
     some ten rows of the widest activation any part says it makes (intermediate results live one or two at a
     time), and the float32 logits of one row per request; twice over, because captured decode graphs keep a
     pool of their own."""
     elem = torch.empty((), dtype=dtype).element_size()
     spec = model.spec
     widest = max([spec.hidden_size] + [blk.activation_width() for blk in model.blocks])
-    per_token = 4 * spec.hidden_size + 10 * widest * elem
+    per_token = 4 * spec.hidden_size * max(spec.streams, 1) + 10 * widest * elem
     return 2 * (max_batched_tokens * per_token + max(max_seqs, 1) * spec.vocab_size * 4)
 
 

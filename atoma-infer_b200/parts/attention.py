@@ -43,6 +43,13 @@ matrix).
 ``head_scale``: head h's scores are multiplied by a learned number per head (``.temp``; it multiplies the query);
 ``talk``: the softmax weights are mixed across the heads, p_h <- sum_g T[h, g] p_g with a learned T [heads, heads] (``.talk``),
 before head h weighs the values of its own key/value head (goes with ``chunk``; not with a window, a sink or score options).
+``differential`` ``{"diff": c, "eps": e}``: every query head and every key head holds two maps of ``head_dim`` each, laid out head
+by head as [map 1, map 2]; each map is an attention of its own over the same values, o = a_1 - lambda a_2 with lambda =
+exp(sum lq1 lk1) - exp(sum lq2 lk2) + c (learned vectors of head_dim, one lambda for the layer), o is divided by its root
+mean square over the head's values (eps e, no weight) and multiplied by 1 - c.  It runs on the attention kernels as they
+are: a key head's two maps side by side are ONE key head of the cache, a query map is a query head that holds zeros where
+the other map's key lies.  Goes with ``bias``, ``conv``, ``head_gate``, ``window``, ``chunk`` and ``softcap``; not with what
+norms, rotates or mixes the rows.  Biases are part of the projection: the convolution reads rows that have them.
 The position encoding's ``interleaved`` pairs dimension 2i with 2i + 1.
 With any of ``v_head_dim``, ``bias``, ``qk_norm``, ``v_mix``, ``head_norm`` (and the options above that touch the rows) the rows are prepared by one kernel (``qkv_prepare``) that writes queries, keys and values
 as heads of one padded size, the next multiple of 16 above both sizes, which the tensor-core kernels read like any
@@ -99,25 +106,34 @@ class Attention(Mixer):
         if self.keep_first and not self.window:
             raise ValueError("keep_first goes with a window")
         interleaved = bool((p.get("position") or {}).get("interleaved", False))
+        self.differential = p.get("differential")
+        self.maps = 2 if self.differential is not None else 1
+        if self.differential is not None and (self.qk_norm is not None or self.v_mix is not None or self.head_norm is not None or self.gate
+                                              or self.q_temp or self.head_scale or self.talk or self.sink or self.distance_bias or self.out_bias
+                                              or self.keep_first or (p.get("position") or {"kind": "none"})["kind"] != "none"):
+            raise ValueError("differential goes with biases, a convolution, a gate per head, a window, a chunk and a score cap only")
+        if self.taps and self.bias and self.differential is None:
+            raise ValueError("a convolution behind projections with biases goes with differential attention only")
         self.prepared = bool(self.bias or self.qk_norm is not None or self.v_mix is not None or self.head_norm is not None
                              or self.gate or self.v_head_dim != self.head_dim or interleaved or self.q_temp or self.taps
-                             or self.head_gate or self.head_scale or self.talk)
-        self.padded_dim = -(-max(self.head_dim, self.v_head_dim) // 16) * 16 if self.prepared else self.head_dim
+                             or self.head_gate or self.head_scale or self.talk or self.differential is not None)
+        self.padded_dim = -(-max(self.maps * self.head_dim, self.v_head_dim) // 16) * 16 if self.prepared else self.head_dim
         self.names = {"q": ".q_proj.weight", "k": ".k_proj.weight", "v": ".v_proj.weight", "o": ".o_proj.weight",
                       "q_bias": ".q_proj.bias", "k_bias": ".k_proj.bias", "v_bias": ".v_proj.bias",
                       "q_norm": ".q_norm.weight", "k_norm": ".k_norm.weight", "v_mix": ".v_mix", "gate": ".g_proj.weight",
-                      "o_bias": ".o_proj.bias", "sink": ".sink", "conv": ".conv", "temp": ".temp", "talk": ".talk", **(p.get("names") or {})}
+                      "o_bias": ".o_proj.bias", "sink": ".sink", "conv": ".conv", "temp": ".temp", "talk": ".talk", "lq1": ".lq1",
+                      "lk1": ".lk1", "lq2": ".lq2", "lk2": ".lk2", **(p.get("names") or {})}
         pos = dict(p.get("position") or {"kind": "none"})
         pos.setdefault("head_dim", self.head_dim)
         self.position = part_class("position", pos["kind"])(pos, prefix)
 
     @property
     def q_size(self):
-        return self.num_heads * self.head_dim
+        return self.num_heads * self.maps * self.head_dim
 
     @property
     def kv_size(self):
-        return self.num_kv_heads * self.head_dim
+        return self.num_kv_heads * self.maps * self.head_dim
 
     @property
     def v_size(self):
@@ -126,7 +142,7 @@ class Attention(Mixer):
     def activation_width(self):
         gate = self.num_heads * self.v_head_dim if self.gate else (self.num_heads if self.head_gate else 0)
         rows = self.q_size + self.kv_size + self.v_size
-        return max(rows + gate + (rows if self.taps else 0), 2 * self.num_heads * self.padded_dim)
+        return max(rows + gate + (rows if self.taps else 0), 2 * self.num_heads * self.maps * self.padded_dim)
 
     def state_bytes(self):
         """The convolution's ring: the last taps - 1 projected rows [q | k | v] of a request, float32."""
@@ -177,6 +193,8 @@ class Attention(Mixer):
                       for x, size in (("q", self.q_size), ("k", self.kv_size), ("v", self.v_size))]
         if self.v_mix is not None:
             decls.append(TensorDecl(pre + n["v_mix"], ()))
+        if self.differential is not None:
+            decls += [TensorDecl(pre + n[x], (self.head_dim,)) for x in ("lq1", "lk1", "lq2", "lk2")]
         if self.gate:
             decls.append(TensorDecl(pre + n["gate"], (self.num_heads * self.v_head_dim, self.hidden)))
         return decls + self.position.declare()
@@ -199,6 +217,15 @@ class Attention(Mixer):
                        .to(torch.float32).to(rt.device).contiguous() if self.distance_bias else None)
         if not self.prepared:
             return
+        self.conv_w = None
+        if self.differential is not None:
+            # rows added to a multiple of 8: with a gate per head behind q, k and v every row still starts on 16 bytes
+            self.w_qkv = torch.cat([self.w_qkv, self.w_qkv.new_zeros((-self.w_qkv.shape[0] % 8, self.hidden))], 0).contiguous()
+            self.b_qkv = torch.cat([f32("q_bias"), f32("k_bias"), f32("v_bias")]).contiguous() if self.bias else None
+            lam = torch.exp((f32("lq1") * f32("lk1")).sum()) - torch.exp((f32("lq2") * f32("lk2")).sum()) + float(self.differential["diff"])
+            self.map_weight = lam.reshape(1).contiguous()
+            self._bind_conv(tensors)
+            return  # (what follows the difference has heads of v_head_dim: the output matrix stays as it is)
         # Biases and norm weights stay as the loader left them when that is one type for all (bfloat16 from a bfloat16
         # checkpoint: the kernel widens them, exactly, as it reads them); else all are widened here.
         normed = self.qk_norm is not None or self.head_norm_weight
@@ -208,13 +235,17 @@ class Attention(Mixer):
         self.b_qkv = torch.cat([get("q_bias"), get("k_bias"), get("v_bias")]).contiguous() if self.bias else None
         self.w_q_norm, self.w_k_norm = (get("q_norm"), get("k_norm")) if normed else (None, None)
         self.v_lambda = f32("v_mix").reshape(1) if self.v_mix is not None else None
-        # [taps, channels] over the fused [q | k | v] rows: neighbouring threads read neighbouring weights
-        self.conv_w = (torch.cat([tensors[pre + n[x] + n["conv"]] for x in ("q", "k", "v")], 0).to(torch.float32).t().contiguous()
-                       if self.taps else None)
+        self._bind_conv(tensors)
         if self.padded_dim != self.v_head_dim:  # the attention's output has heads of the padded size: zero columns for the tail
             w = self.w_o.new_zeros((self.hidden, self.num_heads, self.padded_dim))
             w[:, :, :self.v_head_dim] = self.w_o.view(self.hidden, self.num_heads, self.v_head_dim)
             self.w_o = w.view(self.hidden, self.num_heads * self.padded_dim).contiguous()
+
+    def _bind_conv(self, tensors):
+        """[taps, channels] over the fused [q | k | v] rows: neighbouring threads read neighbouring weights."""
+        pre, n = self.prefix, self.names
+        self.conv_w = (torch.cat([tensors[pre + n[x] + n["conv"]] for x in ("q", "k", "v")], 0).to(torch.float32).t().contiguous()
+                       if self.taps else None)
 
     def fused(self):
         rotary = self.position.rotary()
@@ -228,6 +259,23 @@ class Attention(Mixer):
         """What changes a score or the mask beyond window, chunk and sink, as keyword arguments of ``ops.attention``."""
         return {k: v for k, v in (("keep_first", self.keep_first), ("softcap", self.softcap), ("slopes", self.slopes))
                 if v is not None and (torch.is_tensor(v) or v)}
+
+    def _forward_differential(self, x, ctx, cache):
+        ops = self.rt.ops
+        H, G, dp, n = self.num_heads, self.num_kv_heads, self.padded_dim, self.q_size + self.kv_size + self.v_size
+        rows = ops.linear(x, self.w_qkv, meta=ctx.meta)
+        q = torch.empty((ctx.T, H * 2 * dp), dtype=x.dtype, device=x.device)
+        ops.map_rows(rows[:, :n], ctx, cache.pages, cache.group, q, heads=H, kv_heads=G, maps=2, d=self.head_dim, dv=self.v_head_dim,
+                     dp=dp, page_size=cache.page_size, num_pages=cache.num_pages, store_kv=cache.writes and cache.pages is not None,
+                     bias=self.b_qkv, conv_w=self.conv_w, ring=self.ring(cache.state))
+        a = torch.empty_like(q)
+        ops.attention(q, H * 2 * dp, cache.pages, ctx, cache.group, a, 2 * H, G, dp, cache.page_size, cache.num_pages,
+                      int(self.window or 0), self.scale, **({"chunk": self.chunk} if self.chunk else {}), **self._score_options())
+        out = torch.empty((ctx.T, H * self.v_head_dim), dtype=x.dtype, device=x.device)
+        c = float(self.differential["diff"])
+        ops.map_difference(a, rows[:, n:n + H] if self.head_gate else None, self.map_weight, 1.0 - c, float(self.differential["eps"]), out,
+                           ctx.meta, heads=H, dp=dp)
+        return ops.linear(out, self.w_o, meta=ctx.meta)
 
     def _forward_prepared(self, x, ctx, cache):
         ops = self.rt.ops
@@ -281,6 +329,8 @@ class Attention(Mixer):
         return PendingSum((y,), vector=self.b_o) if self.out_bias else y
 
     def forward(self, x, ctx, cache):
+        if self.differential is not None:
+            return self._forward_differential(x, ctx, cache)
         if self.prepared:
             return self._forward_prepared(x, ctx, cache)
         ops = self.rt.ops

@@ -108,6 +108,20 @@ class PendingSum:
         return tuple(self.factors) if self.factors is not None else (1.0,) * len(self.terms)
 
 
+@dataclass
+class StreamMix:
+    """What a sublayer leaves pending where the residual is several streams side by side (float32 [T, streams * H]): with
+    y = ``result`` times ``scale`` (float32 [H], one factor per channel; None: none), stream k becomes sum_j ``mix``[j, k] x_j
+    + ``give``[k] y, all from the old streams (``mix`` float32 [streams, streams], from and to; ``give`` float32 [streams]).
+    ``result``: terms, weights, a factor and a vector.  The norm that follows (``Norm.forward_streams``) does this in
+    float32 in the pass that also reads and norms the new streams."""
+
+    result: "PendingSum"
+    scale: Optional[torch.Tensor]
+    mix: torch.Tensor
+    give: torch.Tensor
+
+
 def without_norms(ops, pending, ctx: "StepContext"):
     """The same sum with every normed term replaced by its normed rows, in the terms' type."""
     if not isinstance(pending, PendingSum) or pending.norms is None:
@@ -139,10 +153,12 @@ def join_terms(parts, mult: float = 1.0) -> "PendingSum":
 
 
 def apply_pending(ops, resid: torch.Tensor, delta, ctx: "StepContext") -> None:
-    """Adds what a block left pending (a tensor or a ``PendingSum``; None: nothing) into the float32 stream."""
+    """Adds what a block left pending (a tensor, a ``PendingSum`` or a ``StreamMix``; None: nothing) into the float32 stream(s)."""
     if delta is None:
         return
-    if isinstance(delta, PendingSum):
+    if isinstance(delta, StreamMix):
+        ops.stream_mix_norm(resid, delta.give.numel(), delta, None, None, 0.0, None, ctx.meta, ctx.T)
+    elif isinstance(delta, PendingSum):
         delta = without_norms(ops, delta, ctx)
         ops.sum_rmsnorm(resid, delta, None, 0.0, None, ctx.meta, ctx.T)
     else:
@@ -216,6 +232,12 @@ class Norm(Part):
         rows in the compute dtype.  With ``rows``: only those rows, residual left untouched."""
         raise NotImplementedError
 
+    def forward_streams(self, resid: torch.Tensor, streams: int, delta: Optional[StreamMix], read: Optional[torch.Tensor],
+                        ctx: StepContext, rows: Optional[torch.Tensor] = None, num_rows: int = 0) -> torch.Tensor:
+        """The same where the residual is several streams side by side ([T, streams * size]): takes ``delta`` into them and
+        returns the normed sum of the streams weighed by ``read`` (float32 [streams]; None: the plain sum)."""
+        raise NotImplementedError
+
 
 class SequenceFilter(Part):
     """What a sublayer reads instead of the residual rows themselves: a function of a request's rows over time that
@@ -281,6 +303,7 @@ class Block(Part):
     (that block, tensor), which the next block takes if it finds itself named."""
 
     mixer: Mixer
+    streams = 0  # how many streams side by side the block works on ([T, streams * H]); 0: the plain stream [T, H]
 
     def forward(self, resid: torch.Tensor, delta: Optional[torch.Tensor], ctx: StepContext,
                 cache: LayerCache) -> Optional[torch.Tensor]:

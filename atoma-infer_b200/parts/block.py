@@ -11,7 +11,7 @@ sequence filter (f1, f2: a short convolution over time, whose state the block ke
 None), ``names``.
 
 Parallel and sandwich arrangements: see ``ParallelBlock`` and ``SandwichBlock``.  Norms on the results alone: see
-``ResultNormBlock``.
+``ResultNormBlock``.  Several residual streams side by side: see ``HyperBlock``.
 """
 from __future__ import annotations
 
@@ -22,7 +22,7 @@ import torch
 
 from ..config.registry import part_class, register_part
 from ..weights.loader import TensorDecl
-from .base import Block, PendingSum, apply_pending, join_terms, without_norms
+from .base import Block, PendingSum, StreamMix, apply_pending, join_terms, without_norms
 
 _DEFAULT_NAMES = {"norm1": "input_layernorm", "mixer": "self_attn", "norm2": "post_attention_layernorm",
                   "feed_forward": "mlp"}
@@ -392,3 +392,80 @@ class ResultNormBlock(Block):
 
 
 register_part("block", "result_norm", ResultNormBlock)
+
+
+class HyperBlock(Block):
+    """Hyper-connections: the residual is ``streams`` streams x_1 .. x_s side by side (float32 [T, s * H]).  Sublayer q (1: mixer,
+    2: feed-forward) reads u = sum_j in_q[j] x_j through its norm, and with y = ls_q * sublayer(norm_q(u)) (ls_q: one factor per
+    channel) every stream is replaced, all at once: x_k <- sum_j mix_q[j, k] x_j + out_q[k] y.
+
+    The replacement is left pending (``StreamMix``); the next sublayer's norm, of this block or the one after it, takes it in
+    the pass that also reads and norms the new streams, in float32.  Parameters: ``norm``, ``mixer``, ``feed_forward`` (None: the
+    mixer alone), ``streams``, ``layer_scale`` (default True), ``names`` (suffixes behind the layer's prefix)."""
+
+    def __init__(self, params, prefix):
+        super().__init__(params, prefix)
+        names = {"norm1": "norm1", "norm2": "norm2", "mixer": "mix", "feed_forward": "mlp", "scale": ".ls", "streams": ".hc",
+                 "read": ".in", "give": ".out", "mix": ".mix", **(params.get("names") or {})}
+        self.names = names
+        mk = lambda fam, spec, name: part_class(fam, spec["kind"])(spec, f"{prefix}.{name}")  # noqa: E731
+        self.streams = int(params["streams"])
+        if self.streams < 1:
+            raise ValueError("a block of several streams has at least one")
+        self.layer_scale = bool(params.get("layer_scale", True))
+        self.norm1 = mk("norm", params["norm"], names["norm1"])
+        self.mixer = mk("mixer", params["mixer"], names["mixer"])
+        ff = params.get("feed_forward")
+        self.norm2 = mk("norm", params["norm"], names["norm2"]) if ff else None
+        self.feed_forward = mk("feed_forward", ff, names["feed_forward"]) if ff else None
+        self.width = self.norm1.size
+
+    def parts(self):
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.feed_forward) if p is not None]
+
+    def _sublayers(self):
+        return (1, 2) if self.feed_forward is not None else (1,)
+
+    def streamed_weights(self):
+        return self.mixer.streamed_weights() + (self.feed_forward.streamed_weights() if self.feed_forward else [])
+
+    def activation_width(self):
+        return max(p.activation_width() for p in self.parts())
+
+    def declare(self):
+        pre, n, s = self.prefix, self.names, self.streams
+        decls = [d for p in self.parts() for d in p.declare()]
+        for q in self._sublayers():
+            hc = f"{pre}{n['streams']}{q}"
+            decls += [TensorDecl(hc + n["read"], (s,), init="ones"), TensorDecl(hc + n["give"], (s,), init="ones"),
+                      TensorDecl(hc + n["mix"], (s, s), init="identity")]
+            if self.layer_scale:
+                decls.append(TensorDecl(f"{pre}{n['scale']}{q}", (self.width,), init="ones"))
+        return decls
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        for p in self.parts():
+            p.bind(tensors, rt)
+        n = self.names
+        f32 = lambda name: tensors[self.prefix + name].to(torch.float32).contiguous()  # noqa: E731  (exact widening)
+        hc = lambda q, what: f32(f"{n['streams']}{q}{n[what]}")  # noqa: E731
+        self.read = {q: hc(q, "read") for q in self._sublayers()}
+        self.give = {q: hc(q, "give") for q in self._sublayers()}
+        self.mix = {q: hc(q, "mix") for q in self._sublayers()}
+        self.scale = {q: f32(f"{n['scale']}{q}") if self.layer_scale else None for q in self._sublayers()}
+
+    def _pending(self, q, result, ctx):
+        result = without_norms(self.rt.ops, result, ctx)
+        return StreamMix(result if isinstance(result, PendingSum) else PendingSum((result,)), self.scale[q], self.mix[q], self.give[q])
+
+    def forward(self, resid, delta, ctx, cache):
+        h = self.norm1.forward_streams(resid, self.streams, delta, self.read[1], ctx)
+        delta = self._pending(1, self.mixer.forward(h, ctx, cache), ctx)
+        if self.feed_forward is None:
+            return delta
+        h = self.norm2.forward_streams(resid, self.streams, delta, self.read[2], ctx)
+        return self._pending(2, self.feed_forward.forward(h, ctx), ctx)
+
+
+register_part("block", "hyper", HyperBlock)

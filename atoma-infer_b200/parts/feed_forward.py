@@ -2,7 +2,7 @@
 (models/src/llama.rs:362-366, 370-374).  Gate and up are one stacked matrix here.
 
 Parameters: ``hidden``, ``intermediate``.  Checkpoint tensors:
-``<prefix>.{gate,up,down}_proj.weight``.
+``<prefix>.{gate,up,down}_proj.weight`` (other suffixes: ``names``).
 """
 from __future__ import annotations
 
@@ -18,23 +18,23 @@ class SwiGLU(FeedForward):
         super().__init__(params, prefix)
         self.hidden = int(params["hidden"])
         self.intermediate = int(params["intermediate"])
+        names = {"gate": ".gate_proj.weight", "up": ".up_proj.weight", "down": ".down_proj.weight", **(params.get("names") or {})}
+        self.t_gate, self.t_up, self.t_down = (prefix + names[k] for k in ("gate", "up", "down"))
 
     def activation_width(self):
         return 2 * self.intermediate
 
     def declare(self):
-        pre = self.prefix
         return [
-            TensorDecl(pre + ".gate_proj.weight", (self.intermediate, self.hidden)),
-            TensorDecl(pre + ".up_proj.weight", (self.intermediate, self.hidden)),
-            TensorDecl(pre + ".down_proj.weight", (self.hidden, self.intermediate)),
+            TensorDecl(self.t_gate, (self.intermediate, self.hidden)),
+            TensorDecl(self.t_up, (self.intermediate, self.hidden)),
+            TensorDecl(self.t_down, (self.hidden, self.intermediate)),
         ]
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
-        pre = self.prefix
-        self.w_gate_up = torch.cat([tensors[pre + ".gate_proj.weight"], tensors[pre + ".up_proj.weight"]], 0).contiguous()
-        self.w_down = tensors[pre + ".down_proj.weight"].contiguous()
+        self.w_gate_up = torch.cat([tensors[self.t_gate], tensors[self.t_up]], 0).contiguous()
+        self.w_down = tensors[self.t_down].contiguous()
 
     def streamed_weights(self):
         return [self.w_gate_up, self.w_down]

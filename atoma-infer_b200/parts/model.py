@@ -65,6 +65,7 @@ class ModelSpec:
     schedule: Optional[List[LayerRun]] = None       # None: every layer once, in order
     stream_tables: Dict[str, Tuple[int, int]] = field(default_factory=dict)  # checkpoint name -> [rows, hidden], see StreamAdd
     ignored_tensors: Tuple[str, ...] = ()           # globs a checkpoint may carry unused
+    streams: int = 0                                # residual streams side by side (0: one plain stream); every block carries as many
     max_position: int = 0
     eos_token_ids: Tuple[int, ...] = ()
 
@@ -73,7 +74,7 @@ class ModelSpec:
 
     def embedding_spec(self) -> Dict[str, Any]:
         return self.embedding or {"kind": "token", "vocab": self.vocab_size, "hidden": self.hidden_size,
-                                  "tensor": self.embedding_tensor}
+                                  "tensor": self.embedding_tensor, "copies": max(self.streams, 1)}
 
     def head_spec(self) -> Dict[str, Any]:
         return self.head or {"kind": "linear", "vocab": self.vocab_size, "hidden": self.hidden_size,
@@ -109,6 +110,11 @@ class DecoderModel:
         self.embedding, self.head = _build_ends(spec)
         self.final_norm = part_class("norm", spec.final_norm["kind"])(spec.final_norm, spec.final_norm_prefix)
         self.runs = spec.runs()
+        for i, blk in enumerate(self.blocks):
+            if blk.streams != spec.streams:
+                raise ValueError(f"the model carries {spec.streams} streams, the block of layer {i} {blk.streams}")
+        if spec.streams and any(r.before is not None for r in self.runs):
+            raise ValueError("additions to the stream before a run go with one plain stream")
         # Who owns which cache: a run without ``cache_of`` owns pages (and state) of its own, so a layer
         # that runs twice keeps two caches; a run with ``cache_of`` reads the pages of the first owning
         # run of that layer, which must come earlier in the schedule (its keys of this step are written).
@@ -223,7 +229,10 @@ class DecoderModel:
             if join is not None:
                 join()
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=self.rt.device)
-        h = self.final_norm.forward(resid, delta, ctx, rows=rows, num_rows=num_rows)
+        if self.spec.streams:  # the model's result is the sum of the streams
+            h = self.final_norm.forward_streams(resid, self.spec.streams, delta, None, ctx, rows=rows, num_rows=num_rows)
+        else:
+            h = self.final_norm.forward(resid, delta, ctx, rows=rows, num_rows=num_rows)
         logits = self.head.forward(h, ctx)
         join = getattr(self.rt.ops, "join_side_work", None)
         if join is not None:

@@ -8,7 +8,7 @@ stored weight is w - offset, i.e. 1.0 for weights kept around zero; ``tensor_suf
 
 ``forward_post`` is the norm AFTER the sum: resid <- norm(alpha * resid + delta), the
 normed rows being the new residual stream (float32, in place).  ``add_result`` is the norm of a sublayer's RESULT:
-resid <- resid + norm(result).
+resid <- resid + norm(result).  ``forward_streams`` reads several residual streams side by side.
 """
 from __future__ import annotations
 
@@ -61,6 +61,12 @@ class RMSNorm(Norm):
         self.rt.ops.sum_rmsnorm(resid, delta, self.weight, self.eps, out, ctx.meta, ctx.T, second=(other.weight, other.eps, out2))
         return out, out2
 
+    def forward_streams(self, resid, streams, delta, read, ctx, rows=None, num_rows=0):
+        n = num_rows if rows is not None else ctx.T
+        out = torch.empty((n, self.size), dtype=self.rt.dtype, device=resid.device)
+        self.rt.ops.stream_mix_norm(resid, streams, delta, read, self.weight, self.eps, out, ctx.meta, n, rows=rows)
+        return out
+
     def add_result(self, resid, result, ctx, out=None):
         """The norm of a sublayer's result: resid += norm(result), in one pass; ``result`` a tensor or a ``PendingSum`` (terms,
         weights, norms of single terms, a vector), ``out``: the new rows in the compute type."""
@@ -89,6 +95,9 @@ class LayerNorm(RMSNorm):
 
     def forward_post(self, resid, delta, alpha, ctx, keep=None, conv=None):
         raise NotImplementedError("a post-norm block goes with a root-mean-square norm")
+
+    def forward_streams(self, resid, streams, delta, read, ctx, rows=None, num_rows=0):
+        raise NotImplementedError("several streams go with a root-mean-square norm")
 
     def forward_pair(self, resid, delta, ctx, other):
         if other.size != self.size:

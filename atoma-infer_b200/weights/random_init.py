@@ -45,6 +45,10 @@ def random_tensor(decl: TensorDecl, seed: int, *, std: float, norm_jitter: float
         t = torch.ones(decl.shape, dtype=torch.float32, device=device)
         if norm_jitter:
             t = t + torch.randn(decl.shape, generator=g, dtype=torch.float32, device=device) * norm_jitter
+    elif decl.init == "identity":  # a square map around the identity
+        t = torch.eye(decl.shape[0], dtype=torch.float32, device=device)
+        if norm_jitter:
+            t = t + torch.randn(decl.shape, generator=g, dtype=torch.float32, device=device) * norm_jitter
     elif decl.init in ("zeros", "jitter"):  # jitter: N(0, norm_jitter), a norm weight that is stored around zero
         t = torch.zeros(decl.shape, dtype=torch.float32, device=device)
         if decl.init == "jitter" and norm_jitter:

@@ -12,6 +12,7 @@ import plain_bumolix as PB
 import plain_dosovik as PD
 import plain_kavotar as PV
 import plain_kulivik as PK
+import plain_tupunex as PX
 import plain_tutezen as PT
 import plain_llama as P
 from atoma_infer_b200.csrc.ops import (META_BT_OFFSET, META_BT_STRIDE, META_NUM_ROWS, META_NUM_TOKENS, STATUS_WORDS,
@@ -48,13 +49,13 @@ class HostOps:
     def fast_attention(self, *a):
         return False
 
-    def embed(self, tokens, table, resid, meta, T, scale=1.0):
+    def embed(self, tokens, table, resid, meta, T, scale=1.0, copies=1):
         self._count()
         n = int(meta[META_NUM_TOKENS])
         tok = tokens[:n].long()
         neg = tok < 0
         tok = torch.where(neg, self.last_tokens[(-tok - 1).clamp(min=0)].long(), tok)
-        resid[:n] = scale * table[tok].float()
+        resid[:n] = (scale * table[tok].float()).repeat(1, copies)
 
     def add_rmsnorm(self, resid, delta, w, eps, out, meta, n, rows=None):
         self._count()
@@ -334,11 +335,12 @@ class HostOps:
         n = int(meta[META_NUM_TOKENS])
         y = torch.einsum("thk,hnk->thn", x[:n].float(), w.float())
         if gate is not None:
-            y = y * torch.sigmoid(gate[:n].float())
+            g = torch.sigmoid(gate[:n].float())
+            y = y * (g if g.dim() == 3 else g[:, :, None])
         out[:n] = y.to(out.dtype)
 
     def latent_rows(self, q_rot, q_abs, dkv, norm_w, eps, ctx, cache, group, q_out, *, heads, kv_rank, rot_dim, padded,
-                    page_size, num_pages, store, inv_freq=None, rotary_dims=0):
+                    page_size, num_pages, store, inv_freq=None, rotary_dims=0, halves=False):
         self._count()
         meta = ctx.meta
         n = int(meta[META_NUM_TOKENS])
@@ -353,9 +355,11 @@ class HostOps:
                 ang = ang.unsqueeze(1)
             cs, sn = torch.cos(ang), torch.sin(ang)
             o = v.clone()
-            a, b = v[..., 0:rotary_dims:2], v[..., 1:rotary_dims:2]
-            o[..., 0:rotary_dims:2] = a * cs - b * sn
-            o[..., 1:rotary_dims:2] = b * cs + a * sn
+            half = rotary_dims // 2
+            low, high = (slice(0, half), slice(half, rotary_dims)) if halves else (slice(0, rotary_dims, 2), slice(1, rotary_dims, 2))
+            a, b = v[..., low], v[..., high]
+            o[..., low] = a * cs - b * sn
+            o[..., high] = b * cs + a * sn
             return o
 
         c = PT.rms_divide(dkv[:n, :kv_rank].float(), eps) * norm_w
@@ -575,6 +579,72 @@ class HostOps:
         count, keep = groups or (1, 1)
         idx, wt = PV.choose(torch.sigmoid(h[:n].float() @ w_router.T).double(), correction, ids.shape[1], {"count": count, "keep": keep})
         ids[:n], wts[:n] = idx.to(torch.int32), wt.float()
+
+    # -- several streams side by side, attention as the difference of two maps
+    def stream_mix_norm(self, resid, streams, pending, read, w, eps, out, meta, n, rows=None):
+        self._count()
+        idx = torch.arange(int(meta[META_NUM_TOKENS])) if rows is None else rows[:int(meta[META_NUM_ROWS])].long()
+        x = resid[idx].view(len(idx), streams, -1).clone()
+        if pending is not None:
+            r = pending.result
+            y = torch.zeros_like(x[:, 0])
+            for t, f in zip(r.terms, r.weights()):
+                y = y + f * t[idx].float()
+            y = r.mult * y
+            if r.vector is not None:
+                y = y + r.vector
+            if pending.scale is not None:
+                y = y * pending.scale
+            x = torch.einsum("tjw,jk->tkw", x, pending.mix) + pending.give[None, :, None] * y[:, None, :]
+            if rows is None:
+                resid[idx] = x.reshape(len(idx), -1)
+        if out is not None:
+            u = torch.einsum("tjw,j->tw", x, read) if read is not None else x.sum(1)
+            out[:len(idx)] = P.rms_norm(u, w, eps).to(out.dtype)
+
+    def map_rows(self, qkv, ctx, cache, group, q_out, *, heads, kv_heads, maps, d, dv, dp, page_size, num_pages, store_kv, bias=None,
+                 conv_w=None, ring=None):
+        self._count()
+        meta = ctx.meta
+        n, N = int(meta[META_NUM_TOKENS]), (heads + kv_heads) * maps * d + kv_heads * dv
+        off, stride = int(meta[META_BT_OFFSET + group]), int(meta[META_BT_STRIDE + group])
+        add = bias if bias is not None else torch.zeros(N)
+        taps = conv_w.shape[0] if conv_w is not None else 0
+        R = max(taps - 1, 0)
+        for _, a, b, slot in self._entries(ctx):
+            p0 = int(ctx.positions[a])
+            before = [ring[slot, p % R] + add if p >= 0 else torch.zeros(N) for p in range(p0 - R, p0)]
+            rows = torch.stack(before + list(qkv[a:b].float() + add))
+            if taps:
+                rows = sum(conv_w[j] * rows[j:j + b - a] for j in range(taps))
+            for t, row in zip(range(a, b), rows):
+                p = int(ctx.positions[t])
+                q = row[:heads * maps * d].view(heads, maps, d)
+                k = row[heads * maps * d:(heads + kv_heads) * maps * d].view(kv_heads, maps * d)
+                v = row[(heads + kv_heads) * maps * d:].view(kv_heads, dv)
+                wide = torch.zeros(heads, maps, dp)
+                for m in range(maps):
+                    wide[:, m, m * d:(m + 1) * d] = q[:, m]
+                q_out[t] = wide.reshape(-1).to(q_out.dtype)
+                if store_kv:
+                    page = int(meta[off + int(ctx.token_entry[t]) * stride + p // page_size])
+                    if not 0 < page < num_pages:
+                        self.status[1] = t + 1
+                        continue
+                    cache[page, :, :, p % page_size] = 0
+                    cache[page, 0, :, p % page_size, :maps * d] = k.to(cache.dtype)
+                    cache[page, 1, :, p % page_size, :dv] = v.to(cache.dtype)
+            for t in range(max(a, b - R), b) if R else ():
+                ring[slot, int(ctx.positions[t]) % R] = qkv[t].float()
+
+    def map_difference(self, a, gate, lam, factor, eps, out, meta, *, heads, dp):
+        self._count()
+        n, dv = int(meta[META_NUM_TOKENS]), out.shape[1] // heads
+        m = a[:n].float().view(n, heads, 2, dp)[..., :dv]
+        o = PX.unit(m[:, :, 0] - lam * m[:, :, 1], eps) * factor
+        if gate is not None:
+            o = o * torch.sigmoid(gate[:n].float())[:, :, None]
+        out[:n] = o.reshape(n, -1).to(out.dtype)
 
     def sample(self, logits, temperature, top_k, top_p, seed, step, out, num_rows=None, slots=None):
         self._count()
