@@ -1,6 +1,8 @@
 // Kernels of differential attention: the rows that enter it (biases, a short causal convolution over time, the layout in
 // which the attention kernels see two maps over the same values) and the difference of the two maps behind it.
 // Storage is float32 or bfloat16, arithmetic float32.
+#include <type_traits>
+
 #include "common.cuh"
 
 // V neighbouring elements, widened; V = 8 (bfloat16 only) and 4 take one access (16-byte rows), 1 takes any address.
@@ -52,6 +54,18 @@ __device__ __forceinline__ void store_row(T* p, const float (&v)[V]) {
     }
 }
 
+// V elements as they are stored, in one register vector where they make one (16 or 8 bytes).
+template <typename T, int V>
+struct RawRow {
+    using type = typename std::conditional<V * sizeof(T) == 16, uint4, typename std::conditional<V * sizeof(T) == 8, uint2, T>::type>::type;
+};
+template <typename T, int V>
+__device__ __forceinline__ void widen(const typename RawRow<T, V>::type& raw, float (&v)[V]) {
+    const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int k = 0; k < V; ++k) v[k] = to_float(e[k]);
+}
+
 // ----------------------------------------------------------------------------- the rows
 // A token's projected row u is [q: heads * M * d | k: kv_heads * M * d | v: kv_heads * dv] (M maps; the row may be the first
 // part of a wider one).  Per channel r_t = sum_j w[j] * (u_(t - taps + 1 + j) + bias), terms before the request's start
@@ -63,7 +77,7 @@ __device__ __forceinline__ void store_row(T* p, const float (&v)[V]) {
 // so the thread that has read a channel's ring also writes the new row's place; otherwise map_rows_save writes it later.
 //
 // A thread owns V neighbouring channels of one output head and walks the block's tokens with its weights and biases in
-// registers; a row that it reads again, for the tokens behind it, comes from the nearest cache.
+// registers, four tokens at a time where their rows lie side by side.
 #define MAP_ROWS_TOK 16
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(128)
@@ -121,38 +135,68 @@ map_rows_kernel(const T* __restrict__ u, long long u_stride, const float* __rest
     __syncthreads();
     if (!mine) return;
     const size_t head_block = (size_t)page_size * dp, kv_block = (size_t)kv_heads * head_block;
-    for (int i = 0; i < tn; ++i) {
-        const int t = t0 + i, p = s_pos[i], first = s_first[i];
-        float r[V];
-#pragma unroll
-        for (int k = 0; k < V; ++k) r[k] = 0.f;
-        if (ch >= 0) {
-            float cur[V];
-            load_row<T, V>(u + (size_t)t * u_stride + ch, cur);
-#pragma unroll
-            for (int j = 0; j < R; ++j) {  // oldest tap first: a fixed order
-                const int back = R - j;
-                if (p - back < 0) continue;
-                float v[V];
-                if (t - back >= first) load_row<T, V>(u + (size_t)(t - back) * u_stride + ch, v);
-                else load_f32<V>(ring + (size_t)s_slot[i] * slot_stride + (size_t)((p - back) % RR) * N + ch, v);
-#pragma unroll
-                for (int k = 0; k < V; ++k) r[k] = fmaf(wt[j][k], v[k] + b[k], r[k]);
-            }
-            if (R > 0 && save_own) {
-                float* dst = ring + (size_t)s_slot[i] * slot_stride + (size_t)(p % RR) * N + ch;
-#pragma unroll
-                for (int k = 0; k < V; ++k) dst[k] = cur[k];
-            }
-#pragma unroll
-            for (int k = 0; k < V; ++k) r[k] = TAPS > 0 ? fmaf(wt[TAPS > 0 ? TAPS - 1 : 0][k], cur[k] + b[k], r[k]) : cur[k] + b[k];
-        }
+    auto put = [&](int i, const float (&r)[V]) {
         if (kind == 0) {
-            store_row<T, V>(q_out + ((size_t)t * nq + h) * dp + at, r);
+            store_row<T, V>(q_out + ((size_t)(t0 + i) * nq + h) * dp + at, r);
         } else if (s_page[i] > 0) {
             T* page = cache + (size_t)s_page[i] * 2 * kv_block + (kind == 2 ? kv_block : 0);
-            store_row<T, V>(page + (size_t)h * head_block + (size_t)(p % page_size) * dp + at, r);
+            store_row<T, V>(page + (size_t)h * head_block + (size_t)(s_pos[i] % page_size) * dp + at, r);
         }
+    };
+    constexpr int GROUP = 4;
+    for (int i = 0; i < tn;) {
+        float r[V];
+        if (ch < 0) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) r[k] = 0.f;
+            put(i++, r);
+            continue;
+        }
+        const T* row = u + (size_t)(t0 + i) * u_stride + ch;
+        // four tokens whose rows, and the rows before them, are all of one request and of this step: every row is loaded once
+        if (i + GROUP <= tn && s_first[i + GROUP - 1] <= t0 + i - R) {
+            typename RawRow<T, V>::type raw[GROUP + R];
+#pragma unroll
+            for (int j = 0; j < GROUP + R; ++j) raw[j] = *reinterpret_cast<const typename RawRow<T, V>::type*>(row + (long long)(j - R) * u_stride);
+#pragma unroll
+            for (int g = 0; g < GROUP; ++g) {
+#pragma unroll
+                for (int k = 0; k < V; ++k) r[k] = 0.f;
+#pragma unroll
+                for (int j = 0; j <= R; ++j) {
+                    float v[V];
+                    widen<T, V>(raw[g + j], v);
+#pragma unroll
+                    for (int k = 0; k < V; ++k) r[k] = TAPS > 0 ? fmaf(wt[j][k], v[k] + b[k], r[k]) : v[k] + b[k];
+                }
+                put(i + g, r);
+            }
+            i += GROUP;
+            continue;
+        }
+        const int t = t0 + i, p = s_pos[i], first = s_first[i];
+        float cur[V];
+        load_row<T, V>(row, cur);
+#pragma unroll
+        for (int k = 0; k < V; ++k) r[k] = 0.f;
+#pragma unroll
+        for (int j = 0; j < R; ++j) {  // oldest tap first: a fixed order
+            const int back = R - j;
+            if (p - back < 0) continue;
+            float v[V];
+            if (t - back >= first) load_row<T, V>(u + (size_t)(t - back) * u_stride + ch, v);
+            else load_f32<V>(ring + (size_t)s_slot[i] * slot_stride + (size_t)((p - back) % RR) * N + ch, v);
+#pragma unroll
+            for (int k = 0; k < V; ++k) r[k] = fmaf(wt[j][k], v[k] + b[k], r[k]);
+        }
+        if (R > 0 && save_own) {
+            float* dst = ring + (size_t)s_slot[i] * slot_stride + (size_t)(p % RR) * N + ch;
+#pragma unroll
+            for (int k = 0; k < V; ++k) dst[k] = cur[k];
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) r[k] = TAPS > 0 ? fmaf(wt[TAPS > 0 ? TAPS - 1 : 0][k], cur[k] + b[k], r[k]) : cur[k] + b[k];
+        put(i++, r);
     }
 }
 

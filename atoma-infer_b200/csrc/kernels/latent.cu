@@ -102,10 +102,80 @@ head_linear_kernel(const T* __restrict__ x, long long xs_t, long long xs_h, cons
     }
 }
 
+// Few rows of bfloat16 (a decode step): a block takes 8 tokens x 16 outputs of one head, eight lanes share an output.  A lane's
+// pieces of the weight row (16 bytes each, every eighth piece; up to P of them, K <= 64 P) are in registers before the
+// dependency wait; the tokens' rows wait in shared memory as they are; the eight lanes' sums of the eight tokens are
+// exchanged so that lane m ends with token m's.  The order of a sum depends on K alone.
+template <int P>
+__global__ void __launch_bounds__(128)
+head_linear_few_kernel(const __nv_bfloat16* __restrict__ x, long long xs_t, long long xs_h, const __nv_bfloat16* __restrict__ w,
+                       __nv_bfloat16* __restrict__ y, long long ys_t, long long ys_h, const __nv_bfloat16* __restrict__ gate, long long gs_t,
+                       long long gs_h, int gate_per_head, const int* __restrict__ meta, int K, int N) {
+    __shared__ __align__(16) __nv_bfloat16 xs[8][64 * P];
+    const int tid = threadIdx.x, lane = tid & 7, t0 = blockIdx.x * 8, h = blockIdx.y, n = blockIdx.z * 16 + tid / 8;
+    const int rows = min(8, meta[META_NUM_TOKENS] - t0), pieces = K / 8;
+    uint4 wr[P];
+    const __nv_bfloat16* wrow = w + ((size_t)h * N + min(n, N - 1)) * K;
+#pragma unroll
+    for (int j = 0; j < P; ++j) wr[j] = lane + 8 * j < pieces ? *reinterpret_cast<const uint4*>(wrow + (lane + 8 * j) * 8) : make_uint4(0, 0, 0, 0);
+    pdl_wait();
+    pdl_launch_dependents();
+    if (rows <= 0) return;
+    for (int m = 0; m < 8; ++m)
+        for (int k = tid; k < 64 * P; k += 128)
+            xs[m][k] = m < rows && k < K ? x[(size_t)(t0 + m) * xs_t + (size_t)h * xs_h + k] : __float2bfloat16(0.f);
+    __syncthreads();
+    float acc[8];
+#pragma unroll
+    for (int m = 0; m < 8; ++m) acc[m] = 0.f;
+#pragma unroll
+    for (int j = 0; j < P; ++j) {
+        float wv[8];
+        const __nv_bfloat16* we = reinterpret_cast<const __nv_bfloat16*>(&wr[j]);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) wv[k] = to_float(we[k]);
+#pragma unroll
+        for (int m = 0; m < 8; ++m) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(&xs[m][(lane + 8 * j) * 8]);
+            const __nv_bfloat16* xe = reinterpret_cast<const __nv_bfloat16*>(&raw);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) acc[m] = fmaf(to_float(xe[k]), wv[k], acc[m]);
+        }
+    }
+    // halving: after the step with distance s a lane holds the sums of the tokens that agree with it in the bits seen so far
+    float four[4], two[2];
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+        const float keep = lane & 4 ? acc[m + 4] : acc[m], give = lane & 4 ? acc[m] : acc[m + 4];
+        four[m] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+        const float keep = lane & 2 ? four[m + 2] : four[m], give = lane & 2 ? four[m] : four[m + 2];
+        two[m] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+    }
+    float v = (lane & 1 ? two[1] : two[0]) + __shfl_xor_sync(0xffffffffu, lane & 1 ? two[0] : two[1], 1);
+    if (lane >= rows || n >= N) return;
+    if (gate) v = v / (1.f + expf(-to_float(gate[(size_t)(t0 + lane) * gs_t + (size_t)h * gs_h + (gate_per_head ? 0 : n)])));
+    y[(size_t)(t0 + lane) * ys_t + (size_t)h * ys_h + n] = __float2bfloat16_rn(v);
+}
+
 extern "C" int head_linear(const void* x, long long xs_t, long long xs_h, const void* w, void* y, long long ys_t,
                            long long ys_h, const void* gate, long long gs_t, long long gs_h, int gate_per_head, int dtype, const int* meta,
                            int T, int heads, int K, int N, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (dtype == DT_BF16 && T < 64 && K % 8 == 0 && K <= 512 && ((uintptr_t)w & 15) == 0) {
+        const dim3 few((T + 7) / 8, heads, (N + 15) / 16);
+#define FEW_CASE(P)                                                                                                              \
+        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, head_linear_few_kernel<P>, few, 128, 0, stream, (const __nv_bfloat16*)x, xs_t, xs_h, \
+                                      (const __nv_bfloat16*)w, (__nv_bfloat16*)y, ys_t, ys_h, (const __nv_bfloat16*)gate, gs_t, gs_h, gate_per_head, \
+                                      meta, K, N)
+        if (K <= 64) FEW_CASE(1);
+        if (K <= 128) FEW_CASE(2);
+        if (K <= 256) FEW_CASE(4);
+        FEW_CASE(8);
+#undef FEW_CASE
+    }
     const int tn = N <= 32 ? 32 : (N <= 64 ? 64 : HL_TN);  // few outputs a head: smaller blocks, all of their threads at work
     dim3 grid((T + HL_TM - 1) / HL_TM, heads, (N + tn - 1) / tn);
     const int elem = dtype == DT_F32 ? 4 : 2;
@@ -167,8 +237,8 @@ extern "C" int sigmoid_gate(void* y, long long ys_t, long long ys_h, const void*
 
 // ----------------------------------------------------------------------------- the rows of latent attention
 // Per token: the cached vector [c | rotated key part | zeros] with c = dkv[:rank] * rsqrt(mean(.^2) + eps) * norm_w
-// goes to the key plane and to the value plane of the token's page (one key/value head of D elements); the queries
-// become [q_abs[h] | rotated q_rot[h] | zeros] of D elements a head.  Rotation: of the first `rot` dimensions of a
+// goes to the key plane and to the value plane of the token's page (one key/value head of D elements); the queries, whose
+// first `rank` elements are in place, get [rotated q_rot[h] | zeros] behind them, D elements a head.  Rotation: of the first `rot` dimensions of a
 // rotated part, 2i pairs with 2i + 1 (`halves`: i with i + rot / 2), by the angle position * inv_freq[i] (float32 product, sincosf).
 // Two neighbouring elements at once (the address a multiple of two elements): a rotation's pair.
 __device__ __forceinline__ void load2(const float* p, float& a, float& b) { const float2 t = *reinterpret_cast<const float2*>(p); a = t.x; b = t.y; }
@@ -216,64 +286,62 @@ __device__ __forceinline__ float turned1(const T* p, int j, int rot, int halves,
     return low ? lo : hi;
 }
 
-// A block takes one token and `hpb` of its heads + 1 jobs: job h < heads lays out query head h, job `heads` makes the
-// cached vector.  Few tokens: a job a block; many: all of a token's jobs in one block, which takes the cosines and
-// sines once.  `pairs`: sizes, strides and addresses are even, so a thread takes a rotation's pair with one access.
+// A block takes one token.  `pairs`: sizes, strides and addresses are even, so a thread takes two neighbouring elements with
+// one access.
 template <typename T>
-__global__ void __launch_bounds__(256)
-latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, const T* __restrict__ q_abs,
-                   const T* __restrict__ dkv, long long dkv_stride, const float* __restrict__ norm_w, float eps,
-                   const int* __restrict__ positions, const int* __restrict__ token_entry, const int* __restrict__ meta,
-                   int group, const float* __restrict__ inv_freq, int rot, int halves, T* __restrict__ q_out, T* __restrict__ cache,
-                   int heads, int rank, int rdim, int D, int page_size, int num_pages, int store, int pairs, int hpb,
-                   int* __restrict__ status) {
+__global__ void __launch_bounds__(128)
+latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, const T* __restrict__ dkv, long long dkv_stride,
+                   const float* __restrict__ norm_w, float eps, const int* __restrict__ positions,
+                   const int* __restrict__ token_entry, const int* __restrict__ meta, int group,
+                   const float* __restrict__ inv_freq, int rot, int halves, T* __restrict__ q_out, T* __restrict__ cache,
+                   int heads, int rank, int rdim, int D, int page_size, int num_pages, int store, int pairs, int* __restrict__ status) {
     __shared__ float red[33];
     extern __shared__ float cs[];  // rot / 2 cosines, rot / 2 sines
     float* sn = cs + rot / 2;
     // The step's metadata is written by no kernel of the step: it is read before the wait.
-    const int t = blockIdx.x, h_first = blockIdx.y * hpb, h_end = min(heads + (store ? 1 : 0), h_first + hpb), tid = threadIdx.x;
-    const bool live = t < meta[META_NUM_TOKENS] && h_first < h_end;
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const bool live = t < meta[META_NUM_TOKENS];
     const int p = live ? positions[t] : 0;
     int page = 0;
-    if (live && h_end == heads + 1) page = (meta + meta[META_BT_OFFSET + group] + (size_t)token_entry[t] * meta[META_BT_STRIDE + group])[p / page_size];
+    if (live && store) page = (meta + meta[META_BT_OFFSET + group] + (size_t)token_entry[t] * meta[META_BT_STRIDE + group])[p / page_size];
     if (live)
         for (int i = tid; i < rot / 2; i += blockDim.x) sincosf((float)p * inv_freq[i], &sn[i], &cs[i]);
     pdl_wait();
     pdl_launch_dependents();
     if (!live) return;
     __syncthreads();  // the cosines and sines are written
-    for (int h = h_first; h < min(h_end, heads); ++h) {
-        const T* qr = q_rot + (size_t)t * qs_t + (size_t)h * qs_h;
-        const T* qa = q_abs + ((size_t)t * heads + h) * rank;
-        T* dst = q_out + ((size_t)t * heads + h) * D;
-        if (pairs) {
-            for (int i = tid * 2; i < D; i += blockDim.x * 2) {
-                float a = 0.f, b = 0.f;
-                if (i < rank) {
-                    load2(qa + i, a, b);
-                } else if (i < rank + rdim) {
-                    turned2(qr, i - rank, rot, halves, cs, sn, a, b);
-                }
-                store2(dst + i, a, b);
-            }
-            continue;
+    const int tail = D - rank;
+    const T* qt = q_rot + (size_t)t * qs_t;
+    T* qo = q_out + (size_t)t * heads * D + rank;
+    if (pairs) {
+        const int per = tail / 2;
+        for (int it = tid; it < heads * per; it += blockDim.x) {
+            const int h = it / per, j = (it % per) * 2;
+            float a = 0.f, b = 0.f;
+            if (j < rdim) turned2(qt + (size_t)h * qs_h, j, rot, halves, cs, sn, a, b);
+            store2(qo + (size_t)h * D + j, a, b);
         }
-        for (int i = tid; i < D; i += blockDim.x) {
-            float v = 0.f;
-            if (i < rank) {
-                v = to_float(qa[i]);
-            } else if (i < rank + rdim) {
-                v = turned1(qr, i - rank, rot, halves, cs, sn);
-            }
-            dst[i] = from_float<T>(v);
+    } else {
+        for (int it = tid; it < heads * tail; it += blockDim.x) {
+            const int h = it / tail, j = it % tail;
+            qo[(size_t)h * D + j] = from_float<T>(j < rdim ? turned1(qt + (size_t)h * qs_h, j, rot, halves, cs, sn) : 0.f);
         }
     }
-    if (h_end != heads + 1) return;
+    if (!store) return;
     const T* kv = dkv + (size_t)t * dkv_stride;
     float ss = 0.f;
-    for (int i = tid; i < rank; i += blockDim.x) {
-        const float v = to_float(kv[i]);
-        ss = fmaf(v, v, ss);
+    if (pairs) {
+        for (int i = tid * 2; i < rank; i += blockDim.x * 2) {
+            float a, b;
+            load2(kv + i, a, b);
+            ss = fmaf(a, a, ss);
+            ss = fmaf(b, b, ss);
+        }
+    } else {
+        for (int i = tid; i < rank; i += blockDim.x) {
+            const float v = to_float(kv[i]);
+            ss = fmaf(v, v, ss);
+        }
     }
     ss = block_sum(ss, red);
     const float inv = rsqrtf(ss / (float)rank + eps);
@@ -301,38 +369,30 @@ latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, 
     }
     for (int i = tid; i < D; i += blockDim.x) {
         float v = 0.f;
-        if (i < rank) {
-            v = to_float(kv[i]) * inv * norm_w[i];
-        } else if (i < rank + rdim) {
-            v = turned1(kv + rank, i - rank, rot, halves, cs, sn);
-        }
+        if (i < rank) v = to_float(kv[i]) * inv * norm_w[i];
+        else if (i < rank + rdim) v = turned1(kv + rank, i - rank, rot, halves, cs, sn);
         const T o = from_float<T>(v);
         kdst[i] = o;
         vdst[i] = o;
     }
 }
 
-extern "C" int latent_rows(const void* q_rot, long long qs_t, long long qs_h, const void* q_abs, const void* dkv,
-                           long long dkv_stride, const float* norm_w, float eps, const int* positions, const int* token_entry,
-                           const int* meta, int group, const float* inv_freq, int rot, int halves, void* q_out, void* cache, int dtype,
-                           int T, int heads, int rank, int rdim, int D, int page_size, int num_pages, int store, int* status,
-                           cudaStream_t stream) {
+extern "C" int latent_rows(const void* q_rot, long long qs_t, long long qs_h, const void* dkv, long long dkv_stride, const float* norm_w,
+                           float eps, const int* positions, const int* token_entry, const int* meta, int group, const float* inv_freq,
+                           int rot, int halves, void* q_out, void* cache, int dtype, int T, int heads, int rank, int rdim, int D,
+                           int page_size, int num_pages, int store, int* status, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (rot % 2 || rot > rdim || rank + rdim > D || (rot && !inv_freq)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)rot * sizeof(float);
     const int elem = dtype == DT_F32 ? 4 : 2;
-    const int pairs = rank % 2 == 0 && rdim % 2 == 0 && D % 2 == 0 && (!halves || rot % 4 == 0) && qs_t % 2 == 0 && qs_h % 2 == 0 && dkv_stride % 2 == 0 &&
-                      (((uintptr_t)q_rot | (uintptr_t)q_abs | (uintptr_t)dkv | (uintptr_t)q_out | (uintptr_t)cache) % (2 * elem)) == 0;
-    const int hpb = T >= 512 ? heads + 1 : 1, threads = hpb > 1 ? 256 : 128;
-    const dim3 grid(T, (heads + 1 + hpb - 1) / hpb);
+    const int pairs = rank % 2 == 0 && rdim % 2 == 0 && D % 2 == 0 && (!halves || rot % 4 == 0) && qs_t % 2 == 0 && qs_h % 2 == 0 &&
+                      dkv_stride % 2 == 0 && (((uintptr_t)q_rot | (uintptr_t)dkv | (uintptr_t)q_out | (uintptr_t)cache) % (2 * elem)) == 0;
     if (dtype == DT_F32)
-        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<float>, grid, threads, smem, stream, (const float*)q_rot, qs_t,
-                                      qs_h, (const float*)q_abs, (const float*)dkv, dkv_stride, norm_w, eps, positions, token_entry,
-                                      meta, group, inv_freq, rot, halves, (float*)q_out, (float*)cache, heads, rank, rdim, D, page_size,
-                                      num_pages, store, pairs, hpb, status);
-    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<__nv_bfloat16>, grid, threads, smem, stream,
-                                  (const __nv_bfloat16*)q_rot, qs_t, qs_h, (const __nv_bfloat16*)q_abs, (const __nv_bfloat16*)dkv,
-                                  dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq, rot, halves,
-                                  (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, heads, rank, rdim, D, page_size, num_pages, store,
-                                  pairs, hpb, status);
+        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<float>, T, 128, smem, stream, (const float*)q_rot, qs_t, qs_h,
+                                      (const float*)dkv, dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq, rot, halves,
+                                      (float*)q_out, (float*)cache, heads, rank, rdim, D, page_size, num_pages, store, pairs, status);
+    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<__nv_bfloat16>, T, 128, smem, stream, (const __nv_bfloat16*)q_rot,
+                                  qs_t, qs_h, (const __nv_bfloat16*)dkv, dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq,
+                                  rot, halves, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, heads, rank, rdim, D, page_size, num_pages, store,
+                                  pairs, status);
 }

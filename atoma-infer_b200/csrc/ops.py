@@ -762,7 +762,7 @@ class CudaOps:
         elif gate is not None:
             gp, gt, gh = self._heads(gate, "head_linear")
         if x.dtype == torch.bfloat16 and T >= self.HEAD_LINEAR_LIBRARY_ROWS:
-            out.copy_(torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1))
+            torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))  # (written in place: a row stride is all it needs)
             if per_head:
                 self.head_gate(out, gate, meta)
             elif gate is not None:
@@ -773,18 +773,16 @@ class CudaOps:
         self._check(lib.head_linear(xp, xt, xh, _p(w), op, ot, oh, gp, gt, gh, int(per_head), _code(x), _p(meta), T, heads, K, N,
                                     self._stream()), "head_linear")
 
-    def latent_rows(self, q_rot, q_abs, dkv, norm_w, eps: float, ctx, cache_layer, group: int, q_out, *, heads: int,
+    def latent_rows(self, q_rot, dkv, norm_w, eps: float, ctx, cache_layer, group: int, q_out, *, heads: int,
                     kv_rank: int, rot_dim: int, padded: int, page_size: int, num_pages: int, store: bool, inv_freq=None,
                     rotary_dims: int = 0, halves: bool = False):
         """The rows of latent attention.  The cached vector [rmsnorm(dkv[:kv_rank]) * norm_w | rotated dkv[kv_rank:] |
-        zeros] of ``padded`` elements goes to the key plane and the value plane of the token's page; the queries become
-        [q_abs[h] | rotated q_rot[h] | zeros] in ``q_out`` [T, heads * padded].  Rotation: of the first ``rotary_dims``
+        zeros] of ``padded`` elements goes to the key plane and the value plane of the token's page; the queries in ``q_out``
+        [T, heads * padded], whose first kv_rank elements a head are in place, get [rotated q_rot[h] | zeros] behind them.  Rotation: of the first ``rotary_dims``
         dimensions, 2i pairs with 2i + 1 (``halves``: i with i + rotary_dims / 2), angle position * inv_freq[i]."""
         qp, qt, qh = self._heads(q_rot, "latent_rows")
         dp, ds = self._rows(dkv, "latent_rows")
-        if not q_abs.is_contiguous():
-            raise KernelError("latent_rows: q_abs must be contiguous")
-        self._check(self._mixers().latent_rows(qp, qt, qh, _p(q_abs), dp, ds, _p(norm_w), ctypes.c_float(eps), _p(ctx.positions),
+        self._check(self._mixers().latent_rows(qp, qt, qh, dp, ds, _p(norm_w), ctypes.c_float(eps), _p(ctx.positions),
                                                _p(ctx.token_entry), _p(ctx.meta), max(group, 0), _p(inv_freq),
                                                int(rotary_dims) if inv_freq is not None else 0, int(halves), _p(q_out), _p(cache_layer),
                                                _code(q_out), ctx.T, heads, kv_rank, rot_dim, padded, page_size, num_pages,

@@ -62,7 +62,7 @@ class LatentAttention(Mixer):
         self.a_rows = -(-(self.first + self.latent + self.gate_rows) // 8) * 8
 
     def activation_width(self):
-        return max(self.a_rows, 2 * self.heads * self.padded + self.heads * self.kv_rank)
+        return max(self.a_rows, 2 * self.heads * self.padded)
 
     def cache_need(self):
         return CacheNeed.kv(1, self.padded, self.window)
@@ -117,10 +117,9 @@ class LatentAttention(Mixer):
             q = ops.linear(cq, self.w_uq, meta=ctx.meta).view(T, H, self.q_head)
         else:
             q = a[:, :self.first].view(T, H, self.q_head)
-        q_abs = torch.empty((T, H, self.kv_rank), dtype=x.dtype, device=x.device)
-        ops.head_linear(q[:, :, :self.dim], self.w_uk_t, q_abs, ctx.meta)
         q_full = torch.empty((T, H * D), dtype=x.dtype, device=x.device)
-        ops.latent_rows(q[:, :, self.dim:], q_abs, a[:, self.first:self.first + self.latent], self.dkv_norm, self.eps, ctx,
+        ops.head_linear(q[:, :, :self.dim], self.w_uk_t, q_full.view(T, H, D)[:, :, :self.kv_rank], ctx.meta)
+        ops.latent_rows(q[:, :, self.dim:], a[:, self.first:self.first + self.latent], self.dkv_norm, self.eps, ctx,
                         cache.pages, cache.group, q_full, heads=H, kv_rank=self.kv_rank, rot_dim=self.rot_dim, padded=D,
                         page_size=cache.page_size, num_pages=cache.num_pages,
                         store=cache.writes and cache.pages is not None, inv_freq=self.inv_freq, rotary_dims=self.rotary_dims,

@@ -80,7 +80,13 @@ class RotaryEncoding(PositionEncoding):
 
 
 class NoPositionEncoding(RotaryEncoding):
-    """Keys and queries as they are: a rotation by angle zero."""
+    """Keys and queries as they are: a rotation by angle zero (of no dimension, where a head has an odd number of them)."""
+
+    def __init__(self, params, prefix):
+        odd = int(params["head_dim"]) % 2
+        super().__init__({**params, "head_dim": int(params["head_dim"]) + odd}, prefix)
+        if odd:
+            self.head_dim, self.rotary_dim = self.head_dim - 1, 0
 
     def _frequencies(self):
         return torch.zeros(self.rotary_dim // 2, dtype=torch.float32)

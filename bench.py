@@ -11,7 +11,8 @@ fraction of the measured HBM bandwidth.  Prints ONE JSON line.
 
 ``--designs`` instead of the benchmark: prefill and decode throughput of the Dosovik design beside Llama at equal
 layer sizes, and the design's own kernels beside Llama's like kernels with their fractions of the copy bandwidth.
-``--kavotar``: the same for the Kavotar design (attention with weights mixed across heads beside a decaying state with a
+``--tupunex``: the same for the Tupunex design (several residual streams, differential attention, latent attention), beside
+Llama and Tutezen.  ``--kavotar``: the same for the Kavotar design (attention with weights mixed across heads beside a decaying state with a
 bonus, matrix memories with exponential gates, routed experts), beside Llama and Kulivik.  ``--kulivik``: the same for the Kulivik design (windowed, biased and convolved attention, linear attention with constant
 decays, routed experts), beside Llama and Bumolix.  ``--bumolix``: the same for the Bumolix design (attention beside gated linear attention, selective-scan layers), beside
 Llama and Tutezen.  ``--tutezen``: the same for the Tutezen design (state-space and latent-attention layers, routed experts) at Llama's width
@@ -323,6 +324,24 @@ def kavotar_config(size: str, layers: int, vocab: int = 32768, chunk: int = 1024
             "layers": [pair[i % 2] for i in range(layers)]}
 
 
+def tupunex_config(size: str, layers: int, vocab: int = 32768, window: int = 1024, streams: int = 2):
+    """A Tupunex configuration of the width and feed-forward size of ``size`` on ``streams`` residual streams: differential
+    attention (as many elements of q, k and v as the heads of ``size``, in maps of 64 and values of 128, windows of
+    ``window``, 4 taps, capped scores) alternates with latent attention over all keys that caches 224 + 32 elements a token;
+    every layer has the dense feed-forward, the middle two run twice."""
+    H, I, nq, nkv, d = DESIGN_SIZES[size]
+    att = {"heads": nq * d // 128, "kv_heads": nkv * d // 128, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.4, "conv": 4,
+           "softcap": 50.0, "mask": {"size": window}}
+    lat = {"heads": 16, "dim": d, "rot_dim": 32, "vdim": d, "kv_rank": 224, "scale": (d + 32) ** -0.5, "rot": {"dims": 32, "base": 500000.0}}
+    mlp = {"kind": "dense", "ff": I}
+    pair = [{"type": "attention", "mixer": att, "mlp": mlp}, {"type": "latent_attention", "mixer": lat, "mlp": mlp}]
+    cfg = {"architecture": "Tupunex", "vocab": vocab, "width": H, "norm": {"eps": 1e-5}, "embedding": {"scale": H ** 0.5},
+           "streams": streams, "layers": [pair[i % 2] for i in range(layers)]}
+    if layers >= 4:
+        cfg["loop"] = {"start": layers // 2 - 1, "stop": layers // 2 + 1, "times": 2}
+    return cfg
+
+
 def design_comparison(args, other: str = "dosovik") -> int:
     """Prefill (one prompt of 2,048 tokens) and decode (8 requests, 2,048 tokens cached each, captured graphs)
     through the step function for both designs at each size; then single kernels.  Timing: CUDA events, the median
@@ -362,6 +381,10 @@ def design_comparison(args, other: str = "dosovik") -> int:
         if other == "kulivik":  # beside Llama (equal sizes) and Bumolix (the closest design: two mixers side by side)
             names = ("llama", "bumolix", other)
             pairs = (pairs[0], bumolix_config(size, layers), kulivik_config(size, layers))
+        if other == "tupunex":  # beside Llama (equal sizes) and Tutezen (latent attention too, and a stretch of layers that runs twice)
+            names = ("llama", "tutezen", other, other)
+            fewer = max(layers - 2, 2)
+            pairs = (pairs[0], tutezen_config(size, fewer), tupunex_config(size, fewer), tupunex_config(size, fewer, streams=4))
         if other == "kavotar":  # beside Llama (equal sizes) and Kulivik (the closest design: two mixers side by side, routed experts)
             names = ("llama", "kulivik", other)
             pairs = (pairs[0], kulivik_config(size, layers), kavotar_config(size, layers))
@@ -399,7 +422,7 @@ def design_comparison(args, other: str = "dosovik") -> int:
                 if hasattr(ff, "w_gate_up") and ff.w_gate_up.dim() == 3:
                     per = (ff.w_gate_up[0].numel() + ff.w_down[0].numel()) * 2
                     weights += per * min(ff.experts, batch * ff.top)
-            row = {"size": size, "design": name, "layers": layers, "prefill_tokens": prefill, "prefill_ms": round(pre_ms, 3),
+            row = {"size": size, "design": name, "layers": layers, **({"streams": cfg["streams"]} if "streams" in cfg else {}), "prefill_tokens": prefill, "prefill_ms": round(pre_ms, 3),
                    "prefill_tok_s": round(prefill / pre_ms * 1e3), "decode_batch": batch, "context": ctx_len,
                    "decode_ms_per_step": round(dec_ms, 4), "decode_tok_s": round(batch / dec_ms * 1e3),
                    "decode_weight_bytes_over_copy_bandwidth": round(weights / (dec_ms * 1e-3) / (hbm * 1e9), 3),
@@ -409,7 +432,7 @@ def design_comparison(args, other: str = "dosovik") -> int:
             del lm
             torch.cuda.empty_cache()
     kernels = {"tutezen": tutezen_kernels, "bumolix": bumolix_kernels, "kulivik": kulivik_kernels,
-               "kavotar": kavotar_kernels}.get(other, design_kernels)
+               "kavotar": kavotar_kernels, "tupunex": tupunex_kernels}.get(other, design_kernels)
     kernels(make_runtime("bfloat16", "cuda:0"), hbm, median_ms)
     return 0
 
@@ -587,9 +610,9 @@ def tutezen_kernels(rt, hbm, median_ms) -> None:
             ("llama:   SiLU * up", lambda: ops.silu_mul(gu, act, ctx.meta, T, I), T * I * 2 * 3, None),
             ("tutezen: GELU", lambda: ops.activation(z_up, act, "gelu_tanh", ctx.meta), T * I * 2 * 2, None),
             ("tutezen: latent rows (norm, rotation, pages, queries)",
-             lambda: ops.latent_rows(q_rot[:, :, 64:], q_abs, dkv, nrm, 1e-5, ctx, cache_t, 0, q_full, heads=lh, kv_rank=rank, rot_dim=rdim,
+             lambda: ops.latent_rows(q_rot[:, :, 64:], dkv, nrm, 1e-5, ctx, cache_t, 0, q_full, heads=lh, kv_rank=rank, rot_dim=rdim,
                                      padded=D, page_size=PAGE, num_pages=num_pages, store=True, inv_freq=fr, rotary_dims=rdim),
-             T * (lh * (rank + rdim) * 2 + (rank + rdim) * 2 + lh * D * 2 + 2 * D * 2), None),
+             T * (lh * rdim * 2 * 2 + (rank + rdim) * 2 + 2 * D * 2), None),
             ("llama:   rotation + pages", lambda: ops.rope_kv_store(qkv, ctx.positions, ctx.token_entry, ctx.meta, 0, inv_freq, cache_l, num_pages,
                                                                     T, 32, 8, 64, 64, PAGE, True), T * 48 * 64 * 2 * 2, None),
             ("tutezen: linear per head, 64 -> 224 (queries)", lambda: ops.head_linear(q_rot[:, :, :64], wgu[0, :lh * rank, :64].reshape(lh, rank, 64).contiguous(),
@@ -855,6 +878,112 @@ def kulivik_kernels(rt, hbm, median_ms) -> None:
     ops.check_status()
 
 
+def tupunex_kernels(rt, hbm, median_ms) -> None:
+    """The Tupunex layers' own kernels beside the framework's like kernels, alone, at width 2048 (the sizes of
+    ``tupunex_config("w2048-h64", ...)``): microseconds a call and the fraction of the copy bandwidth that the bytes each
+    must move give; for the attention kernels the rate of the arithmetic that the design asks for.  Rows of 16,384 tokens
+    and of 8 tokens (a decode step: the time of a launch inside a graph)."""
+    import torch
+
+    sys.path.insert(0, os.path.join(ROOT, "tests"))
+    import kernel_utils as K
+    from atoma_infer_b200.parts.base import PendingSum, StreamMix
+
+    ops, dev, bf = rt.ops, rt.device, torch.bfloat16
+    H, taps = 2048, 4
+    heads, kvh, md, dv, dp = 16, 4, 64, 128, 128     # differential attention: two maps of 64 a head, values of 128
+    N = (heads + kvh) * 2 * md + kvh * dv
+    nq, nkv, d = 32, 8, 64
+    lh, rank, rdim, D = 16, 224, 32, 256
+    print(f"kernels alone (copy bandwidth {hbm:.0f} GB/s): name, rows, us, bytes moved / time / copy bandwidth, or the rate")
+    for T in (16384, 8):
+        entries = [(0, T)] if T > 64 else [(100 + i, 1) for i in range(T)]
+        S = len(entries)
+        tables, num_pages = K.scrambled_tables([c + n for c, n in entries], PAGE, 0)
+        ctx, _ = K.make_context(rt, entries, PAGE, tables)
+        rnd = lambda *shape: torch.randn(*shape, device=dev)  # noqa: E731
+        resid, w, a, b = rnd(T, H), torch.ones(H, device=dev), rnd(T, H).to(bf), rnd(T, H).to(bf)
+        out = torch.empty(T, H, device=dev, dtype=bf)
+        mixes = {s: (rnd(T, s * H), StreamMix(PendingSum((a,)), torch.ones(H, device=dev), torch.eye(s, device=dev) * 0.9 + 0.1 / s,
+                                               torch.ones(s, device=dev)), torch.full((s,), 1.0 / s, device=dev)) for s in (1, 2, 4)}
+        rows = rnd(T, N + heads).to(bf)
+        bias, cw, ring = torch.ones(N, device=dev), rnd(taps, N), torch.zeros(S, taps - 1, N, device=dev)
+        q_maps, c_maps = torch.empty(T, heads * 2 * dp, device=dev, dtype=bf), torch.zeros(num_pages, 2, kvh, PAGE, dp, device=dev, dtype=bf)
+        two, one_out, lam = rnd(T, heads * 2 * dp).to(bf), torch.empty(T, heads * dv, device=dev, dtype=bf), torch.tensor([0.4], device=dev)
+        qkv = rnd(T, (nq + 2 * nkv) * d).to(bf)
+        cache = torch.zeros(num_pages, 2, nkv, PAGE, d, device=dev, dtype=bf)
+        q_out, inv_freq = torch.empty(T, nq * d, device=dev, dtype=bf), torch.ones(d // 2, device=dev)
+        k_w, k_ring, k_out = rnd(taps, (nq + 2 * nkv) * d), torch.zeros(S, taps - 1, (nq + 2 * nkv) * d, device=dev), torch.empty(T, (nq + 2 * nkv) * d, device=dev, dtype=bf)
+        g_o, g_gate, g_w, g_y = rnd(T, H), rnd(T, H).to(bf), torch.ones(128, device=dev), torch.empty(T, H, device=dev, dtype=bf)
+        q_rot, q_abs, dkv = rnd(T, lh, 64 + rdim).to(bf), rnd(T, lh, rank).to(bf), rnd(T, rank + rdim).to(bf)
+        cache_t, q_full = torch.zeros(num_pages, 2, 1, PAGE, D, device=dev, dtype=bf), torch.empty(T, lh * D, device=dev, dtype=bf)
+        nrm, fr = torch.ones(rank, device=dev), torch.ones(rdim // 2, device=dev)
+        lat_o, w_uv, lat_out = rnd(T, lh, D).to(bf), (rnd(lh, 64, rank) * 0.05).to(bf), torch.empty(T, lh, 64, device=dev, dtype=bf)
+        gate_h, gate_c = rnd(T, lh).to(bf), rnd(T, lh, 64).to(bf)
+        mixed = lambda s: ops.stream_mix_norm(mixes[s][0], s, mixes[s][1], mixes[s][2], w, 1e-5, out, ctx.meta, T)  # noqa: E731
+        latent = lambda halves: ops.latent_rows(q_rot[:, :, 64:], dkv, nrm, 1e-5, ctx, cache_t, 0, q_full, heads=lh, kv_rank=rank,  # noqa: E731
+                                                rot_dim=rdim, padded=D, page_size=PAGE, num_pages=num_pages, store=True, inv_freq=fr,
+                                                rotary_dims=rdim, halves=halves)
+        lat_bytes = T * (lh * rdim * 2 * 2 + (rank + rdim) * 2 + 2 * D * 2)
+        uv_bytes = T * lh * (rank + 64) * 2 + lh * 64 * rank * 2
+        cases = [
+            ("tupunex: 1 stream mixed + RMSNorm of their sum", lambda: mixed(1), T * H * (4 + 2 + 4 + 2)),
+            ("tupunex: 2 streams mixed + RMSNorm of their sum", lambda: mixed(2), T * H * (2 * 4 + 2 + 2 * 4 + 2)),
+            ("tupunex: 4 streams mixed + RMSNorm of their sum", lambda: mixed(4), T * H * (4 * 4 + 2 + 4 * 4 + 2)),
+            ("tutezen: pending sum of two + RMSNorm", lambda: ops.sum_rmsnorm(resid, PendingSum((a, b), 0.5), w, 1e-5, out, ctx.meta, T), T * H * (4 + 2 + 2 + 4 + 2)),
+            ("llama:   add + RMSNorm", lambda: ops.add_rmsnorm(resid, a, w, 1e-5, out, ctx.meta, T), T * H * (4 + 2 + 4 + 2)),
+            ("tupunex: rows of two maps (bias, convolution of 4 taps + ring, pages)",
+             lambda: ops.map_rows(rows[:, :N], ctx, c_maps, 0, q_maps, heads=heads, kv_heads=kvh, maps=2, d=md, dv=dv, dp=dp, page_size=PAGE,
+                                  num_pages=num_pages, store_kv=True, bias=bias, conv_w=cw, ring=ring), T * (N + heads * 2 * dp + 2 * kvh * dp) * 2),
+            ("kulivik: convolution of 4 taps on q, k, v (+ ring)",
+             lambda: (ops.causal_conv_act(qkv, k_w, None, k_ring, ctx, k_out, act="none") or ops.causal_conv_save(qkv, k_ring, ctx, taps)),
+             T * (nq + 2 * nkv) * d * 2 * 2),
+            ("kulivik: attention rows (query temperature, pages; no rotation)",
+             lambda: ops.qkv_prepare(qkv, ctx, cache, 0, q_out, nq=nq, nkv=nkv, d=d, dv=d, dp=d, page_size=PAGE, num_pages=num_pages,
+                                     store_kv=True, eps=1e-6, q_temp=(0.25, 128)), T * (nq + 2 * nkv) * d * 2 * 2),
+            ("llama:   rotation + pages", lambda: ops.rope_kv_store(qkv, ctx.positions, ctx.token_entry, ctx.meta, 0, inv_freq,
+                                                                    cache, num_pages, T, nq, nkv, d, d, PAGE, True), T * (nq + 2 * nkv) * d * 2 * 2),
+            ("tupunex: difference of the maps, norm per head, gate per head",
+             lambda: ops.map_difference(two, rows[:, N:], lam, 0.6, 1e-5, one_out, ctx.meta, heads=heads, dp=dp), T * heads * (2 * dv + dv) * 2),
+            ("bumolix: norm per head, shared weight, SiLU gate (16 x 128)", lambda: ops.head_norm_gate(g_o, g_gate, g_w, 1e-5, g_y, ctx.meta, heads), T * H * (4 + 2 + 2)),
+            ("tupunex: latent rows (norm, rotation of halves, pages, queries)", lambda: latent(True), lat_bytes),
+            ("tutezen: latent rows (norm, rotation of neighbours, pages, queries)", lambda: latent(False), lat_bytes),
+            ("tupunex: linear per head, 224 -> 64 (values), gate per head", lambda: ops.head_linear(lat_o[:, :, :rank], w_uv, lat_out, ctx.meta, gate=gate_h), uv_bytes),
+            ("tutezen: linear per head, 224 -> 64 (values), gate per channel", lambda: ops.head_linear(lat_o[:, :, :rank], w_uv, lat_out, ctx.meta, gate=gate_c),
+             uv_bytes + T * lh * 64 * 2),
+        ]
+        for name, fn, nbytes in cases:
+            us = _graph_us(fn, n=16 if T <= 64 else 2)
+            print(f"  {name:76s} {T:5d} rows {us:9.1f} us  {nbytes / (us * 1e-6) / (hbm * 1e9):5.2f}")
+        del mixes
+    # attention: a prompt of T tokens (or T decode tokens over 2,048 cached ones).  The rate counts what the design asks for: a
+    # score of 64 and a value product of 128 for a map and key of differential attention.
+    for T in (16384, 64, 8):
+        entries = [(0, T)] if T > 64 else [(2047, 1)] * T
+        tables, num_pages = K.scrambled_tables([c + n for c, n in entries], PAGE, 1)
+        ctx, _ = K.make_context(rt, entries, PAGE, tables)
+        for name, n1, n2, hd, per, kw in (
+                ("llama:   attention, 32 x 64 over 8 x 64, all keys", nq, nkv, d, 2 * d, {}),
+                ("llama:   attention, 32 x 128 over 4 x 128, all keys", 2 * heads, kvh, dp, 2 * dp, {}),
+                ("llama:   attention, 32 x 128 over 4 x 128, window 1024", 2 * heads, kvh, dp, 2 * dp, {"window": 1024}),
+                ("tupunex: attention, 16 heads of two maps, window 1024", 2 * heads, kvh, dp, md + dv, {"window": 1024}),
+                ("tupunex: attention, 16 heads of two maps, window 1024, capped scores", 2 * heads, kvh, dp, md + dv, {"window": 1024, "softcap": 50.0}),
+                ("tutezen: latent attention, 16 x 256 over 1 x 256, window 1024 + sinks", lh, 1, D, 2 * D, {"window": 1024, "sink": torch.zeros(lh, device=dev)}),
+                ("tupunex: latent attention, 16 x 256 over 1 x 256, all keys", lh, 1, D, 2 * D, {})):
+            c = torch.randn(num_pages, 2, n2, PAGE, hd, device=dev).to(bf)
+            q, o = torch.randn(T, n1 * hd, device=dev).to(bf), torch.empty(T, n1 * hd, device=dev, dtype=bf)
+            if name.startswith("tupunex: attention"):
+                q.view(T, heads, 2, 2, md)[:, :, 0, 1] = 0
+                q.view(T, heads, 2, 2, md)[:, :, 1, 0] = 0
+            window = kw.pop("window", 0)
+            us = _graph_us(lambda: ops.attention(q, n1 * hd, c, ctx, 0, o, n1, n2, hd, PAGE, num_pages, window, 0.125, **kw), n=4)
+            keys = (window if window and T > window else T / 2) if T > 64 else min(window or 2048, 2048)
+            rate = 2.0 * T * n1 * per * keys / (us * 1e-6) / 1e12
+            moved = f"  {T * keys * n2 * 2 * hd * 2 / (us * 1e-6) / (hbm * 1e9):5.2f} of copy" if T <= 64 else ""
+            print(f"  {name:76s} {T:5d} rows {us:9.1f} us         {rate:7.1f} TFLOP/s{moved}")
+    ops.check_status()
+
+
 def kavotar_kernels(rt, hbm, median_ms) -> None:
     """The Kavotar layers' own kernels beside the framework's like kernels, alone, at width 2048 (the sizes of
     ``kavotar_config("w2048-h64", ...)``): microseconds a call and the fraction of the copy bandwidth that the bytes each
@@ -1099,6 +1228,8 @@ def main() -> int:
                     help="the Kulivik design beside Llama and Bumolix at equal layer sizes through the step function, then its kernels alone")
     ap.add_argument("--kavotar", action="store_true",
                     help="the Kavotar design beside Llama and Kulivik at equal layer sizes through the step function, then its kernels alone")
+    ap.add_argument("--tupunex", action="store_true",
+                    help="the Tupunex design beside Llama and Tutezen at equal layer sizes through the step function, then its kernels alone")
     ap.add_argument("--kernels-alone", action="store_true", help="with an option that compares designs: only the kernels alone")
     ap.add_argument("--bumolix", action="store_true",
                     help="instead of the benchmark: prefill and decode throughput of the Bumolix design beside Llama and Tutezen "
@@ -1125,6 +1256,8 @@ def main() -> int:
         return design_comparison(args, other="tutezen")
     if args.bumolix:
         return design_comparison(args, other="bumolix")
+    if args.tupunex:
+        return design_comparison(args, other="tupunex")
     if args.kavotar:
         return design_comparison(args, other="kavotar")
     if args.kulivik:

@@ -339,7 +339,7 @@ class HostOps:
             y = y * (g if g.dim() == 3 else g[:, :, None])
         out[:n] = y.to(out.dtype)
 
-    def latent_rows(self, q_rot, q_abs, dkv, norm_w, eps, ctx, cache, group, q_out, *, heads, kv_rank, rot_dim, padded,
+    def latent_rows(self, q_rot, dkv, norm_w, eps, ctx, cache, group, q_out, *, heads, kv_rank, rot_dim, padded,
                     page_size, num_pages, store, inv_freq=None, rotary_dims=0, halves=False):
         self._count()
         meta = ctx.meta
@@ -364,9 +364,8 @@ class HostOps:
 
         c = PT.rms_divide(dkv[:n, :kv_rank].float(), eps) * norm_w
         key = torch.cat([c, turn(dkv[:n, kv_rank:].float())], -1)
-        q_out[:n] = 0
         qv = q_out[:n].view(n, heads, padded)
-        qv[..., :kv_rank] = q_abs[:n].to(q_out.dtype)
+        qv[..., kv_rank:] = 0
         qv[..., kv_rank:kv_rank + rot_dim] = turn(q_rot[:n].float()).to(q_out.dtype)
         if store:
             for t in range(n):

@@ -166,7 +166,7 @@ def test_norm_over_a_slice_and_linears_per_head(rts, dtype):
     rt = rts[dtype]
     tol = 1e-5 if dtype == "float32" else 1.5e-2
     g = torch.Generator().manual_seed(3)
-    for T in (5, 70):  # few rows: the own kernel; many rows in bfloat16: a batched library product
+    for T in (5, 19, 70):  # few rows: the own kernels; many rows in bfloat16: a batched library product
         entries = [(0, T - 1), (4, 1)]
         ctx, _ = K.make_context(rt, entries, 4, _tables(entries, 4)[0])
         x = torch.randn(T, 100, generator=g).to(rt.dtype)
@@ -174,7 +174,7 @@ def test_norm_over_a_slice_and_linears_per_head(rts, dtype):
         out = torch.empty(T, 40, dtype=rt.dtype, device=rt.device)
         rt.ops.rms_rows(x.to(rt.device)[:, 30:70], w.to(rt.device), 1e-6, out, ctx.meta)
         assert _err(out, PT.rms_divide(x[:, 30:70].double(), 1e-6) * w.double()) < tol
-        for heads, Kd, N in ((3, 20, 48), (5, 130, 24)):
+        for heads, Kd, N in ((3, 20, 48), (5, 130, 24), (4, 64, 40), (2, 136, 30), (1, 512, 16), (3, 520, 9)):
             xs = torch.randn(T, heads, Kd + 6, generator=g).to(rt.dtype)
             wh = (torch.randn(heads, N, Kd, generator=g) / math.sqrt(Kd)).to(rt.dtype)
             gate = torch.randn(T, heads * N + 11, generator=g).to(rt.dtype)
@@ -186,14 +186,20 @@ def test_norm_over_a_slice_and_linears_per_head(rts, dtype):
             rt.ops.head_linear(xs.to(rt.device)[:, :, 2:2 + Kd], wh.to(rt.device), out, ctx.meta,
                                gate=gate.to(rt.device)[:, 11:].view(T, heads, N))
             assert _err(out, want * torch.sigmoid(gv.double())) < tol
+            # one number per head, into the first elements of wider heads
+            wide = torch.full((T, heads, N + 8), 7.0, dtype=rt.dtype, device=rt.device)
+            rt.ops.head_linear(xs.to(rt.device)[:, :, 2:2 + Kd], wh.to(rt.device), wide[:, :, :N], ctx.meta, gate=gate.to(rt.device)[:, 11:11 + heads])
+            assert _err(wide[:, :, :N], want * torch.sigmoid(gate[:, 11:11 + heads].double())[:, :, None]) < tol
+            assert bool((wide[:, :, N:] == 7.0).all())
     rt.ops.check_status()
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("heads,rank,rdim,rot,page", [(3, 48, 8, 8, 4), (2, 20, 16, 6, 8), (5, 32, 16, 0, 16), (2, 21, 10, 4, 4)])
-def test_latent_rows(rts, dtype, heads, rank, rdim, rot, page):
-    """Queries laid out for the attention kernels, the cached vector on both planes of its page, zeros behind both; the
-    rotation pairs neighbours, of the first `rot` rotated dimensions only."""
+@pytest.mark.parametrize("halves", [False, True])
+@pytest.mark.parametrize("heads,rank,rdim,rot,page", [(3, 48, 8, 8, 4), (2, 20, 16, 6, 8), (5, 32, 16, 0, 16), (2, 21, 10, 4, 4), (4, 24, 24, 24, 8)])
+def test_latent_rows(rts, dtype, heads, rank, rdim, rot, page, halves):
+    """Queries completed for the attention kernels (their first elements stay), the cached vector on both planes of its page,
+    zeros behind both; the rotation pairs neighbours, or the halves, of the first `rot` rotated dimensions only."""
     rt = rts[dtype]
     tol = 1e-5 if dtype == "float32" else 1e-2
     g = torch.Generator().manual_seed(rank)
@@ -210,11 +216,24 @@ def test_latent_rows(rts, dtype, heads, rank, rdim, rot, page):
     cache = torch.full((num_pages, 2, 1, page, D), float("nan"), dtype=rt.dtype, device=rt.device)
     q_out = torch.full((T, heads * D), float("nan"), dtype=rt.dtype, device=rt.device)
     dev = lambda t: t.to(rt.device) if t is not None else None  # noqa: E731
-    rt.ops.latent_rows(dev(q)[:, :, 12:], dev(q_abs), dev(dkv)[:, 7:], dev(w), 1e-5, ctx, cache, 0, q_out, heads=heads, kv_rank=rank,
-                       rot_dim=rdim, padded=D, page_size=page, num_pages=num_pages, store=True, inv_freq=dev(inv_freq), rotary_dims=rot)
+    q_out.view(T, heads, D)[:, :, :rank] = dev(q_abs)
+    rt.ops.latent_rows(dev(q)[:, :, 12:], dev(dkv)[:, 7:], dev(w), 1e-5, ctx, cache, 0, q_out, heads=heads, kv_rank=rank,
+                       rot_dim=rdim, padded=D, page_size=page, num_pages=num_pages, store=True, inv_freq=dev(inv_freq), rotary_dims=rot, halves=halves)
     rt.ops.check_status()
     pos = torch.cat([torch.arange(c, c + n) for c, n in entries])
-    turn = (lambda v: PT.rotate_pairs(v.double(), pos, rot, 1e4)) if rot else (lambda v: v.double())  # noqa: E731
+    def turn(v):
+        if not rot:
+            return v.double()
+        if not halves:
+            return PT.rotate_pairs(v.double(), pos, rot, 1e4)
+        order = torch.arange(rot).view(2, rot // 2).t().reshape(-1)   # i and i + rot / 2 become neighbours, and go back
+        mixed = v.double().clone()
+        mixed[..., :rot] = v.double()[..., order]
+        out = PT.rotate_pairs(mixed, pos, rot, 1e4)
+        back = out.clone()
+        back[..., order] = out[..., :rot]
+        return back
+
     want_q = torch.zeros(T, heads, D, dtype=torch.float64)
     want_q[..., :rank], want_q[..., rank:rank + rdim] = q_abs.double(), turn(q[:, :, 12:])
     assert _err(q_out.view(T, heads, D), want_q) < tol
