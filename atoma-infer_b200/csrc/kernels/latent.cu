@@ -110,7 +110,7 @@ template <int P>
 __global__ void __launch_bounds__(128)
 head_linear_few_kernel(const __nv_bfloat16* __restrict__ x, long long xs_t, long long xs_h, const __nv_bfloat16* __restrict__ w,
                        __nv_bfloat16* __restrict__ y, long long ys_t, long long ys_h, const __nv_bfloat16* __restrict__ gate, long long gs_t,
-                       long long gs_h, int gate_per_head, const int* __restrict__ meta, int K, int N) {
+                       long long gs_h, int gate_per_head, const int* __restrict__ meta, int K, int N, int xvec) {
     __shared__ __align__(16) __nv_bfloat16 xs[8][64 * P];
     const int tid = threadIdx.x, lane = tid & 7, t0 = blockIdx.x * 8, h = blockIdx.y, n = blockIdx.z * 16 + tid / 8;
     const int rows = min(8, meta[META_NUM_TOKENS] - t0), pieces = K / 8;
@@ -121,9 +121,21 @@ head_linear_few_kernel(const __nv_bfloat16* __restrict__ x, long long xs_t, long
     pdl_wait();
     pdl_launch_dependents();
     if (rows <= 0) return;
-    for (int m = 0; m < 8; ++m)
-        for (int k = tid; k < 64 * P; k += 128)
-            xs[m][k] = m < rows && k < K ? x[(size_t)(t0 + m) * xs_t + (size_t)h * xs_h + k] : __float2bfloat16(0.f);
+    if (xvec) {  // the rows' slices start on 16 bytes
+#pragma unroll
+        for (int it = 0; it < (8 * 8 * P + 127) / 128; ++it) {
+            const int idx = it * 128 + tid, m = idx / (8 * P), pc = idx % (8 * P);
+            if (m < 8) {
+                uint4 v = make_uint4(0, 0, 0, 0);
+                if (m < rows && pc < pieces) v = *reinterpret_cast<const uint4*>(x + (size_t)(t0 + m) * xs_t + (size_t)h * xs_h + pc * 8);
+                *reinterpret_cast<uint4*>(&xs[m][pc * 8]) = v;
+            }
+        }
+    } else {
+        for (int m = 0; m < 8; ++m)
+            for (int k = tid; k < 64 * P; k += 128)
+                xs[m][k] = m < rows && k < K ? x[(size_t)(t0 + m) * xs_t + (size_t)h * xs_h + k] : __float2bfloat16(0.f);
+    }
     __syncthreads();
     float acc[8];
 #pragma unroll
@@ -166,10 +178,11 @@ extern "C" int head_linear(const void* x, long long xs_t, long long xs_h, const 
     if (T <= 0) return 0;
     if (dtype == DT_BF16 && T < 64 && K % 8 == 0 && K <= 512 && ((uintptr_t)w & 15) == 0) {
         const dim3 few((T + 7) / 8, heads, (N + 15) / 16);
+        const int xvec = xs_t % 8 == 0 && xs_h % 8 == 0 && ((uintptr_t)x & 15) == 0;
 #define FEW_CASE(P)                                                                                                              \
         return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, head_linear_few_kernel<P>, few, 128, 0, stream, (const __nv_bfloat16*)x, xs_t, xs_h, \
                                       (const __nv_bfloat16*)w, (__nv_bfloat16*)y, ys_t, ys_h, (const __nv_bfloat16*)gate, gs_t, gs_h, gate_per_head, \
-                                      meta, K, N)
+                                      meta, K, N, xvec)
         if (K <= 64) FEW_CASE(1);
         if (K <= 128) FEW_CASE(2);
         if (K <= 256) FEW_CASE(4);
@@ -289,7 +302,7 @@ __device__ __forceinline__ float turned1(const T* p, int j, int rot, int halves,
 // A block takes one token.  `pairs`: sizes, strides and addresses are even, so a thread takes two neighbouring elements with
 // one access.
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 latent_rows_kernel(const T* __restrict__ q_rot, long long qs_t, long long qs_h, const T* __restrict__ dkv, long long dkv_stride,
                    const float* __restrict__ norm_w, float eps, const int* __restrict__ positions,
                    const int* __restrict__ token_entry, const int* __restrict__ meta, int group,
@@ -387,11 +400,12 @@ extern "C" int latent_rows(const void* q_rot, long long qs_t, long long qs_h, co
     const int elem = dtype == DT_F32 ? 4 : 2;
     const int pairs = rank % 2 == 0 && rdim % 2 == 0 && D % 2 == 0 && (!halves || rot % 4 == 0) && qs_t % 2 == 0 && qs_h % 2 == 0 &&
                       dkv_stride % 2 == 0 && (((uintptr_t)q_rot | (uintptr_t)dkv | (uintptr_t)q_out | (uintptr_t)cache) % (2 * elem)) == 0;
+    const int threads = T >= 512 ? 128 : 256;  // few tokens: the shortest path through a token
     if (dtype == DT_F32)
-        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<float>, T, 128, smem, stream, (const float*)q_rot, qs_t, qs_h,
+        return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<float>, T, threads, smem, stream, (const float*)q_rot, qs_t, qs_h,
                                       (const float*)dkv, dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq, rot, halves,
                                       (float*)q_out, (float*)cache, heads, rank, rdim, D, page_size, num_pages, store, pairs, status);
-    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<__nv_bfloat16>, T, 128, smem, stream, (const __nv_bfloat16*)q_rot,
+    return (int)launch_kernel_pdl((g_use_pdl & 5) != 0, latent_rows_kernel<__nv_bfloat16>, T, threads, smem, stream, (const __nv_bfloat16*)q_rot,
                                   qs_t, qs_h, (const __nv_bfloat16*)dkv, dkv_stride, norm_w, eps, positions, token_entry, meta, group, inv_freq,
                                   rot, halves, (__nv_bfloat16*)q_out, (__nv_bfloat16*)cache, heads, rank, rdim, D, page_size, num_pages, store,
                                   pairs, status);
