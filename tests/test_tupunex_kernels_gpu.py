@@ -80,7 +80,7 @@ def test_streams_mixed_and_normed(rts, dtype, S, H):
 
 
 # (heads, key/value heads, maps, map, value, taps): sizes that take 16-byte and 8-byte pieces and single elements
-ROWS = [(4, 2, 2, 16, 32, 4), (4, 2, 2, 48, 92, 3), (2, 1, 2, 12, 20, 2), (3, 1, 2, 9, 10, 3), (4, 4, 2, 32, 48, 1), (2, 2, 2, 64, 128, 0),
+ROWS = [(4, 2, 2, 16, 32, 4), (6, 2, 2, 44, 92, 3), (2, 1, 2, 12, 20, 2), (3, 1, 2, 9, 10, 3), (4, 4, 2, 32, 48, 1), (2, 2, 2, 64, 128, 0),
         (2, 1, 2, 8, 16, 6), (6, 3, 1, 24, 16, 4), (2, 1, 3, 8, 40, 3), (8, 2, 2, 64, 128, 4)]
 
 
